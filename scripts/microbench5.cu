@@ -1,6 +1,6 @@
-// microbench5.cu -- is the legacy warp-level integer MMA (mma.sync m16n8k32 u8 x s8 -> s32, SASS IMMA.16832) fast
+// microbench5.cu -- is the legacy warp-level integer MMA (mma.sync m16n8k32 u8 x s8 -> s32) fast
 // enough on a B200 to carry the decode GEMV's main loop?  Measures (1) the issue rate and latency of the instruction and
-// (2) a candidate inner loop: LDS.128 of packed INT4 weights + 8 LOP3 + LDS.128 of activation digits + 2 IMMA per
+// (2) a candidate inner loop: 16-byte shared loads of packed INT4 weights + 8 mask operations + 16-byte loads of activation digits + 2 integer MMAs per
 // 512-byte item, out of shared memory, 16 warps per SM.
 // build: nvcc -gencode arch=compute_100a,code=sm_100a -O3 -std=c++17 -lineinfo -o scripts/microbench5 scripts/microbench5.cu
 #include <cstdio>
@@ -91,7 +91,7 @@ static int rate(int warps, long long* cyc, int* sink) {
     CK(cudaDeviceSynchronize());
     CK(cudaMemcpy(&h, cyc, 8, cudaMemcpyDeviceToHost));
     const double per_sm = (double)h / ((double)iters * CHAINS * warps);
-    printf("IMMA.16832 u8*s8: %2d warps/SM x %d chains: %.2f cycles per MMA per SM (%.2f per SM sub-partition), %.0f int-ops/clk/SM; dependent-chain step %.1f cycles\n",
+    printf("m16n8k32 u8*s8: %2d warps/SM x %d chains: %.2f cycles per MMA per SM (%.2f per SM sub-partition), %.0f int-ops/clk/SM; dependent-chain step %.1f cycles\n",
            warps, CHAINS, per_sm, per_sm * 4, 16.0 * 8 * 32 * 2 / per_sm, (double)h / iters);
     return 0;
 }
@@ -118,6 +118,6 @@ int main() {
     rate<1>(16, cyc, sink); rate<2>(16, cyc, sink); rate<4>(16, cyc, sink);
     loop<2>("loads only", cyc, sink);
     loop<1>("loads + unpack", cyc, sink);
-    loop<0>("loads + unpack + IMMA", cyc, sink);
+    loop<0>("loads + unpack + MMA", cyc, sink);
     return 0;
 }

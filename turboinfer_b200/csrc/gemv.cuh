@@ -13,14 +13,14 @@
 //     prologue   x (fp32, optionally RMS-normalised with the reference's roundings) is converted ONCE per GEMV to
 //                24-bit block fixed point, x_k ~= s_x * xf_k with |xf_k| < 2^23, and stored in shared memory as three
 //                signed 8-bit digit planes (xf = d2*65536 + d1*256 + d0, every digit in [-128, 127])
-//     main loop  warp-level integer MMAs (mma.sync.m16n8k32 u8/s8 x s8 -> s32, SASS IMMA.16832): the A operand is 16
-//                weight columns x 32 k, stored in HBM in fragment order so that one LDS.128 per lane is the fragment (INT4:
+//     main loop  warp-level integer MMAs (mma.sync.m16n8k32 u8/s8 x s8 -> s32): the A operand is 16
+//                weight columns x 32 k, stored in HBM in fragment order so that one 16-byte load per lane is the fragment (INT4:
 //                of two MMAs -- `w & 0x0F0F0F0F` is the first, `w & 0xF0F0F0F0` the second, 16x too large, which a
 //                shift of its own accumulator undoes exactly); the B operand's 8 columns carry the three digit planes
 //                (5 columns idle: the tensor pipe has >10x headroom here).  Integer accumulation is exact and order-
 //                independent, so the result does not depend on how k is split over warps or (tensor-parallel) GPUs.
-//                B200 measurement (scripts/microbench5.cu): IMMA.16832 issues every ~2-3 cycles per SM; the loop runs at
-//                9 cycles per 512-byte item per SM out of shared memory (bound by the LDS wavefronts) = 2.4x the HBM
+//                B200 measurement (scripts/microbench5.cu): the integer MMA issues every ~2-3 cycles per SM; the loop runs at
+//                9 cycles per 512-byte item per SM out of shared memory (bound by the shared-memory wavefronts) = 2.4x the HBM
 //                rate.  The IDP4A loop it replaces needed 19-27 (scripts/microbench2/3.cu), the fp32 unpack before 18+.
 //     reduction  none across lanes: the C fragment of lane (g, t) already holds the sums of columns g, g+8 for digit
 //                planes 2t, 2t+1; one shared-memory integer atomic per (column, digit) when a warp leaves a group
@@ -158,7 +158,7 @@ struct QuadAcc {
 // INT4: a byte b = lo + 16 hi holds the nibbles of k and k + 32.  The low nibbles need their mask (4 LOP3); the high nibbles
 // are taken WITHOUT masking: b . x2 = lo . x2 + 16 hi . x2, and lo . x2 is one more MMA on the already masked registers, kept
 // in its own accumulator and subtracted when the group's sums are flushed -- exact, since everything is an integer.  One
-// extra IMMA (the tensor pipe is ~20 % busy in this loop) replaces four LOP3 on the ALU pipe.
+// extra MMA (the tensor pipe is ~20 % busy in this loop) replaces four mask operations on the ALU pipe.
 template <int BITS>
 __device__ __forceinline__ void kitem_mma(QuadAcc<BITS>& acc, int par, const uint4& w, const uint4& xv) {
     if constexpr (BITS == 4) {
@@ -498,8 +498,8 @@ __device__ __forceinline__ float gemv_stage_x_lean(const GemvArgs& a, const floa
     return s_x;
 }
 
-// consumers, main loop: one quad per warp per ring stage -- 4 k-items, each one LDS.128 of weights (the A fragments),
-// one LDS of digits (the B fragments) and 2 (INT4) / 1 (INT8) IMMA; when the warp's run over a group ends, the C
+// consumers, main loop: one quad per warp per ring stage -- 4 k-items, each one 16-byte load of weights (the A fragments),
+// one shared load of digits (the B fragments) and 2 (INT4) / 1 (INT8) integer MMAs; when the warp's run over a group ends, the C
 // fragments are added to the column sums in shared memory (no cross-lane reduction needed).
 // Where a warp starts in its slab: depends on the slab's geometry only, so the persistent kernel computes it BEFORE the
 // grid barrier (it holds an integer division).
@@ -521,8 +521,8 @@ __device__ __forceinline__ ConsumePlan make_consume_plan(const QLayout& L, const
 // DBG: 0 production; 1 = no MMAs, 2 = no barrier waits (stand-alone kernel experiments); 3 = timeline stamps through `dbg`
 // (the persistent kernel's debug instance; `xskip` then also takes the timing switches 8 = no MMAs, 16 = no digit loads).
 //
-// The loop is written for the instruction issue slots: a round is only 4 k-items per warp (4 LDS.128 of weights, 4 of
-// digits, 8 IMMA and -- INT4 -- 32 mask LOP3), so every instruction of bookkeeping around them shows: the first version of
+// The loop is written for the instruction issue slots: a round is only 4 k-items per warp (4 16-byte loads of weights, 4 of
+// digits, 8 integer MMAs and -- INT4 -- 32 masks), so every instruction of bookkeeping around them shows: the first version of
 // this loop ran ~170 instructions per round and warp and was issue-bound at 0.8 us per stage with the whole ring already in
 // shared memory (profiles/r02_timeline_*: `rounds`).  Hence: barrier and stage addresses as 32-bit shared-window values
 // advanced incrementally, the per-round offset sum (REDUX) only on rounds that can be ragged -- a warp whose quad is not in

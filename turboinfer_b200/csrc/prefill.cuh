@@ -155,7 +155,7 @@ __global__ void __launch_bounds__(kPfThreads, 1) causal_attention_kernel(const f
         }
         __syncthreads();
         // S = Q K^T for 8 queries x 4 keys
-        // (packed fp32x2 FMAs, SASS FFMA2: two fma.rn per instruction, bit-identical to the scalar form)
+        // (packed fp32x2 FMAs: two fma.rn per instruction, bit-identical to the scalar form)
         f32x2 sacc2[8][2];
 #pragma unroll
         for (int i = 0; i < 8; ++i) sacc2[i][0] = sacc2[i][1] = pack2(0.f, 0.f);

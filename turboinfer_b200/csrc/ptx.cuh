@@ -1,5 +1,5 @@
 // ptx.cuh -- thin inline-PTX wrappers used by the sm_100a kernels: mbarrier, 1-D bulk async copy (TMA
-// engine, SASS UBLKCP), packed fp32x2 arithmetic (SASS FADD2 / FFMA2), lop3 / prmt bit tricks.
+// engine), packed fp32x2 arithmetic (add / fma .f32x2), lop3 / prmt bit tricks.
 #pragma once
 #include <cstdint>
 #include <cuda_runtime.h>
@@ -133,7 +133,7 @@ template <int N> __device__ __forceinline__ void reg_dealloc() { asm volatile("s
 __device__ __forceinline__ void pdl_wait_prior_grid() { asm volatile("griddepcontrol.wait;" ::: "memory"); }
 __device__ __forceinline__ void pdl_launch_dependents() { asm volatile("griddepcontrol.launch_dependents;" ::: "memory"); }
 
-// ---- packed fp32x2 (Blackwell FADD2 / FFMA2) ------------------------------------------------------
+// ---- packed fp32x2 (add.rn.f32x2 / fma.rn.f32x2) ------------------------------------------------------
 typedef unsigned long long f32x2;
 __device__ __forceinline__ f32x2 pack2(float lo, float hi) {
     f32x2 r;
