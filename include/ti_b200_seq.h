@@ -28,10 +28,12 @@ enum {
     TI_SEQ_MIXER_WKV = 1,       /* token-shifted linear recurrence, output read before the state is updated, bonus term */
     TI_SEQ_MIXER_GLA = 2,       /* gated linear attention: S <- diag(a) S + k v^T, o = S^T q, a = sigmoid(.)^(1/tau) per key channel */
     TI_SEQ_MIXER_HGRN2 = 3,     /* the same recurrence with the forget gate f as decay and 1 - f as the written key */
+    TI_SEQ_MIXER_SSM = 5,       /* state space: S <- exp(-exp(A) dt) S + dt B x^T, y = S^T C + D x, behind a short convolution (the ssm_* numbers below) */
     TI_SEQ_MIXER_LATENT = 4     /* softmax attention whose keys / values are linear images of a cached low-rank vector + one shared rotated key part */
 };
 enum {
     TI_SEQ_ACT_RELU = 0, TI_SEQ_ACT_SILU = 1, TI_SEQ_ACT_GELU_TANH = 2,
+    TI_SEQ_ACT_CLAMPED_SWISH = 4, /* gated form only: g = min(gate h, limit), u = up h cut to [-limit, limit], g sigmoid(1.702 g) (u + 1) */
     TI_SEQ_ACT_XIELU = 3 /* a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise; a = softplus(act[0]), b = 1/2 + softplus(act[1]) */
 };
 enum {
@@ -42,18 +44,25 @@ enum {
 };
 enum {
     TI_SEQ_ROUTE_SOFTMAX_ALL = 0, /* softmax over all router outputs, choice by score + correction inside the best groups, weights renormalised */
+    TI_SEQ_ROUTE_SIGMOID = 2,     /* sigmoid scores; choice by score + correction, a group is worth its two largest choice scores; chosen scores
+                                     renormalised, times route_scale */
     TI_SEQ_ROUTE_TOP_LOGITS = 1   /* logits + bias ("mlp.router.b"); the `top` largest are chosen, weights = softmax over the chosen logits */
 };
 enum {
     TI_SEQ_QK_NORM_NONE = 0,
     TI_SEQ_QK_NORM_HEAD = 1,   /* q and k divided by their RMS per head (after rotation), no weights */
+    TI_SEQ_QK_NORM_HEAD_GAIN = 3, /* q and k divided by their RMS per head BEFORE rotation, times one plain weight [dim] for all heads ("mix.q.norm" / "mix.k.norm") */
     TI_SEQ_QK_NORM_WHOLE = 2   /* RMS over the whole projection (all heads at once) times a plain weight "mix.q.norm" / "mix.k.norm" */
 };
 enum {
     TI_SEQ_NORMS_AROUND = 0, /* a norm in front of every sublayer ("norm1", "norm2") and one behind it ("norm1b", "norm2b") */
     TI_SEQ_NORMS_BEHIND = 1, /* the sublayers read the residual stream itself; one norm behind each ("norm1", "norm2") */
-    TI_SEQ_NORMS_FRONT = 2   /* one norm in front of every sublayer ("norm1", "norm2"), none behind it */
+    TI_SEQ_NORMS_FRONT = 2,  /* one norm in front of every sublayer ("norm1", "norm2"), none behind it */
+    TI_SEQ_NORMS_SHARED = 3  /* one norm a layer ("norm1") whose output both sublayers read: x <- x + mixer(norm(x)) + ff(norm(x)) */
 };
+enum { TI_SEQ_WEIGHTS_SOFTMAX = 0, TI_SEQ_WEIGHTS_SIGMOID = 1 /* a visible key's weight is sigmoid(score + "mix.pb"[head]), not normalised */ };
+enum { TI_SEQ_BIAS_NONE = 0, TI_SEQ_BIAS_QKVO = 1, TI_SEQ_BIAS_QKV = 2 };
+enum { TI_SEQ_EXPERT_GATED = 0 /* down(silu(gate h) * up h) */, TI_SEQ_EXPERT_RELU2 = 1 /* down(max(up h, 0)^2) */ };
 enum {
     TI_SEQ_NORM_SCALAR = 0 /* one gain for all coordinates */, TI_SEQ_NORM_ONE_PLUS = 1 /* per-coordinate gain stored as w, applied as 1 + w */,
     TI_SEQ_NORM_VECTOR = 2 /* per-coordinate gain applied as it is stored */
@@ -72,7 +81,9 @@ typedef struct ti_seq_layer_desc {
     int32_t window;          /* attention: a position sees itself and the window - 1 before it; 0 = everything before it */
     int32_t rot_dims;        /* leading coordinates of each head that are rotated, paired (2i, 2i+1); 0 = no rotation */
     float rot_base;
-    int32_t rot_scaled;      /* 1: wavelength-dependent slow-down of the frequencies with the four numbers below */
+    int32_t rot_scaled;      /* 1: wavelength-dependent slow-down of the frequencies with the four numbers below; 2: the same by turns over the
+                                original context (pairs of more than rot_high turns stay, of fewer than rot_low are divided by rot_factor, a
+                                ramp over the pair index between) */
     float rot_factor, rot_low, rot_high, rot_original;
     int32_t qk_norm;         /* TI_SEQ_QK_NORM_* */
     int32_t out_gate;        /* 1: head output times sigmoid of a per-head projection of the mixer input */
@@ -112,12 +123,27 @@ typedef struct ti_seq_layer_desc {
     int32_t rot_half;        /* 1: rotated coordinate i pairs with i + rot_dims / 2 instead of (2i, 2i + 1) */
     float rot_linear;        /* > 0: every frequency is divided by this number (independent of the wavelength) */
     /* -- attention -- */
-    int32_t proj_bias;       /* 1: the q, k, v and output projections add biases ("mix.q.b", "mix.k.b", "mix.v.b", "mix.o.b") */
+    int32_t proj_bias;       /* TI_SEQ_BIAS_*: the q, k, v (and output) projections add biases ("mix.q.b", "mix.k.b", "mix.v.b", "mix.o.b") */
     int32_t v_norm;          /* 1: every value head is divided by its RMS (no weight) before it is cached */
     int32_t head_temp;       /* 1: the scaled score of query head h is multiplied by "mix.temp"[h] */
     /* -- latent attention (`window` and `out_gate` above apply to it as well: "mix.g" [heads][width]) -- */
     int32_t q_rank;          /* > 0: queries through a low-rank vector: q = Uq norm(Dq h) ("mix.dq" [q_rank][width], "mix.dq.norm",
                                 "mix.uq" [heads * (dim + rot_dims)][q_rank]); 0: "mix.q" */
+    /* -- attention -- */
+    int32_t weights_kind;    /* TI_SEQ_WEIGHTS_* */
+    float rot_amp;           /* > 0: factor on the rotation's cosine and sine */
+    /* -- state space mixer: alone (mixer = TI_SEQ_MIXER_SSM) or, with ssm_heads > 0, beside the attention mixer; tensors "mix.<x>" alone,
+          "mix.left.<x>" (attention) and "mix.right.<x>" (state space) side by side: left_scale * attention + right_scale * state space -- */
+    int32_t ssm_heads, ssm_vdim, ssm_state, ssm_groups; /* "in" rows: [z | x | B | C | dt], x = heads * vdim, B = C = groups * state */
+    int32_t ssm_taps;        /* convolution over x, B and C ("conv" [channels][taps], "conv.b", silu) */
+    int32_t ssm_parts;       /* the gated output is normed in this many equal parts */
+    float left_scale, right_scale;
+    /* -- feed-forward -- */
+    float ff_limit;          /* TI_SEQ_ACT_CLAMPED_SWISH */
+    int32_t expert_form;     /* TI_SEQ_EXPERT_* (the shared expert has the same form) */
+    float route_scale;       /* > 0: factor on the routing weights */
+    /* -- the whole layer -- */
+    int32_t weights_of;      /* 1 + j: the layer has no tensors of its own and uses layer j's, with a cache / state of its own; 0: own tensors */
 } ti_seq_layer_desc;
 
 typedef struct ti_seq_model_desc {
@@ -142,6 +168,7 @@ typedef struct ti_seq_model_desc {
                                 reads u = sum_s hcq.in[s] X_s and, with its result y, all copies are rewritten at once from the old ones:
                                 X_t <- sum_s hcq.mix[s][t] X_s + hcq.out[t] y ("l<i>.hc1.*" mixer, "l<i>.hc2.*" feed-forward); the model's
                                 output is sum_s X_s.  Needs TI_SEQ_NORMS_FRONT.  0: one residual stream, x <- x + y */
+    float embed_scale;       /* > 0: factor on the embedding table's rows */
 } ti_seq_model_desc;
 
 int ti_seq_init(int device);

@@ -4,7 +4,8 @@
 //   - ragged steps: a block owns up to 128 consecutive rows of ONE sequence (tiles[2 i] = first row, tiles[2 i + 1] = count),
 //   - grouped key/value heads, a sliding window (only the pages the tile's rows can see are visited),
 //   - the per-head sigmoid output gate and the sink term of the softmax denominator.
-// Scores, softmax and the running sums are fp32.  Head sizes 64 and 128 with dim == vdim; other shapes use the fp32 tiled kernel.
+// Scores, softmax and the running sums are fp32.  Query/key and value sizes up to 128 in fours, each padded with zeros to 64 or 128 (the
+// template's sizes; SIZED: they are the layer's own); other shapes use the fp32 tiled kernel.
 // Also here: the split-key attention of decode rows (flash-decoding: key chunks in parallel, then a merge).
 #pragma once
 #include "prefill.cuh"
@@ -14,18 +15,20 @@ namespace tib {
 namespace seq {
 
 constexpr int kAttnTcTile = kTcQ;   // 128 rows a block
+template <int DK, int DV> constexpr size_t window_h3_smem_bytes() { return 2 * sizeof(__half) * ((size_t)(kTcQ + kTcKT) * (DK + 8) + (size_t)kTcKT * (DV + 8)); }
 
-template <int DH>
+template <int DK, int DV, bool SIZED>
 __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(const float* qkvg, StepMeta m, AttnShape s, const int* tiles,
                                                                              const float* k_pool, const float* v_pool, float* out) {
-    constexpr int LD = DH + 8, KS = DH / 16, NT = DH / 8;
+    constexpr int LD = DK + 8, LDV = DV + 8, KS = DK / 16, NT = DV / 8;
+    const int d = SIZED ? DK : s.dim, dv = SIZED ? DV : s.vdim;
     extern __shared__ __align__(16) __half h3w_smem[];
     __half* Qh = h3w_smem;                 // [128][LD]
     __half* Ql = Qh + kTcQ * LD;
     __half* Kh = Ql + kTcQ * LD;           // [64][LD]
     __half* Kl = Kh + kTcKT * LD;
     __half* Vh = Kl + kTcKT * LD;
-    __half* Vl = Vh + kTcKT * LD;
+    __half* Vl = Vh + kTcKT * LDV;
     const int row0 = tiles[2 * blockIdx.x], M = tiles[2 * blockIdx.x + 1], h = blockIdx.y;
     const int pos0 = m.row_pos[row0];
     const int* table = m.page_table + (size_t)m.ent_slot[m.row_ent[row0]] * m.table_stride;
@@ -38,11 +41,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
         *reinterpret_cast<uint2*>(hi) = make_uint2(pack_h2(a[0], a[1]), pack_h2(a[2], a[3]));
         *reinterpret_cast<uint2*>(lo) = make_uint2(pack_h2(b[0], b[1]), pack_h2(b[2], b[3]));
     };
-    for (int i = tid; i < kTcQ * (DH / 4); i += kTcThreads) {
-        const int q = i / (DH / 4), d4 = (i % (DH / 4)) * 4;
+    const float pb = s.pb ? s.pb[h] : 0.f;
+    for (int i = tid; i < kTcQ * (DK / 4); i += kTcThreads) {
+        const int q = i / (DK / 4), d4 = (i % (DK / 4)) * 4;
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (q < M) {
-            const float* src = qkvg + (size_t)(row0 + q) * s.ld + (size_t)h * DH + d4;   // (the row pitch need not be a multiple of 4)
+        if (q < M && d4 < d) {
+            const float* src = qkvg + (size_t)(row0 + q) * s.ld + (size_t)h * d + d4;   // (the row pitch need not be a multiple of 4)
             v = make_float4(src[0], src[1], src[2], src[3]);
         }
         store_split4(v, Qh + q * LD + d4, Ql + q * LD + d4);
@@ -59,22 +63,36 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
     const uint32_t* ql_row = reinterpret_cast<const uint32_t*>(Ql + (16 * warp + g) * LD) + t;
     const int lm = lane >> 3, lr = lane & 7;
     const uint32_t k_ld = (uint32_t)(((lr + 8 * (lm >> 1)) * LD + 8 * (lm & 1)) * 2);
-    const uint32_t v_ld = (uint32_t)(((lr + 8 * (lm & 1)) * LD + 8 * (lm >> 1)) * 2);
+    const uint32_t v_ld = (uint32_t)(((lr + 8 * (lm & 1)) * LDV + 8 * (lm >> 1)) * 2);
     const uint32_t kh_s = smem_u32(Kh), kl_s = smem_u32(Kl), vh_s = smem_u32(Vh), vl_s = smem_u32(Vl);
-    const size_t pitch = (size_t)s.kv_heads * DH;
+    const size_t kpitch = (size_t)s.kv_heads * d, vpitch = (size_t)s.kv_heads * dv;
     for (int t0 = lo / kPageTokens * kPageTokens; t0 <= last_pos; t0 += kTcKT) {   // a key tile = a page
         __syncthreads();
         const size_t tok0 = (size_t)table[t0 / kPageTokens] * kPageTokens;
-        for (int i = tid; i < kTcKT * (DH / 4); i += kTcThreads) {
-            const int kk = i / (DH / 4), d4 = (i % (DH / 4)) * 4, tk = t0 + kk;
-            float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), vv = kv;
-            if (tk >= lo && tk <= last_pos) {
-                const size_t row = (tok0 + kk) * pitch + (size_t)gkv * DH + d4;
-                kv = *reinterpret_cast<const float4*>(k_pool + row);
-                vv = *reinterpret_cast<const float4*>(v_pool + row);
+        if constexpr (DK == DV) {
+            for (int i = tid; i < kTcKT * (DK / 4); i += kTcThreads) {
+                const int kk = i / (DK / 4), d4 = (i % (DK / 4)) * 4, tk = t0 + kk;
+                float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), vv = kv;
+                if (tk >= lo && tk <= last_pos) {
+                    if (d4 < d) kv = *reinterpret_cast<const float4*>(k_pool + (tok0 + kk) * kpitch + (size_t)gkv * d + d4);
+                    if (d4 < dv) vv = *reinterpret_cast<const float4*>(v_pool + (tok0 + kk) * vpitch + (size_t)gkv * dv + d4);
+                }
+                store_split4(kv, Kh + kk * LD + d4, Kl + kk * LD + d4);
+                store_split4(vv, Vh + kk * LDV + d4, Vl + kk * LDV + d4);
             }
-            store_split4(kv, Kh + kk * LD + d4, Kl + kk * LD + d4);
-            store_split4(vv, Vh + kk * LD + d4, Vl + kk * LD + d4);
+        } else {
+            for (int i = tid; i < kTcKT * (DK / 4); i += kTcThreads) {
+                const int kk = i / (DK / 4), d4 = (i % (DK / 4)) * 4, tk = t0 + kk;
+                float4 kv = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (tk >= lo && tk <= last_pos && d4 < d) kv = *reinterpret_cast<const float4*>(k_pool + (tok0 + kk) * kpitch + (size_t)gkv * d + d4);
+                store_split4(kv, Kh + kk * LD + d4, Kl + kk * LD + d4);
+            }
+            for (int i = tid; i < kTcKT * (DV / 4); i += kTcThreads) {
+                const int kk = i / (DV / 4), d4 = (i % (DV / 4)) * 4, tk = t0 + kk;
+                float4 vv = make_float4(0.f, 0.f, 0.f, 0.f);
+                if (tk >= lo && tk <= last_pos && d4 < dv) vv = *reinterpret_cast<const float4*>(v_pool + (tok0 + kk) * vpitch + (size_t)gkv * dv + d4);
+                store_split4(vv, Vh + kk * LDV + d4, Vl + kk * LDV + d4);
+            }
         }
         __syncthreads();
         if (t0 > warp_last || t0 + kTcKT - 1 < warp_lo || 16 * warp >= M) continue;   // nothing of this page is visible to the warp's rows
@@ -102,16 +120,33 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
         const int qp0 = pos0 + r0, qp1 = pos0 + r1;
         const int w = s.window > 0 ? s.window : 0x3FFFFFFF;
         float mx0 = -INFINITY, mx1 = -INFINITY;
+        if (s.softcap > 0.f) {   // (a multiplication by the scale commutes with nothing here: the cap takes the scaled score)
+#pragma unroll
+            for (int j = 0; j < kTcKT / 8; ++j)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sc[j][i] = s.softcap * tanhf(sc[j][i] * s.scale / s.softcap);
+        } else {
+#pragma unroll
+            for (int j = 0; j < kTcKT / 8; ++j)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sc[j][i] *= s.scale;
+        }
 #pragma unroll
         for (int j = 0; j < kTcKT / 8; ++j) {
             const int key = t0 + 8 * j + 2 * t;
-            sc[j][0] = (key <= qp0 && key > qp0 - w && r0 < M) ? sc[j][0] * s.scale : -INFINITY;
-            sc[j][1] = (key + 1 <= qp0 && key + 1 > qp0 - w && r0 < M) ? sc[j][1] * s.scale : -INFINITY;
-            sc[j][2] = (key <= qp1 && key > qp1 - w && r1 < M) ? sc[j][2] * s.scale : -INFINITY;
-            sc[j][3] = (key + 1 <= qp1 && key + 1 > qp1 - w && r1 < M) ? sc[j][3] * s.scale : -INFINITY;
+            sc[j][0] = (key <= qp0 && key > qp0 - w && r0 < M) ? sc[j][0] : -INFINITY;
+            sc[j][1] = (key + 1 <= qp0 && key + 1 > qp0 - w && r0 < M) ? sc[j][1] : -INFINITY;
+            sc[j][2] = (key <= qp1 && key > qp1 - w && r1 < M) ? sc[j][2] : -INFINITY;
+            sc[j][3] = (key + 1 <= qp1 && key + 1 > qp1 - w && r1 < M) ? sc[j][3] : -INFINITY;
             mx0 = fmaxf(mx0, fmaxf(sc[j][0], sc[j][1]));
             mx1 = fmaxf(mx1, fmaxf(sc[j][2], sc[j][3]));
         }
+        if (s.pb) {   // no softmax: sigmoid of the score and the head's number (0 for a key that is not visible)
+#pragma unroll
+            for (int j = 0; j < kTcKT / 8; ++j)
+#pragma unroll
+                for (int i = 0; i < 4; ++i) sc[j][i] = sc[j][i] == -INFINITY ? 0.f : attn_sigmoid(sc[j][i], pb);
+        } else {
         mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1)); mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
         mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1)); mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
         const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
@@ -134,6 +169,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
         m1 = mn1;
 #pragma unroll
         for (int n = 0; n < NT; ++n) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
+        }
 #pragma unroll
         for (int jp = 0; jp < kTcKT / 16; ++jp) {
             uint32_t ph[4], pl[4];
@@ -149,7 +185,7 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
 #pragma unroll
             for (int np = 0; np < NT / 2; ++np) {
                 uint32_t bh[4], bl[4];
-                const uint32_t off = (uint32_t)((16 * jp * LD + 16 * np) * 2) + v_ld;
+                const uint32_t off = (uint32_t)((16 * jp * LDV + 16 * np) * 2) + v_ld;
                 ldsm_x4_trans(bh, vh_s + off);
                 ldsm_x4_trans(bl, vl_s + off);
                 mma_f16(o[2 * np], pl, bh[0], bh[1]);
@@ -164,11 +200,20 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
     float i0 = 0.f, i1 = 0.f;
     if (r0 < M) i0 = attn_gate(s, qkvg, row0 + r0, h) * attn_finish_factor(s, h, m0, l0);
     if (r1 < M) i1 = attn_gate(s, qkvg, row0 + r1, h) * attn_finish_factor(s, h, m1, l1);
-    const size_t opitch = (size_t)s.heads * DH;
+    const size_t opitch = attn_out_stride(s);
+    const bool pair = SIZED && (opitch & 1) == 0 && (reinterpret_cast<uintptr_t>(out) & 7) == 0;
+    float* o0 = out + (size_t)(row0 + r0) * opitch + (size_t)h * dv;
+    float* o1 = o0 + 8 * opitch;
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
-        if (r0 < M) *reinterpret_cast<float2*>(out + (size_t)(row0 + r0) * opitch + (size_t)h * DH + 8 * n + 2 * t) = make_float2(o[n][0] * i0, o[n][1] * i0);
-        if (r1 < M) *reinterpret_cast<float2*>(out + (size_t)(row0 + r1) * opitch + (size_t)h * DH + 8 * n + 2 * t) = make_float2(o[n][2] * i1, o[n][3] * i1);
+        const int c = 8 * n + 2 * t;
+        if (pair) {
+            if (r0 < M) *reinterpret_cast<float2*>(o0 + c) = make_float2(o[n][0] * i0, o[n][1] * i0);
+            if (r1 < M) *reinterpret_cast<float2*>(o1 + c) = make_float2(o[n][2] * i1, o[n][3] * i1);
+        } else if (c < dv) {   // (dv in fours: c + 1 < dv too)
+            if (r0 < M) { o0[c] = o[n][0] * i0; o0[c + 1] = o[n][1] * i0; }
+            if (r1 < M) { o1[c] = o[n][2] * i1; o1[c + 1] = o[n][3] * i1; }
+        }
     }
 }
 
@@ -197,7 +242,8 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_split_kernel
     const int lo = (s.window > 0 && pos - s.window + 1 > 0) ? pos - s.window + 1 : 0;
     const int chunk = (pos - lo + 1 + splits - 1) / splits;
     const int j0 = lo + z * chunk, j1 = min(pos, j0 + chunk - 1);
-    float mx = -INFINITY, l = 0.f;
+    float mx = s.pb ? 0.f : -INFINITY, l = 0.f;   // (weights without a softmax: the running maximum stays 0)
+    const float pb = s.pb ? s.pb[h] : 0.f;
     const size_t kstride = (size_t)s.kv_heads * s.dim, vstride = attn_vstride(s);
     // a warp takes its keys four at a time: the four K rows (and then the four V rows) are requested together
     for (int jb = j0 + 4 * warp; jb <= j1; jb += 4 * kAttnWarps) {
@@ -226,10 +272,10 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_split_kernel
         }
 #pragma unroll
         for (int u = 0; u < 4; ++u) {
-            const float su = warp_sum(sc[u]) * s.scale;
+            const float su = attn_score(s, warp_sum(sc[u]));
             if (jb + u <= j1) {
-                const float nm = fmaxf(mx, su);
-                const float corr = expf(mx - nm), p = expf(su - nm);
+                const float nm = s.pb ? 0.f : fmaxf(mx, su);
+                const float corr = expf(mx - nm), p = s.pb ? attn_sigmoid(su, pb) : expf(su - nm);
                 l = l * corr + p;
 #pragma unroll
                 for (int i = 0; i < PL; ++i) o[i] = fmaf(p, vv[u][i], o[i] * corr);
@@ -294,7 +340,7 @@ __global__ void attention_merge_kernel(const float* part, const float* qkvg, Ste
 #pragma unroll
         for (int z = 0; z < kMaxSplits; ++z)
             if (z < splits && d < s.vdim) acc = fmaf(p[(size_t)z * ps + 2 + d], fs[z], acc);
-        if (d < s.vdim) out[(size_t)t * (s.heads * s.vdim) + (size_t)h * s.vdim + d] = acc * fin;
+        if (d < s.vdim) out[(size_t)t * attn_out_stride(s) + (size_t)h * s.vdim + d] = acc * fin;
     }
 }
 

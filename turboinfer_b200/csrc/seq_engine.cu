@@ -24,6 +24,7 @@
 #include "seq_experts.cuh"
 #include "seq_headmix.cuh"
 #include "seq_hyper.cuh"
+#include "seq_ssm.cuh"
 #include "sampling.cuh"
 
 using namespace tib;
@@ -208,6 +209,13 @@ struct LayerW {
     const void* uq = nullptr;
     int off_dq = -1, ld_front = 0;             // ld_front: row stride of the fused front product's output (>= n_front: room for q behind it)
     const float *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
+    // norms in front of both sublayers at once: `front` is [mixer parts | second mixer's in | feed-forward front], `back` the output
+    // matrices side by side along K [mixer | second mixer | feed-forward], its width and where the parts' activations start
+    const void* back = nullptr;
+    DevBuf<uint8_t> back_buf;
+    int n_back = 0, back_ssm = -1, back_ff = -1, off_in = -1;
+    const float *qgain = nullptr, *kgain = nullptr, *pb = nullptr;   // attention: gains of the per-head norm, numbers of the sigmoid weights
+    const float *ssm_conv = nullptr, *ssm_conv_b = nullptr, *dt_bias = nullptr, *A_log = nullptr, *ssm_D = nullptr, *ssm_norm = nullptr;
     int mix_HP = 0;   // > 0: the layer's attention is the head-mixing one; register bound of its head count (8 / 16 / 32 / 64)
 };
 
@@ -217,6 +225,7 @@ struct Run {
     bool enters_pass = false;   // the looped block's input projection comes right before this run
     DevBuf<float> k_pool, v_pool;          // attention: [pages * 64][G * d], [pages * 64][G * dv]; latent attention: k_pool [pages * 64][rank + rot]
     DevBuf<float> state, prev;             // wkv: [slots][H][d][d], [slots][D]; gla / hgrn2: state [slots][H][dk][dv]
+    DevBuf<float> ssm_state, ssm_conv;     // state space: [slots][H][N][dv], and its convolution's [slots][taps - 1][channels]
     int kv_run = -1;                       // latent attention reading another layer's cache: the run that owns it
     DevBuf<float> conv_state;              // short convolution: [slots][taps - 1][D], the last inputs of every sequence
     DevBuf<float> conv_state2;             // the same for the convolution in front of the feed-forward
@@ -293,13 +302,22 @@ void require(Model& m, const std::string& name, std::vector<int64_t> shape, bool
     m.order.push_back(name);
 }
 
-bool is_recurrent(int mixer) { return mixer == TI_SEQ_MIXER_WKV || mixer == TI_SEQ_MIXER_GLA || mixer == TI_SEQ_MIXER_HGRN2; }
+// the layer has a state-space mixer (alone or beside the first mixer), its channels behind the convolution, and the rows of its input matrix
+bool has_ssm(const ti_seq_layer_desc& L) { return L.ssm_heads > 0; }
+int ssm_channels(const ti_seq_layer_desc& L) { return L.ssm_heads * L.ssm_vdim + 2 * L.ssm_groups * L.ssm_state; }
+int ssm_in_rows(const ti_seq_layer_desc& L) { return L.ssm_heads * L.ssm_vdim + ssm_channels(L) + L.ssm_heads; }
+// tensors of the two mixers of a layer: "mix." when there is one, "mix.left." / "mix.right." when there are two
+std::string mix_prefix(const ti_seq_layer_desc& L, bool second) {
+    if (!has_ssm(L) || L.mixer == TI_SEQ_MIXER_SSM) return "mix.";
+    return second ? "mix.right." : "mix.left.";
+}
 
 int describe_tensors(Model& m) {
     const int64_t D = m.d.width, V = m.d.vocab;
     if (m.d.norm_kind != TI_SEQ_NORM_SCALAR && m.d.norm_kind != TI_SEQ_NORM_ONE_PLUS && m.d.norm_kind != TI_SEQ_NORM_VECTOR) return fail("norm kind %d", m.d.norm_kind);
     const std::vector<int64_t> gain_shape = m.d.norm_kind != TI_SEQ_NORM_SCALAR ? std::vector<int64_t>{D} : std::vector<int64_t>{};
-    const bool front = m.d.norm_place == TI_SEQ_NORMS_FRONT;
+    const bool front = m.d.norm_place == TI_SEQ_NORMS_FRONT, shared = m.d.norm_place == TI_SEQ_NORMS_SHARED;
+    if (m.d.embed_scale < 0.f) return fail("embedding scale %g", m.d.embed_scale);
     if (m.d.streams < 0 || m.d.streams > kMaxStreams) return fail("%d residual streams (at most %d)", m.d.streams, kMaxStreams);
     if (m.d.streams > 0 && !front) return fail("hyper-connections are built for norms in front of the sublayers only");
     require(m, "embed", {V, D}, true);
@@ -309,8 +327,23 @@ int describe_tensors(Model& m) {
         const ti_seq_layer_desc& L = m.layers[i].d;
         const std::string p = "l" + std::to_string(i) + ".";
         const bool behind = m.d.norm_place == TI_SEQ_NORMS_BEHIND;
+        if (L.weights_of) {
+            const int j = L.weights_of - 1;
+            if (j < 0 || j >= m.d.n_layers || j == i || m.layers[j].d.weights_of) return fail("layer %d: uses the tensors of layer %d, which has none of its own", i, j);
+            if (m.d.side_dim > 0 || L.kv_from >= 0) return fail("layer %d: shared tensors are built without side input and without another layer's cache", i);
+            continue;
+        }
+        if (L.ssm_heads < 0 || (L.mixer == TI_SEQ_MIXER_SSM && !has_ssm(L))) return fail("layer %d: %d state-space heads", i, L.ssm_heads);
+        if (shared && ((L.mixer != TI_SEQ_MIXER_ATTENTION && L.mixer != TI_SEQ_MIXER_GLA && L.mixer != TI_SEQ_MIXER_SSM) || L.res_gate || L.layer_scale || L.conv_taps || L.out_gate ||
+                       L.talk || L.keep_first > 0 || L.qk_norm == TI_SEQ_QK_NORM_WHOLE || L.proj_bias == TI_SEQ_BIAS_QKVO || L.identity > 0 ||
+                       (L.ff > 0 && L.ff_kind != TI_SEQ_FF_GLU && L.ff_kind != TI_SEQ_FF_EXPERTS)))
+            return fail("layer %d: one norm for both sublayers is built for attention, gla and state-space mixers without output / residual gates, mixed heads, kept keys, short "
+                        "convolutions, output bias and layer scale, and for the gated and the routed feed-forward", i);
+        if (!shared && (has_ssm(L) || L.mixer == TI_SEQ_MIXER_SSM)) return fail("layer %d: the state-space mixer is built with one norm for both sublayers", i);
+        if (!shared && (L.ff_act == TI_SEQ_ACT_CLAMPED_SWISH || L.expert_form != TI_SEQ_EXPERT_GATED) && L.ff > 0 && L.ff_kind != TI_SEQ_FF_GLU && L.ff_kind != TI_SEQ_FF_EXPERTS)
+            return fail("layer %d: activation %d / expert form %d", i, L.ff_act, L.expert_form);
         require(m, p + "norm1", gain_shape, false);
-        if (!behind && !front) require(m, p + "norm1b", gain_shape, false);
+        if (!behind && !front && !shared) require(m, p + "norm1b", gain_shape, false);
         if (front && (L.res_gate || L.layer_scale || (L.mixer != TI_SEQ_MIXER_ATTENTION && L.mixer != TI_SEQ_MIXER_LATENT) || (L.ff > 0 && L.ff_kind != TI_SEQ_FF_GLU)))
             return fail("layer %d: norms in front of the sublayers only are built for attention / latent attention layers with a gated feed-forward, without residual gates and layer scale", i);
         for (int q = 1; q <= (m.d.streams > 0 ? (L.ff > 0 ? 2 : 1) : 0); ++q) {
@@ -336,12 +369,22 @@ int describe_tensors(Model& m) {
             if (L.dim <= 0 || L.vdim <= 0 || L.dim > 32 * kAttnMaxPerLane || L.vdim > 32 * kAttnMaxPerLane)
                 return fail("layer %d: head sizes %d / %d outside 1..%d", i, L.dim, L.vdim, 32 * kAttnMaxPerLane);
             if (L.rot_dims < 0 || L.rot_dims > L.dim || (L.rot_dims & 1)) return fail("layer %d: rot dims %d of %d", i, L.rot_dims, L.dim);
-            require(m, p + "mix.q", {(int64_t)L.heads * L.dim, D}, true);
-            require(m, p + "mix.k", {(int64_t)L.kv_heads * L.dim, D}, true);
-            require(m, p + "mix.v", {(int64_t)L.kv_heads * L.vdim, D}, true);
+            const std::string px = p + mix_prefix(L, false);
+            require(m, px + "q", {(int64_t)L.heads * L.dim, D}, true);
+            require(m, px + "k", {(int64_t)L.kv_heads * L.dim, D}, true);
+            require(m, px + "v", {(int64_t)L.kv_heads * L.vdim, D}, true);
             if (L.out_gate) require(m, p + "mix.g", {(int64_t)L.heads, D}, true);
-            require(m, p + "mix.o", {D, (int64_t)L.heads * L.vdim}, true);
-            if (L.qk_norm == TI_SEQ_QK_NORM_WHOLE) {
+            require(m, px + "o", {D, (int64_t)L.heads * L.vdim}, true);
+            if (L.weights_kind != TI_SEQ_WEIGHTS_SOFTMAX && L.weights_kind != TI_SEQ_WEIGHTS_SIGMOID) return fail("layer %d: attention weights %d", i, L.weights_kind);
+            if (L.weights_kind == TI_SEQ_WEIGHTS_SIGMOID) {
+                if (L.sink != TI_SEQ_SINK_NONE) return fail("layer %d: a sink belongs to a softmax", i);
+                require(m, px + "pb", {(int64_t)L.heads}, false);
+            }
+            if (L.rot_amp < 0.f || L.rot_scaled < 0 || L.rot_scaled > 2) return fail("layer %d: rotation factor %g, scaling kind %d", i, L.rot_amp, L.rot_scaled);
+            if (L.qk_norm == TI_SEQ_QK_NORM_HEAD_GAIN) {
+                require(m, px + "q.norm", {(int64_t)L.dim}, false);
+                require(m, px + "k.norm", {(int64_t)L.dim}, false);
+            } else if (L.qk_norm == TI_SEQ_QK_NORM_WHOLE) {
                 if (L.rot_dims > 0 || L.out_gate) return fail("layer %d: the whole-projection q / k norm is built without rotation and output gate", i);
                 require(m, p + "mix.q.norm", {(int64_t)L.heads * L.dim}, false);
                 require(m, p + "mix.k.norm", {(int64_t)L.kv_heads * L.dim}, false);
@@ -349,18 +392,20 @@ int describe_tensors(Model& m) {
             if (L.talk) require(m, p + "mix.talk", {(int64_t)L.heads, (int64_t)L.heads}, false);
             if (L.sink == TI_SEQ_SINK_LEARNED) require(m, p + "mix.sink", {(int64_t)L.heads}, false);
             if (L.proj_bias) {
-                require(m, p + "mix.q.b", {(int64_t)L.heads * L.dim}, false);
-                require(m, p + "mix.k.b", {(int64_t)L.kv_heads * L.dim}, false);
-                require(m, p + "mix.v.b", {(int64_t)L.kv_heads * L.vdim}, false);
-                require(m, p + "mix.o.b", {D}, false);
-                if (!front) return fail("layer %d: the output projection's bias is built with norms in front of the sublayers only", i);
+                require(m, px + "q.b", {(int64_t)L.heads * L.dim}, false);
+                require(m, px + "k.b", {(int64_t)L.kv_heads * L.dim}, false);
+                require(m, px + "v.b", {(int64_t)L.kv_heads * L.vdim}, false);
+                if (L.proj_bias != TI_SEQ_BIAS_QKV && L.proj_bias != TI_SEQ_BIAS_QKVO) return fail("layer %d: projection biases %d", i, L.proj_bias);
+                if (L.proj_bias == TI_SEQ_BIAS_QKVO) require(m, p + "mix.o.b", {D}, false);
+                if (!front && L.proj_bias == TI_SEQ_BIAS_QKVO) return fail("layer %d: the output projection's bias is built with norms in front of the sublayers only", i);
             }
             if (L.head_temp) require(m, p + "mix.temp", {(int64_t)L.heads}, false);
             if ((L.proj_bias || L.head_temp || L.v_norm || L.rot_half) && L.qk_norm == TI_SEQ_QK_NORM_WHOLE)
                 return fail("layer %d: biases, per-head score factors, value norms and half-split rotation are built without the whole-projection q / k norm", i);
             if (L.keep_first < 0 || L.softcap < 0.f) return fail("layer %d: keep_first %d softcap %g", i, L.keep_first, L.softcap);
-            if (L.talk || L.softcap > 0.f || L.keep_first > 0) {   // the head-mixing kernel takes the layer
-                if (L.out_gate || L.qk_norm == TI_SEQ_QK_NORM_HEAD || L.rot_dims > 0) return fail("layer %d: capped / mixed scores and kept first keys are built without rotation, per-head norm and output gate", i);
+            if (L.talk || L.keep_first > 0) {   // the head-mixing kernel takes the layer
+                if (L.out_gate || L.qk_norm == TI_SEQ_QK_NORM_HEAD || L.qk_norm == TI_SEQ_QK_NORM_HEAD_GAIN || L.rot_dims > 0 || L.weights_kind != TI_SEQ_WEIGHTS_SOFTMAX)
+                    return fail("layer %d: mixed scores and kept first keys are built without rotation, per-head norm, output gate and sigmoid weights", i);
                 if (L.heads > 64) return fail("layer %d: %d heads exceed the 64 the head-mixing attention holds in registers", i, L.heads);
             }
         } else if (L.mixer == TI_SEQ_MIXER_WKV) {
@@ -422,16 +467,29 @@ int describe_tensors(Model& m) {
             require(m, p + "mix.uv", {(int64_t)L.heads * L.vdim, (int64_t)L.kv_rank}, true);
             if (L.sink == TI_SEQ_SINK_LEARNED) require(m, p + "mix.sink", {(int64_t)L.heads}, false);
             require(m, p + "mix.o", {D, (int64_t)L.heads * L.vdim}, true);
-        } else {
+        } else if (L.mixer != TI_SEQ_MIXER_SSM) {
             return fail("layer %d: unknown mixer %d", i, L.mixer);
+        }
+        if (has_ssm(L)) {
+            const std::string px = p + mix_prefix(L, true);
+            if (L.ssm_vdim <= 0 || L.ssm_state <= 0 || L.ssm_groups <= 0 || L.ssm_heads % L.ssm_groups || L.ssm_taps < 1 || L.ssm_parts <= 0 || (L.ssm_heads * L.ssm_vdim) % L.ssm_parts)
+                return fail("layer %d: state-space heads %d x %d, state %d, groups %d, taps %d, norm parts %d", i, L.ssm_heads, L.ssm_vdim, L.ssm_state, L.ssm_groups, L.ssm_taps, L.ssm_parts);
+            if (L.ssm_state > kSsmMaxState) return fail("layer %d: state size %d exceeds %d", i, L.ssm_state, kSsmMaxState);
+            const int64_t inner = (int64_t)L.ssm_heads * L.ssm_vdim, ch = ssm_channels(L);
+            require(m, px + "in", {(int64_t)ssm_in_rows(L), D}, true);
+            require(m, px + "conv", {ch, (int64_t)L.ssm_taps}, false);
+            require(m, px + "conv.b", {ch}, false);
+            for (const char* s : {"dt_bias", "A_log", "D"}) require(m, px + s, {(int64_t)L.ssm_heads}, false);
+            require(m, px + "norm", {inner}, false);
+            require(m, px + "o", {D, inner}, true);
         }
         if (L.res_gate) {
             require(m, p + "rg1", {D, D}, true);
             require(m, p + "rg1.b", {D}, false);
         }
         if (L.ff > 0) {
-            require(m, p + "norm2", gain_shape, false);
-            if (!behind && !front) require(m, p + "norm2b", gain_shape, false);
+            if (!shared) require(m, p + "norm2", gain_shape, false);
+            if (!behind && !front && !shared) require(m, p + "norm2b", gain_shape, false);
             if (behind && L.ff_kind != TI_SEQ_FF_DENSE && L.ff_kind != TI_SEQ_FF_EXPERTS) return fail("layer %d: norms behind the sublayers only are built for the dense and the routed feed-forward", i);
             if (L.ff_kind == TI_SEQ_FF_DENSE) {
                 if (L.ff_act != TI_SEQ_ACT_XIELU && L.ff_act != TI_SEQ_ACT_RELU && L.ff_act != TI_SEQ_ACT_SILU && L.ff_act != TI_SEQ_ACT_GELU_TANH)
@@ -440,6 +498,7 @@ int describe_tensors(Model& m) {
                 require(m, p + "mlp.down", {D, (int64_t)L.ff}, true);
                 if (L.ff_act == TI_SEQ_ACT_XIELU) require(m, p + "mlp.act", {2}, false);
             } else if (L.ff_kind == TI_SEQ_FF_GLU) {
+                if (L.ff_act == TI_SEQ_ACT_CLAMPED_SWISH && !(L.ff_limit > 0.f)) return fail("layer %d: feed-forward limit %g", i, L.ff_limit);
                 require(m, p + "mlp.gate", {(int64_t)L.ff, D}, true);
                 require(m, p + "mlp.up", {(int64_t)L.ff, D}, true);
                 require(m, p + "mlp.down", {D, (int64_t)L.ff}, true);
@@ -453,19 +512,21 @@ int describe_tensors(Model& m) {
                     return fail("layer %d: %d experts + %d identity, top %d, %d groups keep %d", i, L.experts, L.identity, L.top, L.groups, L.groups_keep);
                 for (int e = 0; e < L.experts; ++e) {
                     const std::string q = p + "mlp.e" + std::to_string(e) + ".";
-                    require(m, q + "gate", {(int64_t)L.ff, D}, true);
+                    if (L.expert_form == TI_SEQ_EXPERT_GATED) require(m, q + "gate", {(int64_t)L.ff, D}, true);
                     require(m, q + "up", {(int64_t)L.ff, D}, true);
                     require(m, q + "down", {D, (int64_t)L.ff}, true);
                 }
+                if (L.expert_form != TI_SEQ_EXPERT_GATED && L.expert_form != TI_SEQ_EXPERT_RELU2) return fail("layer %d: expert form %d", i, L.expert_form);
+                if (L.route_scale < 0.f) return fail("layer %d: router scale %g", i, L.route_scale);
                 require(m, p + "mlp.router", {(int64_t)n, D}, true);
                 if (L.route_kind == TI_SEQ_ROUTE_TOP_LOGITS) {
                     if (L.groups != 1 || L.groups_keep != 1) return fail("layer %d: the choice by logits has no groups", i);
                     require(m, p + "mlp.router.b", {(int64_t)n}, false);
-                } else if (L.route_kind == TI_SEQ_ROUTE_SOFTMAX_ALL) {
+                } else if (L.route_kind == TI_SEQ_ROUTE_SOFTMAX_ALL || L.route_kind == TI_SEQ_ROUTE_SIGMOID) {
                     require(m, p + "mlp.correction", {(int64_t)n}, false);
                 } else return fail("layer %d: router kind %d", i, L.route_kind);
                 if (L.shared_ff > 0) {
-                    require(m, p + "mlp.shared.gate", {(int64_t)L.shared_ff, D}, true);
+                    if (L.expert_form == TI_SEQ_EXPERT_GATED) require(m, p + "mlp.shared.gate", {(int64_t)L.shared_ff, D}, true);
                     require(m, p + "mlp.shared.up", {(int64_t)L.shared_ff, D}, true);
                     require(m, p + "mlp.shared.down", {D, (int64_t)L.shared_ff}, true);
                     if (!L.shared_plain) require(m, p + "mlp.shared.sg", {1, D}, true);
@@ -486,8 +547,9 @@ int describe_tensors(Model& m) {
     }
     require(m, "final.norm", gain_shape, false);
     if (!m.d.tied_head) require(m, "head", {V, D}, true);
-    if (m.d.norm_place != TI_SEQ_NORMS_AROUND && m.d.norm_place != TI_SEQ_NORMS_BEHIND && !front) return fail("norm placement %d", m.d.norm_place);
+    if (m.d.norm_place != TI_SEQ_NORMS_AROUND && m.d.norm_place != TI_SEQ_NORMS_BEHIND && !front && !shared) return fail("norm placement %d", m.d.norm_place);
     if (front && (m.d.side_dim > 0 || (m.d.loop_times > 0 && !m.d.loop_plain))) return fail("norms in front of the sublayers only are built without side input and without a projection between the passes of a looped block");
+    if (shared && (m.d.side_dim > 0 || (m.d.loop_times > 0 && !m.d.loop_plain) || m.d.norm_kind == TI_SEQ_NORM_ONE_PLUS)) return fail("one norm for both sublayers is built without side input, without a projection between the passes of a looped block, and for gains applied as they are stored");
     if (m.d.norm_place == TI_SEQ_NORMS_BEHIND && (m.d.loop_times > 0 || m.d.side_dim > 0)) return fail("norms behind the sublayers only are built without a looped block and side input");
     return 0;
 }
@@ -512,7 +574,12 @@ std::vector<float> rotary_frequencies(const ti_seq_layer_desc& L) {
     const double two_pi = 6.283185307179586476925286766559;
     for (size_t i = 0; i < f.size(); ++i) {
         double fi = std::pow((double)L.rot_base, -2.0 * (double)i / (double)L.rot_dims);
-        if (L.rot_scaled) {
+        if (L.rot_scaled == 2) {   // by the turns a pair makes over the original context: slow pairs are stretched, fast ones kept, a ramp between
+            const auto pair_with = [&](double turns) { return L.rot_dims * std::log(L.rot_original / (two_pi * turns)) / (2.0 * std::log((double)L.rot_base)); };
+            const double lo = std::max(std::floor(pair_with(L.rot_high)), 0.0), hi = std::min(std::ceil(pair_with(L.rot_low)), (double)L.rot_dims - 1.0);
+            const double ramp = std::min(1.0, std::max(0.0, ((double)i - lo) / std::max(hi - lo, 0.001)));
+            fi = fi / L.rot_factor * ramp + fi * (1.0 - ramp);
+        } else if (L.rot_scaled) {
             const double wl = two_pi / fi, orig = L.rot_original;
             if (wl > orig / L.rot_low) fi = fi / L.rot_factor;
             else if (!(wl < orig / L.rot_high)) {
@@ -624,7 +691,8 @@ struct Fuse {
     const float* norm_gain = nullptr;   // RMS norm of the input rows in front of the product (gvec: one gain per coordinate)
     int gvec = 0;
     float eps = 0.f;
-    int glu_ff = 0, glu_act = 0;        // act(gate) * up behind a fused [gate | up] product: N is then the inner size
+    GluCols glu{};                      // act(gate) * up behind a fused [gate | up] product (N then counts the plain columns in front of it
+                                        // and the gates; out null: the product's own output)
     ExpertSkip nskip{}, kskip{};        // few rows over stacked expert matrices: column tiles / k chunks of experts no row chose are not read
 };
 bool few_rows(int M, int K) { return M <= kRowGemvMaxRows && (size_t)M * K * sizeof(float) <= g_smem_optin; }
@@ -639,7 +707,7 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
     // bf16 weights with K in whole 32-element chunks: the tensor-core form (a weight byte costs the same for 1 and for 8 rows; rows staged as bf16)
     const bool mma_ok = M <= kRowGemvMaxRows && m.d.mode == TI_SEQ_BF16 && g_use_row_mma && K % 32 == 0 && K >= 256 && (reinterpret_cast<uintptr_t>(W) & 15) == 0 &&
                         mma_bytes <= g_smem_optin;
-    const bool plain = !fuse || (!fuse->norm_gain && !fuse->glu_ff);   // (a request to skip unused experts' rows is only a permission)
+    const bool plain = !fuse || (!fuse->norm_gain && !fuse->glu.ff);   // (a request to skip unused experts' rows is only a permission)
     if (plain && M > 1 && M <= kRowGemvMaxRows && !mma_ok && !few_rows(M, K) && few_rows(1, K)) {
         const int half = M / 2;
         TRY(gemm(m, A, lda, W, C, ldc, half, N, K, epi, alpha, fuse, beta));
@@ -651,10 +719,11 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
         // beside the weight bytes: 2 blocks an SM (their registers allow no more) as far as their shared memory allows, columns looped inside
         const int per_sm = (int)std::max<size_t>(1, std::min<size_t>(2, (200u << 10) / std::max<size_t>(xs_bytes, 1)));
         const int grid = std::max(1, std::min((N + warps - 1) / warps, g_num_sms * per_sm));
-        const Fuse f = fuse ? *fuse : Fuse{};
+        Fuse f = fuse ? *fuse : Fuse{};
+        if (f.glu.ff > 0 && !f.glu.out) { f.glu.out = C; f.glu.ld = ldc; }
         if (mma_ok) {
             const int fit = (int)std::max<size_t>(1, std::min<size_t>(2, (200u << 10) / mma_bytes));
-            const int blocks = std::max(1, std::min((N + kMmaCols - 1) / kMmaCols, g_num_sms * fit));
+            const int blocks = std::max(1, std::min((N + kMmaCols - 1) / kMmaCols + (f.glu.ff > 0 && f.glu.first > 0 ? 1 : 0), g_num_sms * fit));
             cudaLaunchConfig_t cfg{};
             cfg.gridDim = dim3(blocks);
             cfg.blockDim = dim3(256);
@@ -665,12 +734,12 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
             attr[0].val.programmaticStreamSerializationAllowed = 1;
             cfg.attrs = attr;
             cfg.numAttrs = g_use_pdl ? 1 : 0;
-            if (f.glu_ff > 0)
-                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<true>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu_ff,
-                                      f.glu_act, f.gvec, f.nskip, f.kskip));
+            if (f.glu.ff > 0)
+                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<true>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
+                                      f.gvec, f.nskip, f.kskip));
             else
-                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<false>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu_ff,
-                                      f.glu_act, f.gvec, f.nskip, f.kskip));
+                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<false>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
+                                      f.gvec, f.nskip, f.kskip));
             LAUNCHED();
             return 0;
         }
@@ -686,10 +755,10 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
         cfg.numAttrs = g_use_pdl ? 1 : 0;
         if (m.d.mode == TI_SEQ_BF16)
             CK(cudaLaunchKernelEx(&cfg, gemv_rows_kernel<__nv_bfloat16>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps,
-                                  f.glu_ff, f.glu_act, f.gvec));
+                                  f.glu, f.gvec));
         else
-            CK(cudaLaunchKernelEx(&cfg, gemv_rows_kernel<float>, A, lda, (const float*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu_ff,
-                                  f.glu_act, f.gvec));
+            CK(cudaLaunchKernelEx(&cfg, gemv_rows_kernel<float>, A, lda, (const float*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
+                                  f.gvec));
         LAUNCHED();
         return 0;
     }
@@ -956,8 +1025,9 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
     const bool front = m.d.norm_place == TI_SEQ_NORMS_FRONT;   // norms in front of the sublayers only: the residual lives in m.xs (one or more streams)
     float* emb_out = front ? m.xs.p : m.x.p;
     const int emb_copies = front ? m.n_streams : 1;
-    if (bf) TRY(launch_dep(embed_rows_kernel<__nv_bfloat16>, dim3(T), dim3(nt), 0, (const __nv_bfloat16*)m.embed, sm, D, emb_out, m.loop_in ? m.x0.p : nullptr, (const float*)m.pos_freq.p, emb_copies));
-    else TRY(launch_dep(embed_rows_kernel<float>, dim3(T), dim3(nt), 0, (const float*)m.embed, sm, D, emb_out, m.loop_in ? m.x0.p : nullptr, (const float*)m.pos_freq.p, emb_copies));
+    const float emb_scale = m.d.embed_scale > 0.f ? m.d.embed_scale : 1.f;
+    if (bf) TRY(launch_dep(embed_rows_kernel<__nv_bfloat16>, dim3(T), dim3(nt), 0, (const __nv_bfloat16*)m.embed, sm, D, emb_out, m.loop_in ? m.x0.p : nullptr, (const float*)m.pos_freq.p, emb_copies, emb_scale));
+    else TRY(launch_dep(embed_rows_kernel<float>, dim3(T), dim3(nt), 0, (const float*)m.embed, sm, D, emb_out, m.loop_in ? m.x0.p : nullptr, (const float*)m.pos_freq.p, emb_copies, emb_scale));
     LAUNCHED();
     const float eps = m.d.norm_eps;
     const int gv = m.gvec;
@@ -1016,20 +1086,33 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         return 0;
     };
     // the short convolution in front of a sublayer: y = x + conv(x) over the sequence's last inputs; the slot then keeps the newest ones
-    auto short_conv = [&](const float* in, const float* w, int taps, float* state, float* out) -> int {
+    auto conv = [&](const float* in, const ConvForm& cf, int D, const float* w, int taps, float* state, float* out) -> int {   // over D channels
         constexpr int kConvRows = 8;   // rows a block of the many-rows kernel takes
         const dim3 rows_grid((T + kConvRows - 1) / kConvRows, (D / 4 + 127) / 128);
-        if (T > 64 && D % 4 == 0 && taps <= 4) TRY(launch_dep(short_conv_rows_kernel<kConvRows, 4>, rows_grid, dim3(128), 0, in, sm, T, D, taps, w, state, out));
-        else if (T > 64 && D % 4 == 0 && taps <= 8) TRY(launch_dep(short_conv_rows_kernel<kConvRows, 8>, rows_grid, dim3(128), 0, in, sm, T, D, taps, w, state, out));
-        else if (T > 64 && D % 4 == 0) TRY(launch_dep(short_conv_kernel<4>, dim3(T), dim3(std::min(nt, (D / 4 + 31) / 32 * 32)), 0, in, sm, D, taps, w, state, out));
-        else TRY(launch_dep(short_conv_kernel<1>, dim3(T, T <= 64 ? (D + nt - 1) / nt : 1), dim3(nt), 0, in, sm, D, taps, w, state, out));
+        const bool v4 = T > 64 && D % 4 == 0 && cf.ldx % 4 == 0 && (reinterpret_cast<uintptr_t>(in) & 15) == 0;
+        if (v4 && taps <= 4) TRY(launch_dep(short_conv_rows_kernel<kConvRows, 4>, rows_grid, dim3(128), 0, in, cf, sm, T, D, taps, w, state, out));
+        else if (v4 && taps <= 8) TRY(launch_dep(short_conv_rows_kernel<kConvRows, 8>, rows_grid, dim3(128), 0, in, cf, sm, T, D, taps, w, state, out));
+        else if (v4) TRY(launch_dep(short_conv_kernel<4>, dim3(T), dim3(std::min(nt, (D / 4 + 31) / 32 * 32)), 0, in, cf, sm, D, taps, w, state, out));
+        else TRY(launch_dep(short_conv_kernel<1>, dim3(T, T <= 64 ? (D + nt - 1) / nt : 1), dim3(nt), 0, in, cf, sm, D, taps, w, state, out));
         LAUNCHED();
         bool many = false;   // (an entry of one row has shifted its state in the kernel above)
         for (int e = 0; e < E; ++e) many = many || counts[e] > 1;
         if (taps > 1 && many) {
-            TRY(launch_dep(short_conv_save_kernel, dim3(E, (D + nt - 1) / nt), dim3(nt), 0, in, sm, D, taps, state));
+            TRY(launch_dep(short_conv_save_kernel, dim3(E, (D + nt - 1) / nt), dim3(nt), 0, in, cf.ldx, sm, D, taps, state));
             LAUNCHED();
         }
+        return 0;
+    };
+    auto short_conv = [&](const float* in, const float* w, int taps, float* state, float* out) -> int {
+        ConvForm cf{};
+        cf.ldx = D; cf.add_input = 1;
+        return conv(in, cf, D, w, taps, state, out);
+    };
+    auto glu = [&](const float* gu, int ld, int F, const LayerW& L, float* y, int ldy) -> int {   // act(gate) * up of all rows
+        const bool v4 = F % 4 == 0 && ld % 4 == 0 && ldy % 4 == 0 && (reinterpret_cast<uintptr_t>(gu) & 15) == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0;
+        if (v4) TRY(launch_dep(glu_kernel<4>, dim3(grid_for((size_t)T * F / 4)), dim3(256), 0, gu, ld, F, L.d.ff_act, L.d.ff_limit, y, ldy, T));
+        else TRY(launch_dep(glu_kernel<1>, dim3(grid_for((size_t)T * F)), dim3(256), 0, gu, ld, F, L.d.ff_act, L.d.ff_limit, y, ldy, T));
+        LAUNCHED();
         return 0;
     };
     if (front) TRY(hyper(0, -1));
@@ -1040,9 +1123,8 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         const bool v_in_k = kp == vp && s.kv_heads == 1 && s.v_ld == s.dim && s.vdim <= s.dim;
         const size_t tsmem = attn_tiled_smem_bytes(s.dim, s.vdim, v_in_k);
         const bool tiled_ok = g_use_tiled_attn && n_tiles > 0 && s.dim % 4 == 0 && s.vdim % 4 == 0 && s.vdim <= 512 && tsmem <= g_smem_optin && (s.v_ld % 4 == 0);
-        // bf16 mode, head sizes 64 / 128: the split-half tensor-core kernel (fp32-accurate); fp32 mode keeps true fp32 arithmetic
-        const bool h3_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles128 > 0 && s.dim == s.vdim && (s.dim == 64 || s.dim == 128) &&
-                           (s.kv_heads * s.dim) % 4 == 0 && s.v_ld == 0;
+        // bf16 mode, head sizes up to 128 in fours: the split-half tensor-core kernel (fp32-accurate); fp32 mode keeps true fp32 arithmetic
+        const bool h3_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles128 > 0 && s.dim <= 128 && s.vdim <= 128 && s.dim % 4 == 0 && s.vdim % 4 == 0 && s.v_ld == 0;
         // bf16 mode, a shared key/value head with the values inside the key rows (latent attention), instantiated sizes: tensor cores
         const bool lat_size = (s.dim == 320 && s.vdim == 256) || (s.dim == 192 && s.vdim == 128) || (s.dim == 160 && s.vdim == 128);
         const bool lat_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles > 0 && v_in_k && (!s.out_gate || s.gate) && !s.qk_norm && lat_size;
@@ -1056,8 +1138,14 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             LAUNCHED();
         } else if (h3_ok) {
             const dim3 grid(n_tiles128, s.heads);
-            if (s.dim == 64) window_attention_h3_kernel<64><<<grid, kTcThreads, attn_h3_smem_bytes<64>(), g_stream>>>(q, sm, s, d_tiles128, kp, vp, out);
-            else window_attention_h3_kernel<128><<<grid, kTcThreads, attn_h3_smem_bytes<128>(), g_stream>>>(q, sm, s, d_tiles128, kp, vp, out);
+            const int dk = s.dim <= 64 ? 64 : 128, dv = s.vdim <= 64 ? 64 : 128;
+            const bool sized = dk == s.dim && dv == s.vdim;
+#define TI_H3_CASE(K, V, X) window_attention_h3_kernel<K, V, X><<<grid, kTcThreads, window_h3_smem_bytes<K, V>(), g_stream>>>(q, sm, s, d_tiles128, kp, vp, out)
+            if (dk == 64 && dv == 64) { if (sized) TI_H3_CASE(64, 64, true); else TI_H3_CASE(64, 64, false); }
+            else if (dk == 128 && dv == 128) { if (sized) TI_H3_CASE(128, 128, true); else TI_H3_CASE(128, 128, false); }
+            else if (dk == 64) TI_H3_CASE(64, 128, false);
+            else TI_H3_CASE(128, 64, false);
+#undef TI_H3_CASE
             LAUNCHED();
         } else if (tiled_ok) {
             const dim3 grid(n_tiles, s.heads);
@@ -1152,9 +1240,144 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         }
         return 0;
     };
+    // a gated linear recurrence over the step's rows
+    auto linear_scan = [&](const LinScanArgs& a, int layer) -> int {
+        const int H = a.heads, dk = a.dk, dv = a.dv;
+        const int threads = std::min(128, (dv + 31) / 32 * 32);
+        const dim3 grid(E, H, (dv + threads - 1) / threads);
+        const int zg = (dv + 31) / 32;
+        if (dk == 32) TRY(launch_dep(linear_scan_split_kernel<32, 8, 4>, dim3(E, H, zg), dim3(128), 0, a, sm));
+        else if (dk == 64) TRY(launch_dep(linear_scan_split_kernel<64, 8, 8>, dim3(E, H, zg), dim3(256), 0, a, sm));
+        else if (dk == 128) TRY(launch_dep(linear_scan_split_kernel<128, 4, 16>, dim3(E, H, zg), dim3(512), 0, a, sm));
+        else if (dk <= 32) TRY(launch_dep(linear_scan_kernel<32>, grid, dim3(threads), linear_scan_smem_bytes(dk, threads, false), a, sm));
+        else if (dk <= 64) TRY(launch_dep(linear_scan_kernel<64>, grid, dim3(threads), linear_scan_smem_bytes(dk, threads, false), a, sm));
+        else if (dk <= 128) TRY(launch_dep(linear_scan_kernel<128>, grid, dim3(threads), linear_scan_smem_bytes(dk, threads, false), a, sm));
+        else {
+            const int th = linear_scan_smem_bytes(dk, threads, true) <= g_smem_optin ? threads : 32;
+            const dim3 g2(E, H, (dv + th - 1) / th);
+            if (linear_scan_smem_bytes(dk, th, true) > g_smem_optin) return fail("layer %d: %d key channels do not fit the recurrence kernel", layer, dk);
+            TRY(launch_dep(linear_scan_kernel<0>, g2, dim3(th), linear_scan_smem_bytes(dk, th, true), a, sm));
+        }
+        LAUNCHED();
+        return 0;
+    };
+    auto route_shape = [&](const ti_seq_layer_desc& d) {
+        RouteShape r{};
+        r.n_real = d.experts; r.n_id = d.identity; r.top = d.top; r.groups = d.groups; r.keep = d.groups_keep;
+        r.kind = d.route_kind == TI_SEQ_ROUTE_TOP_LOGITS ? ROUTE_LOGITS : d.route_kind == TI_SEQ_ROUTE_SIGMOID ? ROUTE_SIGMOID : ROUTE_SOFTMAX;
+        r.scale = d.route_scale > 0.f ? d.route_scale : 1.f;
+        return r;
+    };
+    auto route_row_bytes = [&](const ti_seq_layer_desc& d) { return (size_t)(2 * (d.experts + d.identity) + 2 * d.groups) * sizeof(float); };
+    // weights of all rows from the router's columns of m.proj; used != null: one block over all (few) rows, which also marks the chosen experts
+    auto route = [&](const RouteShape& r, size_t row_bytes, int ld, const LayerW& L, float* wdense, float* idw, int* used) -> int {
+        const float* vec = r.kind == ROUTE_LOGITS ? L.route_bias : L.correction;
+        const int rw = used ? T : 4;
+        TRY(launch_dep(moe_route_kernel, dim3(used ? 1 : (T + rw - 1) / rw), dim3(rw * 32), rw * row_bytes, (const float*)m.proj.p, ld, L.off_router, r, vec, T, wdense, idw, used));
+        LAUNCHED();
+        return 0;
+    };
+    // one norm for both sublayers: x <- x + mixer(norm(x)) + ff(norm(x)).  ONE product in front (all mixers' and the feed-forward's input
+    // matrices stacked; few rows: the norm in its prologue, the dense feed-forward's gating in its epilogue), the mixers and the
+    // feed-forward each write their part of the rows of ONE product behind (output matrices side by side along K, residual sum in its epilogue)
+    auto shared_norm_layer = [&](size_t ri) -> int {
+        Run& R = m.runs[ri];
+        LayerW& L = m.layers[R.layer];
+        const ti_seq_layer_desc& d = L.d;
+        const int nf = L.ld_front, KB = L.n_back, F = d.ff;
+        const bool few = few_rows(T, D);
+        Fuse fn;
+        const float* in = m.x.p;
+        if (few) { fn.norm_gain = L.norm1; fn.eps = eps; fn.gvec = gv; }
+        else {
+            TRY(launch_dep(rmsnorm_kernel, dim3(T), dim3(nt), 0, (const float*)m.x.p, D, (const int*)nullptr, D, L.norm1, gv, eps, m.h.p));
+            LAUNCHED();
+            in = m.h.p;
+        }
+        float* ffo = m.act.p + L.back_ff;   // the feed-forward's part of the back product's rows
+        const bool gated = F > 0 && d.ff_kind == TI_SEQ_FF_GLU, routed = F > 0 && d.ff_kind == TI_SEQ_FF_EXPERTS;
+        const RouteShape rs = routed ? route_shape(d) : RouteShape{};
+        const size_t rper = routed ? route_row_bytes(d) : 0;
+        const bool sparse = routed && few && bf && d.experts > 0 && T * rper <= 40 * 1024;   // the router first, then only the chosen experts' rows
+        if (few && gated) {
+            Fuse f = fn;
+            f.glu = GluCols{F, d.ff_act, L.off_up, d.ff_limit, ffo, KB};
+            TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, L.off_up + F, D, EPI_NONE, 1.f, &f));
+        } else {
+            TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, sparse ? L.off_up : L.n_front, D, EPI_NONE, 1.f, few ? &fn : nullptr));
+        }
+        if (d.mixer == TI_SEQ_MIXER_ATTENTION) {
+            AttnShape s{};
+            s.heads = d.heads; s.kv_heads = d.kv_heads; s.dim = d.dim; s.vdim = d.vdim; s.window = d.window; s.rot_dims = d.rot_dims; s.rot_half = d.rot_half;
+            s.qk_norm = d.qk_norm == TI_SEQ_QK_NORM_HEAD ? 1 : 0; s.qgain = L.qgain; s.kgain = L.kgain; s.rot_amp = d.rot_amp > 0.f ? d.rot_amp : 1.f;
+            s.scale = d.scale; s.eps = eps; s.ld = nf; s.sink = L.sink; s.softcap = d.softcap; s.v_norm = d.v_norm; s.bias = L.qkv_bias.p; s.temp = L.temp; s.pb = L.pb;
+            s.out_ld = KB; s.out_scale = has_ssm(d) ? d.left_scale : 1.f;
+            TRY(launch_dep(attn_prepare_kernel, dim3(T), dim3(128), 0, m.proj.p, sm, s, L.inv_freq.p, R.k_pool.p, R.v_pool.p));
+            LAUNCHED();
+            TRY(attention(s, m.proj.p, R.k_pool.p, R.v_pool.p, m.act.p));
+        } else if (d.mixer == TI_SEQ_MIXER_GLA) {
+            const int H = d.heads, C = H * d.dim;
+            TRY(gemm(m, m.proj.p + L.off_a1, nf, L.a2, m.aux.p, C, T, C, d.decay_rank));
+            LinScanArgs a{};
+            a.q = m.proj.p + L.off_q; a.ldq = nf; a.k = m.proj.p + L.off_k; a.ldk = nf; a.v = m.proj.p + L.off_v; a.ldv = nf;
+            a.a = m.aux.p; a.lda = C; a.qscale = 1.f / sqrtf((float)d.dim);
+            a.gates = LIN_GATES_GLA; a.bias = L.a2b; a.inv_tau = 1.f / d.decay_tau;
+            a.state = R.state.p; a.out = m.act.p; a.ldo = KB; a.heads = H; a.dk = d.dim; a.dv = d.vdim;
+            TRY(linear_scan(a, R.layer));
+            TRY(launch_dep(head_rmsnorm_gate_kernel, dim3((T * H + 7) / 8), dim3(256), 0, m.act.p, KB, (const float*)(m.proj.p + L.off_g), nf, 1, L.normw, 0, T, H, d.vdim, eps));
+            LAUNCHED();
+        }
+        if (has_ssm(d)) {
+            const int inner = d.ssm_heads * d.ssm_vdim, ch = ssm_channels(d);
+            const float* u = m.proj.p + L.off_in;   // [z | x | B | C | dt]
+            ConvForm cf{};
+            cf.ldx = nf; cf.bias = L.ssm_conv_b; cf.silu = 1;
+            TRY(conv(u + inner, cf, ch, L.ssm_conv, d.ssm_taps, R.ssm_conv.p, m.aux2.p));
+            SsmArgs a{};
+            a.xbc = m.aux2.p; a.ld = ch; a.dt = u + inner + ch; a.ld_dt = nf; a.dt_bias = L.dt_bias; a.A_log = L.A_log; a.state = R.ssm_state.p;
+            a.out = m.act.p + L.back_ssm; a.ldo = KB; a.heads = d.ssm_heads; a.N = d.ssm_state; a.dv = d.ssm_vdim; a.groups = d.ssm_groups;
+            const dim3 grid(E, a.heads, (a.dv + 31) / 32);
+            if (a.N <= 32) TRY(launch_dep(ssm_scan_kernel<4>, grid, dim3(256), 0, a, sm));
+            else if (a.N <= 64) TRY(launch_dep(ssm_scan_kernel<8>, grid, dim3(256), 0, a, sm));
+            else if (a.N <= 128) TRY(launch_dep(ssm_scan_kernel<16>, grid, dim3(256), 0, a, sm));
+            else if (a.N <= 256) TRY(launch_dep(ssm_scan_kernel<32>, grid, dim3(256), 0, a, sm));
+            else TRY(launch_dep(ssm_scan_kernel<64>, grid, dim3(256), 0, a, sm));
+            LAUNCHED();
+            SsmFinishArgs fa{};
+            fa.y = a.out; fa.ldy = KB; fa.x = m.aux2.p; fa.ldx = ch; fa.z = u; fa.ldz = nf; fa.D = L.ssm_D; fa.w = L.ssm_norm; fa.inner = inner; fa.dv = d.ssm_vdim;
+            fa.parts = d.ssm_parts; fa.eps = eps; fa.scale = d.mixer == TI_SEQ_MIXER_SSM ? 1.f : d.right_scale;
+            const int size = inner / d.ssm_parts;
+            TRY(launch_dep(ssm_finish_kernel, dim3(T, d.ssm_parts), dim3(std::min(nt, (size + 31) / 32 * 32)), 0, fa));
+            LAUNCHED();
+        }
+        Fuse fk;
+        if (gated && !few) TRY(glu(m.proj.p + L.off_up, nf, F, L, ffo, KB));
+        else if (routed) {
+            const int Ex = d.experts, W = (d.expert_form == TI_SEQ_EXPERT_RELU2 ? 1 : 2) * F;   // columns of an expert in the front product
+            float *wdense = m.route.p, *idw_buf = m.route.p + (size_t)T * std::max(Ex, 1);
+            int* used = sparse ? reinterpret_cast<int*>(idw_buf + T) : nullptr;
+            TRY(route(rs, rper, nf, L, wdense, idw_buf, used));
+            if (sparse) {
+                Fuse f = fn;
+                f.nskip = ExpertSkip{used, 0, W, Ex};
+                TRY(gemm(m, in, D, (const uint8_t*)L.front + (size_t)L.off_up * D * m.wsize, m.proj.p + L.off_up, nf, T, L.n_front - L.off_up, D, EPI_NONE, 1.f, &f));
+                fk.kskip = ExpertSkip{used, L.back_ff, F, Ex};
+            }
+            TRY(launch_dep(moe_act_kernel, dim3(grid_for((size_t)T * L.ff_width)), dim3(256), 0, (const float*)m.proj.p, nf, L.off_up, Ex, F, (const float*)wdense, L.off_sh,
+                           d.shared_ff, L.off_sg, ffo, KB, d.expert_form, T));
+            LAUNCHED();
+        }
+        return gemm(m, m.act.p, KB, L.back, m.x.p, D, T, D, KB, EPI_ADD, 1.f, &fk);
+    };
+    const bool shared_norm = m.d.norm_place == TI_SEQ_NORMS_SHARED;
     for (size_t ri = 0; ri < m.runs.size(); ++ri) {
         Run& R = m.runs[ri];
         LayerW& L = m.layers[R.layer];
+        if (shared_norm) {
+            TRY(shared_norm_layer(ri));
+            if (m.dbg) CK(cudaMemcpyAsync(m.dbg_buf.p + ri * (size_t)T * D, m.x.p, (size_t)T * D * sizeof(float), cudaMemcpyDeviceToDevice, g_stream));
+            continue;
+        }
         if (R.enters_pass) {
             TRY(launch_dep(concat_rows_kernel, dim3(T), dim3(nt), 0, m.x.p, m.x0.p, D, m.xc.p));
             LAUNCHED();
@@ -1193,7 +1416,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         if (attn) {
             AttnShape s{};
             s.heads = L.d.heads; s.kv_heads = L.d.kv_heads; s.dim = L.d.dim; s.vdim = L.d.vdim;
-            s.window = L.d.window; s.rot_dims = L.d.rot_dims; s.qk_norm = L.d.qk_norm; s.out_gate = L.d.out_gate;
+            s.window = L.d.window; s.rot_dims = L.d.rot_dims; s.qk_norm = L.d.qk_norm == TI_SEQ_QK_NORM_HEAD ? 1 : 0; s.out_gate = L.d.out_gate;
             s.scale = L.d.scale; s.eps = eps; s.ld = L.n_qkvg;
             if (fuse_rows) {
                 Fuse f;
@@ -1204,6 +1427,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             }
             s.sink = L.sink; s.softcap = L.d.softcap; s.keep_first = L.d.keep_first; s.talk = L.talk;
             s.rot_half = L.d.rot_half; s.v_norm = L.d.v_norm; s.bias = L.qkv_bias.p; s.temp = L.temp;
+            s.qgain = L.qgain; s.kgain = L.kgain; s.rot_amp = L.d.rot_amp > 0.f ? L.d.rot_amp : 1.f; s.pb = L.pb;
             if (L.d.qk_norm == TI_SEQ_QK_NORM_WHOLE) TRY(launch_dep(attn_prepare_whole_kernel, dim3(T), dim3(256), 0, m.proj.p, sm, s, L.qnorm, L.knorm, R.k_pool.p, R.v_pool.p));
             else TRY(launch_dep(attn_prepare_kernel, dim3(T), dim3(128), 0, m.proj.p, sm, s, L.inv_freq.p, R.k_pool.p, R.v_pool.p));
             LAUNCHED();
@@ -1244,7 +1468,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
                 TRY(launch_dep(wkv_scan_kernel, dim3(grid), dim3((d + 31) / 32 * 32), a.s_in_smem ? full : small, a, sm));
             }
             LAUNCHED();
-            TRY(launch_dep(head_rmsnorm_gate_kernel, dim3((T * L.d.heads + 7) / 8), dim3(256), 0, m.att.p, (const float*)pg, C, 0, L.normw, 1, T, L.d.heads, d, eps));
+            TRY(launch_dep(head_rmsnorm_gate_kernel, dim3((T * L.d.heads + 7) / 8), dim3(256), 0, m.att.p, C, (const float*)pg, C, 0, L.normw, 1, T, L.d.heads, d, eps));
             LAUNCHED();
             TRY(gemm(m, m.att.p, C, L.o, m.mo.p, D, T, D, C));
         } else if (mixer == TI_SEQ_MIXER_GLA || mixer == TI_SEQ_MIXER_HGRN2) {
@@ -1266,24 +1490,9 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
                 a.qscale = 1.f;
                 a.gates = LIN_GATES_HGRN2; a.bias = L.fb; a.lower = L.lower; a.inv_tau = 1.f;
             }
-            a.state = R.state.p; a.out = m.att.p; a.heads = H; a.dk = dk; a.dv = dv;
-            const int threads = std::min(128, (dv + 31) / 32 * 32);
-            const dim3 grid(E, H, (dv + threads - 1) / threads);
-            const int zg = (dv + 31) / 32;
-            if (dk == 32) TRY(launch_dep(linear_scan_split_kernel<32, 8, 4>, dim3(E, H, zg), dim3(128), 0, a, sm));
-            else if (dk == 64) TRY(launch_dep(linear_scan_split_kernel<64, 8, 8>, dim3(E, H, zg), dim3(256), 0, a, sm));
-            else if (dk == 128) TRY(launch_dep(linear_scan_split_kernel<128, 4, 16>, dim3(E, H, zg), dim3(512), 0, a, sm));
-            else if (dk <= 32) TRY(launch_dep(linear_scan_kernel<32>, grid, dim3(threads), linear_scan_smem_bytes(dk, threads, false), a, sm));
-            else if (dk <= 64) TRY(launch_dep(linear_scan_kernel<64>, grid, dim3(threads), linear_scan_smem_bytes(dk, threads, false), a, sm));
-            else if (dk <= 128) TRY(launch_dep(linear_scan_kernel<128>, grid, dim3(threads), linear_scan_smem_bytes(dk, threads, false), a, sm));
-            else {
-                const int th = linear_scan_smem_bytes(dk, threads, true) <= g_smem_optin ? threads : 32;
-                const dim3 g2(E, H, (dv + th - 1) / th);
-                if (linear_scan_smem_bytes(dk, th, true) > g_smem_optin) return fail("layer %d: %d key channels do not fit the recurrence kernel", R.layer, dk);
-                TRY(launch_dep(linear_scan_kernel<0>, g2, dim3(th), linear_scan_smem_bytes(dk, th, true), a, sm));
-            }
-            LAUNCHED();
-            TRY(launch_dep(head_rmsnorm_gate_kernel, dim3((T * H + 7) / 8), dim3(256), 0, m.att.p, gla ? (const float*)(m.proj.p + L.off_g) : (const float*)nullptr, nf, 1,
+            a.state = R.state.p; a.out = m.att.p; a.ldo = Cv; a.heads = H; a.dk = dk; a.dv = dv;
+            TRY(linear_scan(a, R.layer));
+            TRY(launch_dep(head_rmsnorm_gate_kernel, dim3((T * H + 7) / 8), dim3(256), 0, m.att.p, Cv, gla ? (const float*)(m.proj.p + L.off_g) : (const float*)nullptr, nf, 1,
                            L.normw, 0, T, H, dv, eps));
             LAUNCHED();
             TRY(gemm(m, m.att.p, Cv, L.o, m.mo.p, D, T, D, Cv));
@@ -1348,16 +1557,15 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             } else if (L.d.ff_kind == TI_SEQ_FF_GLU) {
                 if (fuse_ff) {   // norm -> [gate | up] -> act(gate) * up in one launch
                     Fuse f;
-                    f.norm_gain = L.norm2; f.eps = eps; f.gvec = gv; f.glu_ff = F; f.glu_act = L.d.ff_act;
+                    f.norm_gain = L.norm2; f.eps = eps; f.gvec = gv; f.glu.ff = F; f.glu.act = L.d.ff_act; f.glu.limit = L.d.ff_limit;
                     TRY(gemm(m, m.x.p, D, L.gateup, m.act.p, F, T, F, D, EPI_NONE, 1.f, &f));
                 } else if (few_rows(T, D)) {   // [gate | up] -> act(gate) * up in one launch
                     Fuse f;
-                    f.glu_ff = F; f.glu_act = L.d.ff_act;
+                    f.glu.ff = F; f.glu.act = L.d.ff_act; f.glu.limit = L.d.ff_limit;
                     TRY(gemm(m, ff_in, D, L.gateup, m.act.p, F, T, F, D, EPI_NONE, 1.f, &f));
                 } else {
                     TRY(gemm(m, ff_in, D, L.gateup, m.proj.p, 2 * F, T, 2 * F, D));
-                    glu_kernel<<<grid_for((size_t)T * F), 256, 0, g_stream>>>(m.proj.p, F, L.d.ff_act, m.act.p, (size_t)T * F);
-                    LAUNCHED();
+                    TRY(glu(m.proj.p, 2 * F, F, L, m.act.p, F));
                 }
             } else if (L.d.ff_kind == TI_SEQ_FF_POLYNORM) {
                 TRY(gemm(m, m.h.p, D, L.ffront, m.proj.p, L.n_ffront, T, L.n_ffront, D));
@@ -1365,33 +1573,26 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
                 LAUNCHED();
             } else {
                 const int nfw = L.n_ffront, Ex = L.d.experts;
-                RouteShape r{};
-                r.n_real = Ex; r.n_id = L.d.identity; r.top = L.d.top; r.groups = L.d.groups; r.keep = L.d.groups_keep;
-                r.by_logits = L.d.route_kind == TI_SEQ_ROUTE_TOP_LOGITS ? 1 : 0;
-                const float* route_vec = r.by_logits ? L.route_bias : L.correction;
+                const RouteShape r = route_shape(L.d);
                 float* wdense = m.route.p;
                 float* idw_buf = m.route.p + (size_t)T * std::max(Ex, 1);
-                const size_t rper = (size_t)(2 * (Ex + L.d.identity) + 2 * L.d.groups) * sizeof(float);
+                const size_t rper = route_row_bytes(L.d);
                 // few rows: [router | shared scale | residual gate] first, then the experts' rows with the ones nobody chose left out
                 const bool sparse = few_rows(T, D) && bf && Ex > 0 && L.off_up > 0 && T * rper <= 40 * 1024;
                 if (sparse) {
                     int* used = reinterpret_cast<int*>(idw_buf + T);
                     TRY(gemm(m, ff_in, D, L.ffront, m.proj.p, nfw, T, L.off_up, D));
-                    TRY(launch_dep(moe_route_kernel, dim3(1), dim3(T * 32), T * rper, (const float*)m.proj.p, nfw, L.off_router, r, route_vec, T, wdense, idw_buf, used));
-                    LAUNCHED();
+                    TRY(route(r, rper, nfw, L, wdense, idw_buf, used));
                     Fuse f;
-                    f.nskip = ExpertSkip{used, 0, 2 * F, Ex};
+                    f.nskip = ExpertSkip{used, 0, (L.d.expert_form == TI_SEQ_EXPERT_RELU2 ? 1 : 2) * F, Ex};
                     TRY(gemm(m, ff_in, D, (const uint8_t*)L.ffront + (size_t)L.off_up * D * m.wsize, m.proj.p + L.off_up, nfw, T, nfw - L.off_up, D, EPI_NONE, 1.f, &f));
                 } else {
                     TRY(gemm(m, ff_in, D, L.ffront, m.proj.p, nfw, T, nfw, D));
-                    const int rw = 4;
-                    TRY(launch_dep(moe_route_kernel, dim3((T + rw - 1) / rw), dim3(rw * 32), rw * rper, (const float*)m.proj.p, nfw, L.off_router, r, route_vec, T, wdense, idw_buf,
-                                   (int*)nullptr));
-                    LAUNCHED();
+                    TRY(route(r, rper, nfw, L, wdense, idw_buf, nullptr));
                 }
                 if (L.ff_width > 0) {
                     TRY(launch_dep(moe_act_kernel, dim3(grid_for((size_t)T * L.ff_width)), dim3(256), 0, (const float*)m.proj.p, nfw, L.off_up, Ex, F, (const float*)wdense, L.off_sh,
-                                   L.d.shared_ff, L.off_sg, m.act.p, T));
+                                   L.d.shared_ff, L.off_sg, m.act.p, L.ff_width, L.d.expert_form, T));
                     LAUNCHED();
                 }
                 if (sparse) {
@@ -1498,6 +1699,74 @@ int close_seq(Model& m, int32_t seq) {
     return 0;
 }
 
+// A layer whose sublayers share one norm: its front and back matrices (the order of the front's rows: first mixer, state space, router,
+// shared expert's scale, [gate | up] or the experts' stacked input matrices; of the back's columns: first mixer, state space, feed-forward).
+int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
+    const ti_seq_layer_desc& d = L.d;
+    auto T = [&](const std::string& nm) -> Tensor* {
+        auto it = m.tensors.find(nm);
+        return it == m.tensors.end() ? nullptr : &it->second;
+    };
+    auto F = [&](const std::string& nm) -> const float* { return reinterpret_cast<const float*>(T(nm)->data.p); };
+    std::vector<const Tensor*> fr, bk;
+    std::vector<int*> at;            // where the offset of every front part goes (null: nowhere)
+    std::vector<std::string> used;   // tensors that live on inside the two matrices
+    const auto add = [&](const std::string& nm, int* off) { fr.push_back(T(nm)); at.push_back(off); used.push_back(nm); };
+    const auto add_back = [&](const std::string& nm) { bk.push_back(T(nm)); used.push_back(nm); };
+    int width = 0;
+    const std::string pl = p + mix_prefix(d, false), pr = p + mix_prefix(d, true);
+    if (d.mixer != TI_SEQ_MIXER_SSM) {
+        add(pl + "q", &L.off_q); add(pl + "k", &L.off_k); add(pl + "v", &L.off_v);
+        if (d.mixer == TI_SEQ_MIXER_GLA) { add(pl + "g", &L.off_g); add(pl + "a1", &L.off_a1); }
+        add_back(pl + "o");
+        width += d.heads * d.vdim;
+    }
+    if (has_ssm(d)) {
+        add(pr + "in", &L.off_in);
+        add_back(pr + "o");
+        L.back_ssm = width;
+        width += d.ssm_heads * d.ssm_vdim;
+        L.ssm_conv = F(pr + "conv"); L.ssm_conv_b = F(pr + "conv.b"); L.dt_bias = F(pr + "dt_bias"); L.A_log = F(pr + "A_log"); L.ssm_D = F(pr + "D"); L.ssm_norm = F(pr + "norm");
+        m.max_aux2 = std::max(m.max_aux2, ssm_channels(d));
+    }
+    if (d.ff > 0) {
+        L.back_ff = width;
+        if (d.ff_kind == TI_SEQ_FF_GLU) {
+            add(p + "mlp.gate", &L.off_up); add(p + "mlp.up", nullptr);
+            add_back(p + "mlp.down");
+            L.ff_width = d.ff;
+        } else {
+            add(p + "mlp.router", &L.off_router);
+            if (d.shared_ff > 0 && !d.shared_plain) add(p + "mlp.shared.sg", &L.off_sg);
+            const auto expert = [&](const std::string& q, int* off) {
+                if (d.expert_form == TI_SEQ_EXPERT_GATED) { add(q + "gate", off); add(q + "up", nullptr); }
+                else add(q + "up", off);
+                add_back(q + "down");
+            };
+            for (int e = 0; e < d.experts; ++e) expert(p + "mlp.e" + std::to_string(e) + ".", e == 0 ? &L.off_up : nullptr);
+            if (d.shared_ff > 0) expert(p + "mlp.shared.", &L.off_sh);
+            L.ff_width = d.experts * d.ff + d.shared_ff;
+            if (d.route_kind == TI_SEQ_ROUTE_TOP_LOGITS) L.route_bias = F(p + "mlp.router.b");
+            else L.correction = F(p + "mlp.correction");
+            m.max_route = std::max(m.max_route, 2 * std::max(d.experts, 1) + 1);
+        }
+        width += L.ff_width;
+    }
+    std::vector<int> off;
+    TRY(concat_rows(m, fr, L.front_buf, &L.n_front, &off));
+    for (size_t k = 0; k < at.size(); ++k)
+        if (at[k]) *at[k] = off[k];
+    L.front = L.front_buf.p;
+    L.ld_front = (L.n_front + 3) / 4 * 4;   // (rows of the front product start on 16-byte boundaries)
+    TRY(concat_cols(m, bk, L.back_buf, &L.n_back));
+    if (L.n_back != width) return fail("internal: output matrices of %d columns, %d expected", L.n_back, width);
+    L.back = L.back_buf.p;
+    for (const auto& nm : used) T(nm)->data.release();
+    m.max_proj = std::max(m.max_proj, L.ld_front);
+    m.max_ff = std::max(m.max_ff, L.n_back);
+    return 0;
+}
+
 }  // namespace
 
 extern "C" {
@@ -1527,8 +1796,14 @@ int ti_seq_init(int device) {
     if (const char* e = getenv("TURBOINFER_B200_SEQ_PDL")) g_use_pdl = atoi(e) != 0;
     if (const char* e = getenv("TURBOINFER_B200_SEQ_ROW_MMA")) g_use_row_mma = atoi(e) != 0;
     if (const char* e = getenv("TURBOINFER_B200_SEQ_TILED_ATTN")) g_use_tiled_attn = atoi(e) != 0;
-    CK(cudaFuncSetAttribute(window_attention_h3_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)attn_h3_smem_bytes<64>()));
-    CK(cudaFuncSetAttribute(window_attention_h3_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)attn_h3_smem_bytes<128>()));
+#define TI_H3_ATTR(K, V, X) CK(cudaFuncSetAttribute(window_attention_h3_kernel<K, V, X>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)window_h3_smem_bytes<K, V>()))
+    TI_H3_ATTR(64, 64, true);
+    TI_H3_ATTR(64, 64, false);
+    TI_H3_ATTR(128, 128, true);
+    TI_H3_ATTR(128, 128, false);
+    TI_H3_ATTR(64, 128, false);
+    TI_H3_ATTR(128, 64, false);
+#undef TI_H3_ATTR
     CK(cudaFuncSetAttribute(window_attention_tiled_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(window_attention_tiled_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(window_attention_tiled_kernel<4>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
@@ -1572,7 +1847,7 @@ int ti_seq_model_new(const ti_seq_model_desc* desc, const ti_seq_layer_desc* lay
     // the order of layer runs
     auto add_run = [&](int layer, bool enters) {
         m->runs.emplace_back();
-        m->runs.back().layer = layer;
+        m->runs.back().layer = layers[layer].weights_of ? layers[layer].weights_of - 1 : layer;   // (a run on shared tensors has a cache and state of its own)
         m->runs.back().enters_pass = enters;
     };
     if (desc->loop_times > 0) {
@@ -1694,7 +1969,7 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
     if (m.d.side_dim > 0) m.side_embed = P("side.embed");
     if (m.d.loop_times > 0 && !m.d.loop_plain) m.loop_in = P("loop.in");
     m.gvec = m.d.norm_kind != TI_SEQ_NORM_SCALAR ? 1 : 0;
-    const bool front = m.d.norm_place == TI_SEQ_NORMS_FRONT;
+    const bool front = m.d.norm_place == TI_SEQ_NORMS_FRONT, shared = m.d.norm_place == TI_SEQ_NORMS_SHARED;
     if (front) {   // one stream with in = mix = out = 1 is the plain residual x <- x + y
         m.n_streams = std::max(1, m.d.streams);
         const float one[1] = {1.f};
@@ -1734,9 +2009,10 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
     };
     for (int i = 0; i < m.d.n_layers; ++i) {
         LayerW& L = m.layers[i];
+        if (L.d.weights_of) continue;
         const std::string p = "l" + std::to_string(i) + ".";
         if (behind) L.norm1b = F(p + "norm1");   // the only norm of the sublayer sits behind it
-        else if (front) L.norm1 = F(p + "norm1");
+        else if (front || shared) L.norm1 = F(p + "norm1");
         else { L.norm1 = F(p + "norm1"); L.norm1b = F(p + "norm1b"); }
         if (L.d.conv_taps >= 1) { L.canon = F(p + "canon1"); m.any_conv = true; }
         if (L.d.conv_ff && L.d.ff > 0) L.canon2 = F(p + "canon2");
@@ -1754,10 +2030,15 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
         }
         bool rg1_fused = false, rg2_fused = false;
         if (L.d.mixer == TI_SEQ_MIXER_ATTENTION) {
-            TRY(concat_rows(m, {T(p + "mix.q"), T(p + "mix.k"), T(p + "mix.v"), L.d.out_gate ? T(p + "mix.g") : nullptr}, L.qkvg_buf, &L.n_qkvg));
-            L.qkvg = L.qkvg_buf.p;
-            for (const char* s : {"mix.q", "mix.k", "mix.v", "mix.g"}) release(p + s);
-            L.o = P(p + "mix.o");
+            const std::string px = p + mix_prefix(L.d, false);
+            if (!shared) {
+                TRY(concat_rows(m, {T(p + "mix.q"), T(p + "mix.k"), T(p + "mix.v"), L.d.out_gate ? T(p + "mix.g") : nullptr}, L.qkvg_buf, &L.n_qkvg));
+                L.qkvg = L.qkvg_buf.p;
+                for (const char* s : {"mix.q", "mix.k", "mix.v", "mix.g"}) release(p + s);
+                L.o = P(p + "mix.o");
+            }
+            if (L.d.qk_norm == TI_SEQ_QK_NORM_HEAD_GAIN) { L.qgain = F(px + "q.norm"); L.kgain = F(px + "k.norm"); }
+            if (L.d.weights_kind == TI_SEQ_WEIGHTS_SIGMOID) L.pb = F(px + "pb");
             const std::vector<float> f = rotary_frequencies(L.d);
             TRY(L.inv_freq.alloc(std::max<size_t>(1, f.size())));
             if (!f.empty()) CK(cudaMemcpy(L.inv_freq.p, f.data(), f.size() * sizeof(float), cudaMemcpyHostToDevice));
@@ -1771,12 +2052,12 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             if (L.d.proj_bias) {   // the three biases side by side, as the fused product lays its columns out
                 const size_t nq = (size_t)L.d.heads * L.d.dim, nk = (size_t)L.d.kv_heads * L.d.dim, nv = (size_t)L.d.kv_heads * L.d.vdim;
                 TRY(L.qkv_bias.alloc(nq + nk + nv));
-                CK(cudaMemcpy(L.qkv_bias.p, F(p + "mix.q.b"), nq * sizeof(float), cudaMemcpyDeviceToDevice));
-                CK(cudaMemcpy(L.qkv_bias.p + nq, F(p + "mix.k.b"), nk * sizeof(float), cudaMemcpyDeviceToDevice));
-                CK(cudaMemcpy(L.qkv_bias.p + nq + nk, F(p + "mix.v.b"), nv * sizeof(float), cudaMemcpyDeviceToDevice));
-                L.o_bias = F(p + "mix.o.b");
+                CK(cudaMemcpy(L.qkv_bias.p, F(px + "q.b"), nq * sizeof(float), cudaMemcpyDeviceToDevice));
+                CK(cudaMemcpy(L.qkv_bias.p + nq, F(px + "k.b"), nk * sizeof(float), cudaMemcpyDeviceToDevice));
+                CK(cudaMemcpy(L.qkv_bias.p + nq + nk, F(px + "v.b"), nv * sizeof(float), cudaMemcpyDeviceToDevice));
+                if (L.d.proj_bias == TI_SEQ_BIAS_QKVO) L.o_bias = F(p + "mix.o.b");
             }
-            if (L.d.talk || L.d.softcap > 0.f || L.d.keep_first > 0) {
+            if (L.d.talk || L.d.keep_first > 0) {
                 const int H = L.d.heads, d4 = (L.d.dim + 3) / 4 * 4, dv4 = (L.d.vdim + 3) / 4 * 4;
                 L.mix_HP = H <= 8 ? 8 : H <= 16 ? 16 : H <= 32 ? 32 : 64;
                 (void)dv4;
@@ -1797,6 +2078,13 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             m.max_att = std::max(m.max_att, C);
             m.max_rank = std::max(m.max_rank, L.d.decay_rank);
             m.any_wkv = true;
+        } else if (shared && L.d.mixer == TI_SEQ_MIXER_GLA) {
+            L.a2 = P(p + "mix.a2");
+            L.a2b = F(p + "mix.a2.b");
+            L.normw = F(p + "mix.norm");
+            note_k(L.d.decay_rank);
+            m.max_aux = std::max(m.max_aux, L.d.heads * L.d.dim);
+        } else if (L.d.mixer == TI_SEQ_MIXER_SSM) {   // (below)
         } else if (L.d.mixer == TI_SEQ_MIXER_GLA || L.d.mixer == TI_SEQ_MIXER_HGRN2) {
             const bool gla = L.d.mixer == TI_SEQ_MIXER_GLA;
             const int C = L.d.heads * L.d.dim, Cv = L.d.heads * L.d.vdim;
@@ -1866,6 +2154,10 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             m.max_aux2 = std::max(m.max_aux2, H * L.d.kv_rank);
             m.max_heads_v = std::max(m.max_heads_v, H * (L.d.kv_rank + 2));
         }
+        if (shared) {
+            TRY(build_shared_norm_layer(m, L, p));
+            continue;
+        }
         if (L.d.res_gate) {
             L.rg1b = F(p + "rg1.b");
             if (!rg1_fused) { L.rg1 = P(p + "rg1"); m.any_rgbuf = true; }
@@ -1915,7 +2207,7 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
                 std::vector<const Tensor*> downs;
                 for (int e = 0; e < E; ++e) {
                     const std::string q = p + "mlp.e" + std::to_string(e) + ".";
-                    parts.push_back(T(q + "gate"));
+                    parts.push_back(T(q + "gate"));   // (null for experts without a gate)
                     parts.push_back(T(q + "up"));
                     downs.push_back(T(q + "down"));
                 }
@@ -1928,8 +2220,9 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
                 TRY(concat_rows(m, parts, L.ffront_buf, &L.n_ffront, &off));
                 L.ffront = L.ffront_buf.p;
                 L.off_router = off[0]; L.off_sg = off[1]; L.off_rg2 = off[2];
-                L.off_up = E > 0 ? off[3] : -1;
-                L.off_sh = L.d.shared_ff > 0 ? off[3 + 2 * E] : -1;
+                const int ft = L.d.expert_form == TI_SEQ_EXPERT_RELU2 ? 1 : 0;   // an expert's first tensor: its gate, or its up matrix
+                L.off_up = E > 0 ? off[3 + ft] : -1;
+                L.off_sh = L.d.shared_ff > 0 ? off[3 + 2 * E + ft] : -1;
                 rg2_fused = L.d.res_gate != 0;
                 L.ff_width = E * L.d.ff + L.d.shared_ff;
                 if (L.ff_width > 0) {
@@ -1977,6 +2270,7 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
                     if (m.runs[rj].layer == L.kv_from) R.kv_run = (int)rj;
                 if (R.kv_run < 0) return fail("finalize: layer %d reads the cache of layer %d, which has not run before it", R.layer, L.kv_from);
             }
+        } else if (L.mixer == TI_SEQ_MIXER_SSM) {   // (below)
         } else if (L.mixer == TI_SEQ_MIXER_WKV) {
             TRY(R.state.alloc((size_t)m.d.max_seqs * L.heads * L.dim * L.dim));
             TRY(R.prev.alloc((size_t)m.d.max_seqs * D));
@@ -1985,6 +2279,12 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
         } else {
             TRY(R.state.alloc((size_t)m.d.max_seqs * L.heads * L.dim * L.vdim));
             CK(cudaMemset(R.state.p, 0, R.state.n * sizeof(float)));
+        }
+        if (has_ssm(L)) {
+            TRY(R.ssm_state.alloc((size_t)m.d.max_seqs * L.ssm_heads * L.ssm_state * L.ssm_vdim));
+            CK(cudaMemset(R.ssm_state.p, 0, R.ssm_state.n * sizeof(float)));
+            TRY(R.ssm_conv.alloc(std::max<size_t>(1, (size_t)m.d.max_seqs * (L.ssm_taps - 1) * ssm_channels(L))));
+            CK(cudaMemset(R.ssm_conv.p, 0, R.ssm_conv.n * sizeof(float)));
         }
         if (L.conv_taps > 1) {
             TRY(R.conv_state.alloc((size_t)m.d.max_seqs * (L.conv_taps - 1) * D));
@@ -2203,7 +2503,7 @@ int ti_seq_model_bytes(ti_seq_model_t h, double* weight_bytes, double* kv_bytes_
             w += (2 * C * D + 2 * Cv * D) * ws;   // q, k or f, v, o
             if (L.mixer == TI_SEQ_MIXER_GLA) w += (Cv * D + (double)L.decay_rank * (D + C)) * ws;
             st += (double)L.heads * L.dim * L.vdim * 4;
-        } else {
+        } else if (L.mixer != TI_SEQ_MIXER_SSM) {
             const double H = L.heads;
             w += (H * (L.dim + L.vdim) * L.kv_rank + H * L.vdim * D + (L.out_gate ? H * D : 0.0)) * ws;
             w += (L.q_rank > 0 ? (double)L.q_rank * (D + H * (L.dim + L.rot_dims)) : H * (L.dim + L.rot_dims) * D) * ws;
@@ -2212,13 +2512,17 @@ int ti_seq_model_bytes(ti_seq_model_t h, double* weight_bytes, double* kv_bytes_
                 kv += (double)(L.kv_rank + L.rot_dims) * 4;
             }
         }
+        if (has_ssm(L)) {
+            w += ((double)ssm_in_rows(L) + (double)L.ssm_heads * L.ssm_vdim) * D * ws;
+            st += ((double)L.ssm_heads * L.ssm_state * L.ssm_vdim + (double)(L.ssm_taps - 1) * ssm_channels(L)) * 4;
+        }
         if (L.conv_taps > 1) st += (double)(L.conv_taps - 1) * D * 4 * (L.conv_ff && L.ff > 0 ? 2 : 1);
         if (L.res_gate) w += (L.ff > 0 ? 2.0 : 1.0) * D * D * ws;
         if (L.ff > 0) {
             // routed experts: the stacked products read every expert's weights whatever the tokens chose
             if (L.ff_kind == TI_SEQ_FF_GLU) w += 3.0 * L.ff * D * ws;
             else if (L.ff_kind == TI_SEQ_FF_POLYNORM || L.ff_kind == TI_SEQ_FF_DENSE) w += 2.0 * L.ff * D * ws;
-            else w += (3.0 * ((double)L.experts * L.ff + L.shared_ff) + L.experts + L.identity + (L.shared_ff > 0 && !L.shared_plain ? 1 : 0)) * D * ws;
+            else w += ((L.expert_form == TI_SEQ_EXPERT_RELU2 ? 2.0 : 3.0) * ((double)L.experts * L.ff + L.shared_ff) + L.experts + L.identity + (L.shared_ff > 0 && !L.shared_plain ? 1 : 0)) * D * ws;
         }
         if (m->d.side_dim > 0) w += 2.0 * m->d.side_dim * D * ws;
     }

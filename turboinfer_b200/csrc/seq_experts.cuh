@@ -40,9 +40,13 @@ struct RouteShape {
     int n_real, n_id;    // experts with weights, identity experts behind them (router outputs = n_real + n_id)
     int top;             // experts a token uses
     int groups, keep;    // equal groups of neighbouring router outputs; only the `keep` groups with the largest member can be chosen
-    int by_logits;       // 1: `correction` is a bias added to the logits, the `top` largest biased logits are chosen and the weights are
-                         // the softmax over the chosen ones (no groups)
+    int kind;            // ROUTE_SOFTMAX
+                         // ROUTE_LOGITS: `correction` is a bias added to the logits, the `top` largest biased logits are chosen and the
+                         //   weights are the softmax over the chosen ones (no groups)
+                         // ROUTE_SIGMOID: scores are sigmoids; a group is worth the sum of its two largest choice scores
+    float scale;         // factor on the weights
 };
+enum { ROUTE_SOFTMAX = 0, ROUTE_LOGITS = 1, ROUTE_SIGMOID = 2 };
 // One warp per row.  s = softmax(logits); choice = s + correction; the best `keep` groups by their largest choice score stay, the
 // `top` largest choice scores among them are picked (first index wins a tie); weights = s over the picked ones / (their sum + 1e-20).
 // wdense[t][e] = weight of real expert e or 0; idw[t] = sum of the weights of picked identity experts.
@@ -60,12 +64,19 @@ __global__ void moe_route_kernel(const float* proj, int ld, int off, RouteShape 
     float* gs = ch + n;
     float* kept = gs + r.groups;
     const float* z = proj + (size_t)t * ld + off;
+    if (r.kind == ROUTE_SIGMOID) {
+        for (int i = lane; i < n; i += 32) {
+            const float v = 1.f / (1.f + expf(-z[i]));
+            s[i] = v;
+            ch[i] = v + correction[i];
+        }
+    } else {
     float mx = -INFINITY;
-    for (int i = lane; i < n; i += 32) mx = fmaxf(mx, z[i] + (r.by_logits ? correction[i] : 0.f));
+    for (int i = lane; i < n; i += 32) mx = fmaxf(mx, z[i] + (r.kind == ROUTE_LOGITS ? correction[i] : 0.f));
     mx = warp_max(mx);
     float sum = 0.f;
     for (int i = lane; i < n; i += 32) {
-        const float e = expf(z[i] + (r.by_logits ? correction[i] : 0.f) - mx);
+        const float e = expf(z[i] + (r.kind == ROUTE_LOGITS ? correction[i] : 0.f) - mx);
         s[i] = e;
         sum += e;
     }
@@ -73,15 +84,19 @@ __global__ void moe_route_kernel(const float* proj, int ld, int off, RouteShape 
     for (int i = lane; i < n; i += 32) {
         // by logits: the choice is made among the biased logits, and exp(. - max) of a chosen one over the chosen ones' sum is the
         // softmax over the chosen logits (the largest logit is always among them, so nothing underflows that matters)
-        if (r.by_logits) { ch[i] = z[i] + correction[i]; s[i] = fmaxf(s[i], 1e-37f); }
+        if (r.kind == ROUTE_LOGITS) { ch[i] = z[i] + correction[i]; s[i] = fmaxf(s[i], 1e-37f); }
         else { s[i] = s[i] / sum; ch[i] = s[i] + correction[i]; }
+    }
     }
     __syncwarp();
     const int size = n / r.groups;
     for (int g = lane; g < r.groups; g += 32) {
-        float b = -INFINITY;
-        for (int i = g * size; i < (g + 1) * size; ++i) b = fmaxf(b, ch[i]);
-        gs[g] = b;
+        float b = -INFINITY, b2 = -INFINITY;   // the two largest
+        for (int i = g * size; i < (g + 1) * size; ++i) {
+            b2 = fmaxf(b2, fminf(b, ch[i]));
+            b = fmaxf(b, ch[i]);
+        }
+        gs[g] = r.kind == ROUTE_SIGMOID && size > 1 ? b + b2 : b;
         kept[g] = 0.f;
     }
     __syncwarp();
@@ -139,7 +154,7 @@ __global__ void moe_route_kernel(const float* proj, int ld, int off, RouteShape 
                 if (picked[k] != 0x7FFFFFFF) s[picked[k]] = -s[picked[k]];
         __syncwarp();
     }
-    const float inv = 1.f / (tot + 1e-20f);
+    const float inv = r.scale / (tot + 1e-20f);
     float wi = 0.f;
     for (int i = lane; i < n; i += 32)
         if (s[i] < 0.f) {
@@ -162,8 +177,10 @@ __global__ void moe_route_kernel(const float* proj, int ld, int off, RouteShape 
 
 // act[t][e * F + c] = wdense[t][e] * silu(gate_e[c]) * up_e[c] (0 without reading when the weight is 0), and behind the experts
 // act[t][E * F + c] = sigmoid(proj[t][off_sg]) * silu(gate_s[c]) * up_s[c] for the shared expert (Fs = 0: none).
-// Expert e's [gate | up] block starts at proj column off_gu + e * 2F, the shared expert's at off_sh.
-__global__ void moe_act_kernel(const float* proj, int ld, int off_gu, int E, int F, const float* wdense, int off_sh, int Fs, int off_sg, float* act, int T) {
+// Expert e's [gate | up] block starts at proj column off_gu + e * 2F, the shared expert's at off_sh.  form EXPERT_RELU2: an expert has no
+// gate, its inner value is max(up, 0)^2 and its block is F wide.  lda = row stride of act.
+enum { EXPERT_GATED = 0, EXPERT_RELU2 = 1 };
+__global__ void moe_act_kernel(const float* proj, int ld, int off_gu, int E, int F, const float* wdense, int off_sh, int Fs, int off_sg, float* act, int lda, int form, int T) {
     pdl_launch_dependents();
     pdl_wait_prior_grid();
     const int W = E * F + Fs;
@@ -176,17 +193,25 @@ __global__ void moe_act_kernel(const float* proj, int ld, int off_gu, int E, int
         if (x < E * F) {
             const int e = x / F, c = x % F;
             const float w = wdense[t * E + e];
-            if (w != 0.f) {
+            if (w != 0.f && form == EXPERT_RELU2) {
+                const float u = fmaxf(row[off_gu + (size_t)e * F + c], 0.f);
+                v = w * u * u;
+            } else if (w != 0.f) {
                 const float g = row[off_gu + (size_t)e * 2 * F + c], u = row[off_gu + (size_t)e * 2 * F + F + c];
                 v = w * (g / (1.f + expf(-g))) * u;
             }
         } else {
             const int c = x - E * F;
-            const float g = row[off_sh + c], u = row[off_sh + Fs + c];
-            v = (g / (1.f + expf(-g))) * u;
+            if (form == EXPERT_RELU2) {
+                const float u = fmaxf(row[off_sh + c], 0.f);
+                v = u * u;
+            } else {
+                const float g = row[off_sh + c], u = row[off_sh + Fs + c];
+                v = (g / (1.f + expf(-g))) * u;
+            }
             if (off_sg >= 0) v /= 1.f + expf(-row[off_sg]);
         }
-        act[i] = v;
+        act[t * lda + x] = v;
     }
 }
 

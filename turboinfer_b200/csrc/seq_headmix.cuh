@@ -23,6 +23,23 @@ namespace tib {
 namespace seq {
 
 // ---- short convolution ------------------------------------------------------------------------------------------------------------
+// What a depth-wise convolution over the last `taps` inputs of a sequence adds up to: y = act(start + sum_j w[d][j] x[pos - (taps - 1) + j])
+struct ConvForm {
+    int ldx;            // row stride of the inputs
+    int add_input;      // 1: start = the newest input itself (y = x + conv(x)); 0: start = bias[d]
+    const float* bias;  // [D]; read when add_input is 0
+    int silu;           // 1: act(v) = v sigmoid(v)
+};
+template <int V> __device__ __forceinline__ void conv_start(const ConvForm& f, int d, const float (&xv)[V], float (&acc)[V]) {
+#pragma unroll
+    for (int c = 0; c < V; ++c) acc[c] = f.add_input ? xv[c] : f.bias[d + c];
+}
+template <int V> __device__ __forceinline__ void conv_finish(const ConvForm& f, float (&acc)[V]) {
+    if (f.silu) {
+#pragma unroll
+        for (int c = 0; c < V; ++c) acc[c] = acc[c] / (1.f + expf(-acc[c]));
+    }
+}
 // state [slots][taps - 1][D]: the inputs at positions len - (taps - 1) .. len - 1 of the slot's sequence, oldest first.  Entries
 // for positions before 0 are never read (a slot that is used again needs no clearing).
 // An entry that brings ONE row (a decoded token) also shifts its slot's state here: the thread that read a coordinate's old entries
@@ -41,7 +58,7 @@ template <int V> __device__ __forceinline__ void conv_store(float* p, const floa
 }
 // V = 4: a thread takes four neighbouring coordinates with 16-byte loads and stores (D in whole fours); V = 1: one coordinate at a time.
 template <int V>
-__global__ void short_conv_kernel(const float* x, StepMeta m, int D, int taps, const float* w, float* state, float* y) {
+__global__ void short_conv_kernel(const float* x, ConvForm f, StepMeta m, int D, int taps, const float* w, float* state, float* y) {
     pdl_launch_dependents();
     pdl_wait_prior_grid();
     constexpr int CH = V == 4 ? 4 : 8;   // taps whose inputs are requested together
@@ -50,9 +67,8 @@ __global__ void short_conv_kernel(const float* x, StepMeta m, int D, int taps, c
     const bool alone = m.ent_row0[e + 1] - m.ent_row0[e] == 1;
     for (int d = (blockIdx.y * blockDim.x + threadIdx.x) * V; d < D; d += gridDim.y * blockDim.x * V) {
         float xv[V], acc[V];
-        conv_load<V>(x + (size_t)t * D + d, xv);
-#pragma unroll
-        for (int c = 0; c < V; ++c) acc[c] = xv[c];
+        conv_load<V>(x + (size_t)t * f.ldx + d, xv);
+        conv_start<V>(f, d, xv, acc);
         // the taps' inputs are requested together (CH at a time), then multiplied in ascending order of the tap
         for (int j0 = 0; j0 < taps; j0 += CH) {
             float v[CH][V], wv[CH][V];
@@ -61,7 +77,7 @@ __global__ void short_conv_kernel(const float* x, StepMeta m, int D, int taps, c
                 const int j = j0 + q, back = taps - 1 - j;
                 const bool in_step = i - back >= 0;
                 const bool ok = j < taps && (in_step || pos0 + i - back >= 0);
-                const float* src = in_step ? x + (size_t)(t - back) * D + d : st + (size_t)(taps - 1 + i - back) * D + d;
+                const float* src = in_step ? x + (size_t)(t - back) * f.ldx + d : st + (size_t)(taps - 1 + i - back) * D + d;
                 if (ok) conv_load<V>(src, v[q]);
 #pragma unroll
                 for (int c = 0; c < V; ++c) {
@@ -76,6 +92,7 @@ __global__ void short_conv_kernel(const float* x, StepMeta m, int D, int taps, c
                     for (int c = 0; c < V; ++c) acc[c] = fmaf(wv[q][c], v[q][c], acc[c]);
                 }
         }
+        conv_finish<V>(f, acc);
         conv_store<V>(y + (size_t)t * D + d, acc);
         if (alone) {
             for (int s = 0; s + 2 < taps; ++s) {
@@ -91,9 +108,9 @@ __global__ void short_conv_kernel(const float* x, StepMeta m, int D, int taps, c
 // weights (taps <= KT) it reads ONCE and keeps in registers, the tap that reaches `back` rows back in entry KT - 1 - back.
 // Rows that all lie in one entry, taps - 1 rows or more behind its first: their inputs and those of the taps - 1 rows in front are
 // requested together, each once (no state is read or shifted).  Other blocks (an entry's first rows, entries of few rows) go row by
-// row.  The arithmetic of a coordinate is that of short_conv_kernel either way: acc = x, then the taps from the oldest input on.
+// row.  The arithmetic of a coordinate is that of short_conv_kernel either way: the start, then the taps from the oldest input on.
 template <int R, int KT>
-__global__ void __launch_bounds__(128) short_conv_rows_kernel(const float* __restrict__ x, StepMeta m, int T, int D, int taps, const float* __restrict__ w, float* state, float* __restrict__ y) {
+__global__ void __launch_bounds__(128) short_conv_rows_kernel(const float* __restrict__ x, ConvForm f, StepMeta m, int T, int D, int taps, const float* __restrict__ w, float* state, float* __restrict__ y) {
     pdl_launch_dependents();
     pdl_wait_prior_grid();
     const int d = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
@@ -111,21 +128,21 @@ __global__ void __launch_bounds__(128) short_conv_rows_kernel(const float* __res
 #pragma unroll
         for (int r = 0; r < R + KT - 1; ++r) {
             const int t = t0 - (KT - 1) + r;
-            if (r >= skip && t < t1) conv_load<4>(x + (size_t)t * D + d, xs[r]);
+            if (r >= skip && t < t1) conv_load<4>(x + (size_t)t * f.ldx + d, xs[r]);
             else xs[r][0] = xs[r][1] = xs[r][2] = xs[r][3] = 0.f;
         }
 #pragma unroll
         for (int r = 0; r < R; ++r)
             if (t0 + r < t1) {
                 float acc[4];
-#pragma unroll
-                for (int c = 0; c < 4; ++c) acc[c] = xs[r + KT - 1][c];
+                conv_start<4>(f, d, xs[r + KT - 1], acc);
 #pragma unroll
                 for (int q = 0; q < KT; ++q)
                     if (q >= skip) {
 #pragma unroll
                         for (int c = 0; c < 4; ++c) acc[c] = fmaf(wv[q][c], xs[r + q][c], acc[c]);
                     }
+                conv_finish<4>(f, acc);
                 conv_store<4>(y + (size_t)(t0 + r) * D + d, acc);
             }
         return;
@@ -135,24 +152,24 @@ __global__ void __launch_bounds__(128) short_conv_rows_kernel(const float* __res
         float* st = state + (size_t)m.ent_slot[e] * (taps - 1) * D;
         const bool alone = m.ent_row0[e + 1] - m.ent_row0[e] == 1;
         float xv[4], acc[4], v[KT][4];
-        conv_load<4>(x + (size_t)t * D + d, xv);
+        conv_load<4>(x + (size_t)t * f.ldx + d, xv);
 #pragma unroll
         for (int q = 0; q < KT; ++q) {
             const int back = KT - 1 - q;
             const bool in_step = i - back >= 0;
             const bool ok = q >= skip && (in_step || pos0 + i - back >= 0);
-            const float* src = in_step ? x + (size_t)(t - back) * D + d : st + (size_t)(taps - 1 + i - back) * D + d;
+            const float* src = in_step ? x + (size_t)(t - back) * f.ldx + d : st + (size_t)(taps - 1 + i - back) * D + d;
             if (ok) conv_load<4>(src, v[q]);
             else v[q][0] = v[q][1] = v[q][2] = v[q][3] = 0.f;
         }
-#pragma unroll
-        for (int c = 0; c < 4; ++c) acc[c] = xv[c];
+        conv_start<4>(f, d, xv, acc);
 #pragma unroll
         for (int q = 0; q < KT; ++q)
             if (q >= skip) {
 #pragma unroll
                 for (int c = 0; c < 4; ++c) acc[c] = fmaf(wv[q][c], v[q][c], acc[c]);
             }
+        conv_finish<4>(f, acc);
         conv_store<4>(y + (size_t)t * D + d, acc);
         if (alone) {
             for (int s = 0; s + 2 < taps; ++s) {
@@ -165,7 +182,7 @@ __global__ void __launch_bounds__(128) short_conv_rows_kernel(const float* __res
     }
 }
 // after all rows of the step have read the old state: the slot keeps the last taps - 1 inputs of its sequence
-__global__ void short_conv_save_kernel(const float* x, StepMeta m, int D, int taps, float* state) {
+__global__ void short_conv_save_kernel(const float* x, int ldx, StepMeta m, int D, int taps, float* state) {
     pdl_launch_dependents();
     pdl_wait_prior_grid();
     const int e = blockIdx.x, row0 = m.ent_row0[e], n = m.ent_row0[e + 1] - row0;
@@ -174,7 +191,7 @@ __global__ void short_conv_save_kernel(const float* x, StepMeta m, int D, int ta
     for (int d = blockIdx.y * blockDim.x + threadIdx.x; d < D; d += gridDim.y * blockDim.x)
         for (int s = 0; s < taps - 1; ++s) {   // ascending: entry n + s is still the old one when it is read
             const int i = n - (taps - 1) + s;
-            st[(size_t)s * D + d] = i >= 0 ? x[(size_t)(row0 + i) * D + d] : st[(size_t)(n + s) * D + d];
+            st[(size_t)s * D + d] = i >= 0 ? x[(size_t)(row0 + i) * ldx + d] : st[(size_t)(n + s) * D + d];
         }
 }
 

@@ -53,16 +53,17 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 // ---- embedding -----------------------------------------------------------------------------------------------------
 // x[t] = embed[tok[t]] (+ the sinusoidal position vector: entry 2i = sin(pos * pos_freq[i]), entry 2i + 1 = cos of the same angle,
 // angle and functions in fp32); x0 (optional) keeps the embedding output for the looped block's input projection; copies > 1: the row
-// is written that many times in a row (x [T][copies][D]: the streams of hyper-connections all start from the embedding output)
+// is written that many times in a row (x [T][copies][D]: the streams of hyper-connections all start from the embedding output);
+// scale multiplies the table's row
 template <typename WT>
-__global__ void embed_rows_kernel(const WT* emb, StepMeta m, int D, float* x, float* x0, const float* pos_freq, int copies) {
+__global__ void embed_rows_kernel(const WT* emb, StepMeta m, int D, float* x, float* x0, const float* pos_freq, int copies, float scale) {
     pdl_launch_dependents();   // the kernel behind this one may be scheduled (and a few-row product may fetch its weights) ...
     pdl_wait_prior_grid();     // ... while this one waits here for the kernel before it, when it was launched ahead of its end
     const int t = blockIdx.x;
     const WT* e = emb + (size_t)m.tok[t] * D;
     const float pos = pos_freq ? (float)m.row_pos[t] : 0.f;
     for (int d = threadIdx.x; d < D; d += blockDim.x) {
-        float v = to_f32(e[d]);
+        float v = to_f32(e[d]) * scale;
         if (pos_freq) {
             const float ang = pos * pos_freq[d >> 1];
             v += (d & 1) ? cosf(ang) : sinf(ang);
@@ -155,7 +156,8 @@ __global__ void postnorm_residual_kernel(PostArgs a) {
 // ---- matrix products: C[M, N] = epi(A[M, K] . W[N, K]^T) ----------------------------------------------------------------
 enum {
     EPI_NONE = 0, EPI_TANH = 1, EPI_SCALE = 2, EPI_SILU = 3, EPI_SOFTCAP = 4 /* alpha * tanh(v / alpha) */, EPI_GELU_TANH = 5,
-    EPI_XIELU = 6 /* alpha v^2 + v / 2 for v > 0, beta (exp(v) - 1 - v) + v / 2 otherwise */, EPI_MAX0 = 7
+    EPI_XIELU = 6 /* alpha v^2 + v / 2 for v > 0, beta (exp(v) - 1 - v) + v / 2 otherwise */, EPI_MAX0 = 7,
+    EPI_ADD = 8 /* C += v: the product ends in the residual sum (every element of C has one writer) */
 };
 __device__ __forceinline__ float xielu(float v, float a_pos, float a_neg) {
     return v > 0.f ? fmaf(a_pos * v, v, 0.5f * v) : fmaf(a_neg, expm1f(v) - v, 0.5f * v);
@@ -169,6 +171,10 @@ __device__ __forceinline__ float epi_apply(float v, int epi, float alpha, float 
     if (epi == EPI_SOFTCAP) return alpha * tanhf(v / alpha);
     if (epi == EPI_GELU_TANH) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
     return v;
+}
+
+__device__ __forceinline__ void epi_put(float* c, float v, int epi, float alpha, float beta) {
+    *c = epi == EPI_ADD ? *c + v : epi_apply(v, epi, alpha, beta);
 }
 
 // true fp32: 64 x 64 tile, 16-deep k-steps, 256 threads with 4 x 4 outputs each
@@ -209,7 +215,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* A, int lda, 
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int gm = m0 + ty * 4 + i, gn = n0 + tx * 4 + j;
-            if (gm < M && gn < N) C[(size_t)gm * ldc + gn] = epi_apply(acc[i][j], epi, alpha, beta);
+            if (gm < M && gn < N) epi_put(C + (size_t)gm * ldc + gn, acc[i][j], epi, alpha, beta);
         }
 }
 
@@ -295,17 +301,25 @@ __global__ void __launch_bounds__(128) gemm_bf16_kernel(const float* A, int lda,
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int gm = m0 + wm + i * 16 + g + (e >> 1) * 8, gn = n0 + wn + j * 8 + 2 * t4 + (e & 1);
-                if (gm < M && gn < N) C[(size_t)gm * ldc + gn] = epi_apply(acc[i][j][e], epi, alpha, beta);
+                if (gm < M && gn < N) epi_put(C + (size_t)gm * ldc + gn, acc[i][j][e], epi, alpha, beta);
             }
 }
 
 // few rows (M <= 8, the decode step): the weights are streamed once with 16-byte loads, one warp per output column; the rows
 // sit in shared memory.  Fused in front: the scalar-gain RMS norm of the rows (norm_gain != null).  Fused behind: an activation
-// or scale, or the gated feed-forward's act(gate) * up over the row pair (n, n + glu_ff) of the fused [gate | up] matrix.
-// Bound by the weight bytes.
+// or scale, or the gated feed-forward's act(gate) * up over the row pair (n, n + glu_ff) of the fused [gate | up] matrix, which may sit
+// behind plain columns (GluCols).  Bound by the weight bytes.
 constexpr int kRowGemvMaxRows = 8;
 constexpr int kRowGemvThreads = 256;
-__device__ __forceinline__ float ff_act(float z, int act);
+__device__ __forceinline__ float glu_pair(float g, float u, int act, float limit);
+// Columns [0, first) of the product are plain and go to C; columns first .. N - 1 are gates whose partner column lies ff behind:
+// out[r * ld + n - first] = act(gate) * up.  ff = 0: every column is plain.
+struct GluCols {
+    int ff, act, first;
+    float limit;
+    float* out;
+    int ld;
+};
 // eight consecutive weights as they lie in memory (kept packed while the loads are in flight) and as fp32
 template <typename WT> struct Raw8;
 template <> struct Raw8<float> { float4 a, b; };
@@ -369,7 +383,7 @@ __device__ __forceinline__ void gemv_row_dot(const WT* w, const float* xs, int M
 // still running, and only then waits for that kernel's results (the rows).
 template <typename WT>
 __global__ void __launch_bounds__(kRowGemvThreads, 2) gemv_rows_kernel(const float* A, int lda, const WT* W, float* C, int ldc, int M, int N, int K, int epi,
-                                                                  float alpha, float beta, const float* norm_gain, float eps, int glu_ff, int glu_act, int gvec) {
+                                                                  float alpha, float beta, const float* norm_gain, float eps, GluCols glu, int gvec) {
     extern __shared__ __align__(16) float xs[];   // [M][K]
     __shared__ float rss[kRowGemvMaxRows][kRowGemvThreads / 32];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
@@ -380,8 +394,8 @@ __global__ void __launch_bounds__(kRowGemvThreads, 2) gemv_rows_kernel(const flo
         if (n < N) {
             const char* w = reinterpret_cast<const char*>(W + (size_t)n * K);
             for (size_t o = (size_t)lane * 128; o < row_bytes; o += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
-            if (glu_ff > 0) {
-                const char* w2 = reinterpret_cast<const char*>(W + (size_t)(n + glu_ff) * K);
+            if (glu.ff > 0 && n >= glu.first) {
+                const char* w2 = reinterpret_cast<const char*>(W + (size_t)(n + glu.ff) * K);
                 for (size_t o = (size_t)lane * 128; o < row_bytes; o += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w2 + o));
             }
         }
@@ -427,11 +441,15 @@ __global__ void __launch_bounds__(kRowGemvThreads, 2) gemv_rows_kernel(const flo
     float acc[kRowGemvMaxRows], acc2[kRowGemvMaxRows];
     for (int n = blockIdx.x * nw + warp; n < N; n += gridDim.x * nw) {
         gemv_row_dot<WT>(W + (size_t)n * K, xs, M, K, vec, lane, acc);
-        if (glu_ff > 0) gemv_row_dot<WT>(W + (size_t)(n + glu_ff) * K, xs, M, K, vec, lane, acc2);
+        const bool gated = glu.ff > 0 && n >= glu.first;
+        if (gated) gemv_row_dot<WT>(W + (size_t)(n + glu.ff) * K, xs, M, K, vec, lane, acc2);
         if (lane == 0) {
 #pragma unroll
             for (int r = 0; r < kRowGemvMaxRows; ++r)
-                if (r < M) C[(size_t)r * ldc + n] = glu_ff > 0 ? ff_act(acc[r], glu_act) * acc2[r] : epi_apply(acc[r], epi, alpha, beta);
+                if (r < M) {
+                    if (gated) glu.out[(size_t)r * glu.ld + n - glu.first] = glu_pair(acc[r], acc2[r], glu.act, glu.limit);
+                    else epi_put(C + (size_t)r * ldc + n, acc[r], epi, alpha, beta);
+                }
         }
     }
 }
@@ -491,7 +509,7 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint3
 }
 template <bool GLU>
 __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int lda, const __nv_bfloat16* W, float* C, int ldc, int M, int N, int K, int epi,
-                                                           float alpha, float beta, const float* norm_gain, float eps, int glu_ff, int glu_act, int gvec, ExpertSkip nskip,
+                                                           float alpha, float beta, const float* norm_gain, float eps, GluCols glu, int gvec, ExpertSkip nskip,
                                                            ExpertSkip kskip) {
     extern __shared__ __align__(16) unsigned char smraw[];
     const int Kp = K + 32;
@@ -500,14 +518,18 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
     __shared__ float rss[kRowGemvMaxRows][8];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const int NC = K / 32, c_begin = warp * NC / 8, c_end = (warp + 1) * NC / 8;   // this warp's 32-k chunks
+    // column tiles: the plain columns in sixteens, then (GLU) the gated ones
+    const int plain_cols = GLU ? glu.first : N, plain_tiles = (plain_cols + kMmaCols - 1) / kMmaCols;
+    const int tiles = plain_tiles + (GLU ? (N - plain_cols + kMmaCols - 1) / kMmaCols : 0);
     pdl_launch_dependents();
     {   // ask L2 for this warp's slice of the block's first 16 (32 with the gate's partner) weight rows
-        const int n = min((int)blockIdx.x * kMmaCols + (lane & 15), N - 1);
+        const bool gated = GLU && (int)blockIdx.x >= plain_tiles;
+        const int n = gated ? min(plain_cols + ((int)blockIdx.x - plain_tiles) * kMmaCols + (lane & 15), N - 1) : min((int)blockIdx.x * kMmaCols + (lane & 15), plain_cols - 1);
         const char* w = reinterpret_cast<const char*>(W + (size_t)n * K + (size_t)c_begin * 32);
         const size_t bytes = (size_t)(c_end - c_begin) * 64;
         for (size_t o = (size_t)(lane >> 4) * 128; o < bytes; o += 256) {
             asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
-            if (GLU) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o + (size_t)glu_ff * K * 2));
+            if (gated) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o + (size_t)glu.ff * K * 2));
         }
     }
     pdl_wait_prior_grid();
@@ -564,12 +586,14 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
     constexpr int UNR = GLU ? 4 : 8;   // chunks whose weight loads are in flight together (16-byte loads a lane: 2 or 4 a chunk)
     // when chunks may be skipped the warps take the chunks in turn (every warp gets its share of every expert) instead of one range each
     const int cstep = kskip.used ? 8 : 1, c0 = kskip.used ? warp : c_begin, c1 = kskip.used ? NC : c_end;
-    for (int n0 = blockIdx.x * kMmaCols; n0 < N; n0 += gridDim.x * kMmaCols) {
-        if (!expert_range_used(nskip, n0, min(n0 + kMmaCols, N) - 1)) continue;   // (uniform over the block)
+    for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x) {
+        const bool gated = GLU && tile >= plain_tiles;
+        const int n0 = gated ? plain_cols + (tile - plain_tiles) * kMmaCols : tile * kMmaCols, end = gated ? N : plain_cols;
+        if (!expert_range_used(nskip, n0, min(n0 + kMmaCols, end) - 1)) continue;   // (uniform over the block)
         float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
-        const __nv_bfloat16* w0 = W + (size_t)min(n0 + g, N - 1) * K + 8 * t;
-        const __nv_bfloat16* w1 = W + (size_t)min(n0 + g + 8, N - 1) * K + 8 * t;
-        const size_t up = (size_t)glu_ff * K;
+        const __nv_bfloat16* w0 = W + (size_t)min(n0 + g, end - 1) * K + 8 * t;
+        const __nv_bfloat16* w1 = W + (size_t)min(n0 + g + 8, end - 1) * K + 8 * t;
+        const size_t up = (size_t)glu.ff * K;
         const __nv_bfloat16* xr = xs + (size_t)g * Kp + 8 * t;
         for (int c = c0; c < c1; c += UNR * cstep) {
             uint4 ra[UNR], rb[UNR], ua[GLU ? UNR : 1], ub[GLU ? UNR : 1];
@@ -582,7 +606,7 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
                     const int k = cc * 32;
                     ra[q] = *reinterpret_cast<const uint4*>(w0 + k);
                     rb[q] = *reinterpret_cast<const uint4*>(w1 + k);
-                    if (GLU) {
+                    if (gated) {
                         ua[q] = *reinterpret_cast<const uint4*>(w0 + up + k);
                         ub[q] = *reinterpret_cast<const uint4*>(w1 + up + k);
                     }
@@ -595,7 +619,7 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
                     if (g < M) x = *reinterpret_cast<const uint4*>(xr + (c + q * cstep) * 32);
                     mma_bf16_16816(acc, ra[q].x, rb[q].x, ra[q].y, rb[q].y, x.x, x.y);
                     mma_bf16_16816(acc, ra[q].z, rb[q].z, ra[q].w, rb[q].w, x.z, x.w);
-                    if (GLU) {
+                    if (gated) {
                         mma_bf16_16816(acc2, ua[q].x, ub[q].x, ua[q].y, ub[q].y, x.x, x.y);
                         mma_bf16_16816(acc2, ua[q].z, ub[q].z, ua[q].w, ub[q].w, x.z, x.w);
                     }
@@ -616,7 +640,10 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
                 v += red[(w * 2 + 0) * 128 + src];
                 if (GLU) v2 += red[(w * 2 + 1) * 128 + src];
             }
-            if (r < M && n0 + j < N) C[(size_t)r * ldc + n0 + j] = GLU ? ff_act(v, glu_act) * v2 : epi_apply(v, epi, alpha, beta);
+            if (r < M && n0 + j < end) {
+                if (gated) glu.out[(size_t)r * glu.ld + n0 + j - plain_cols] = glu_pair(v, v2, glu.act, glu.limit);
+                else epi_put(C + (size_t)r * ldc + n0 + j, v, epi, alpha, beta);
+            }
         }
         __syncthreads();
     }
@@ -703,8 +730,8 @@ struct AttnShape {
     int v_ld;                         // token stride of the value pool; 0: kv_heads * vdim.  A cache whose values are the leading
                                       // coordinates of its key rows passes the key pool as the value pool and the key stride here.
     const float* sink;                // [heads] or null: the softmax denominator gains exp(sink[h]), a term without key or value
-    // read by the head-mixing kernel only (seq_headmix.cuh); the step sends a layer there when one of them is set
     float softcap;                    // > 0: score <- cap * tanh(score / cap) after scaling
+    // read by the head-mixing kernel only (seq_headmix.cuh); the step sends a layer there when one of them is set
     int keep_first;                   // with a window: keys at positions < keep_first stay visible
     const float* talk;                // [heads][heads] or null: score_h <- sum_g talk[h][g] score_g before masking
     // read by attn_prepare_kernel: what happens to the projections before they are used / cached
@@ -715,7 +742,19 @@ struct AttnShape {
     // the output gate's pre-activations when they are not part of the fused projection: gate[t * gate_ld + h] (null: behind q | k | v)
     const float* gate;
     int gate_ld;
+    const float *qgain, *kgain;       // [dim] each or null: q and k are divided by their RMS per head and multiplied by these BEFORE they turn
+    float rot_amp = 1.f;              // factor on the rotation's cosine and sine
+    const float* pb;                  // [heads] or null: no softmax, a visible key's weight is sigmoid(score + pb[h])
+    int out_ld = 0;                   // row stride of the output; 0: heads * vdim
+    float out_scale = 1.f;            // factor on the output
 };
+__device__ __forceinline__ size_t attn_out_stride(const AttnShape& s) { return s.out_ld ? (size_t)s.out_ld : (size_t)s.heads * s.vdim; }
+// score of a (query, key) pair from their dot product, and a visible key's weight when there is no softmax
+__device__ __forceinline__ float attn_score(const AttnShape& s, float dot) {
+    const float v = dot * s.scale;
+    return s.softcap > 0.f ? s.softcap * tanhf(v / s.softcap) : v;
+}
+__device__ __forceinline__ float attn_sigmoid(float score, float pb) { return 1.f / (1.f + expf(-(score + pb))); }
 // sigmoid output gate of (row t, head h), 1 without a gate
 __device__ __forceinline__ float attn_gate(const AttnShape& s, const float* qkvg, int t, int h) {
     if (!s.out_gate) return 1.f;
@@ -724,14 +763,16 @@ __device__ __forceinline__ float attn_gate(const AttnShape& s, const float* qkvg
     return 1.f / (1.f + expf(-z));
 }
 __device__ __forceinline__ size_t attn_vstride(const AttnShape& s) { return s.v_ld ? (size_t)s.v_ld : (size_t)s.kv_heads * s.vdim; }
-// the end of a softmax with a sink: (max, sum) -> the factor for the accumulated weighted values
+// the end of a softmax with a sink: (max, sum) -> the factor for the accumulated weighted values (the output's factor included);
+// weights that are not normalised only take that factor
 __device__ __forceinline__ float attn_finish_factor(const AttnShape& s, int h, float mx, float l) {
-    if (!s.sink) return 1.f / l;
+    if (s.pb) return s.out_scale;
+    if (!s.sink) return s.out_scale / l;
     const float sk = s.sink[h], m2 = fmaxf(mx, sk), c = expf(mx - m2);
-    return c / (l * c + expf(sk - m2));
+    return s.out_scale * c / (l * c + expf(sk - m2));
 }
-// Biases, rotation of q and k, unit RMS per head, the per-head query factor, unit-RMS values and the cache append: one block per
-// row.  q is rewritten in place; k and v go to the row's page.  inv_freq[rot_dims / 2] holds the (scaled) frequencies; the angle is
+// Biases, the per-head norm with a gain, rotation of q and k, unit RMS per head, the per-head query factor, unit-RMS values and the
+// cache append: one block per row.  q is rewritten in place; k and v go to the row's page.  inv_freq[rot_dims / 2] holds the (scaled) frequencies; the angle is
 // position * frequency in fp32.  Pair i of the rotated coordinates is (2 i, 2 i + 1) or, with rot_half, (i, i + rot_dims / 2).
 __global__ void attn_prepare_kernel(float* qkvg, StepMeta m, AttnShape s, const float* inv_freq, float* k_pool, float* v_pool) {
     pdl_launch_dependents();   // the kernel behind this one may be scheduled (and a few-row product may fetch its weights) ...
@@ -747,19 +788,36 @@ __global__ void attn_prepare_kernel(float* qkvg, StepMeta m, AttnShape s, const 
     for (int h = warp; h < nqk; h += nw) {
         float* v = row + (size_t)h * s.dim;   // q heads first, k heads right behind them
         const float* b = s.bias ? s.bias + (size_t)h * s.dim : nullptr;
+        const float* gn = h < s.heads ? s.qgain : s.kgain;   // norm in front of the rotation
+        float pre = 1.f;
+        if (gn) {
+            float sq = 0.f;
+            for (int i = lane; i < s.dim; i += 32) {
+                const float a = v[i] + (b ? b[i] : 0.f);
+                sq += a * a;
+            }
+            pre = 1.f / sqrtf(warp_sum(sq) / (float)s.dim + s.eps);
+        }
         float ss = 0.f;
         for (int i = lane; i < half; i += 32) {
             const int i0 = s.rot_half ? i : 2 * i, i1 = s.rot_half ? i + half : 2 * i + 1;
-            const float a = v[i0] + (b ? b[i0] : 0.f), c = v[i1] + (b ? b[i1] : 0.f);
+            float a = v[i0] + (b ? b[i0] : 0.f), c = v[i1] + (b ? b[i1] : 0.f);
+            if (gn) {
+                a *= pre * gn[i0];
+                c *= pre * gn[i1];
+            }
             float sn, cs;
             sincosf((float)pos * inv_freq[i], &sn, &cs);
+            sn *= s.rot_amp;
+            cs *= s.rot_amp;
             const float ra = a * cs - c * sn, rc = c * cs + a * sn;
             v[i0] = ra;
             v[i1] = rc;
             ss += ra * ra + rc * rc;
         }
         for (int i = 2 * half + lane; i < s.dim; i += 32) {
-            const float a = v[i] + (b ? b[i] : 0.f);
+            float a = v[i] + (b ? b[i] : 0.f);
+            if (gn) a *= pre * gn[i];
             v[i] = a;
             ss += a * a;
         }
@@ -820,7 +878,8 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_kernel(const
         o[i] = 0.f;
     }
     const int lo = (s.window > 0 && pos - s.window + 1 > 0) ? pos - s.window + 1 : 0;
-    float mx = -INFINITY, l = 0.f;
+    float mx = s.pb ? 0.f : -INFINITY, l = 0.f;   // (weights without a softmax: the running maximum stays 0)
+    const float pb = s.pb ? s.pb[h] : 0.f;
     const size_t kstride = (size_t)s.kv_heads * s.dim, vstride = attn_vstride(s);
     for (int j = lo + warp; j <= pos; j += kAttnWarps) {
         const size_t off = (size_t)table[j / kPageTokens] * kPageTokens + j % kPageTokens;
@@ -831,9 +890,9 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_kernel(const
             const int d = lane + 32 * i;
             if (d < s.dim) sc = fmaf(qr[i], kr[d], sc);
         }
-        sc = warp_sum(sc) * s.scale;
-        const float nm = fmaxf(mx, sc);
-        const float corr = expf(mx - nm), p = expf(sc - nm);
+        sc = attn_score(s, warp_sum(sc));
+        const float nm = s.pb ? 0.f : fmaxf(mx, sc);
+        const float corr = expf(mx - nm), p = s.pb ? attn_sigmoid(sc, pb) : expf(sc - nm);
         l = l * corr + p;
         const float* vr = v_pool + off * vstride + (size_t)g * s.vdim;
 #pragma unroll
@@ -867,7 +926,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_kernel(const
     for (int d = threadIdx.x; d < s.vdim; d += blockDim.x) {
         float acc = 0.f;
         for (int w = 0; w < kAttnWarps; ++w) acc += po[w * s.vdim + d] * f[w];
-        out[(size_t)t * (s.heads * s.vdim) + (size_t)h * s.vdim + d] = acc * fin;
+        out[(size_t)t * attn_out_stride(s) + (size_t)h * s.vdim + d] = acc * fin;
     }
 }
 
@@ -893,6 +952,7 @@ __global__ void __launch_bounds__(256) window_attention_tiled_kernel(const float
     const int p0 = m.row_pos[row0];
     const int* table = m.page_table + (size_t)m.ent_slot[m.row_ent[row0]] * m.table_stride;
     const int g = h / (s.heads / s.kv_heads);
+    const float pb = s.pb ? s.pb[h] : 0.f;
     for (int i = tid; i < kAttnTile * d; i += 256) {
         const int r = i / d, k = i % d;
         Qs[r * ldq + k] = r < n ? qkvg[(size_t)(row0 + r) * s.ld + (size_t)h * d + k] : 0.f;
@@ -949,8 +1009,13 @@ __global__ void __launch_bounds__(256) window_attention_tiled_kernel(const float
             for (int j = 0; j < 4; ++j) {
                 const int key = pg * kPageTokens + tx + 16 * j;
                 ok[j] = r < n && key <= pos && (s.window <= 0 || key > pos - s.window);
-                sc[i][j] = ok[j] ? sc[i][j] * s.scale : -INFINITY;
+                sc[i][j] = ok[j] ? attn_score(s, sc[i][j]) : -INFINITY;
                 tmax = fmaxf(tmax, sc[i][j]);
+            }
+            if (s.pb) {   // no softmax: nothing to rescale, nothing to add up
+#pragma unroll
+                for (int j = 0; j < 4; ++j) Ps[r * ldp + tx + 16 * j] = ok[j] ? attn_sigmoid(sc[i][j], pb) : 0.f;
+                continue;
             }
 #pragma unroll
             for (int o = 8; o > 0; o >>= 1) tmax = fmaxf(tmax, __shfl_xor_sync(0xFFFFFFFFu, tmax, o));
@@ -1005,7 +1070,7 @@ __global__ void __launch_bounds__(256) window_attention_tiled_kernel(const float
         for (int jj = 0; jj < DV4; ++jj) {
             const int col = tx * 4 + 64 * jj;
             if (col < dv) {
-                float* o = out + (size_t)t * (s.heads * dv) + (size_t)h * dv + col;
+                float* o = out + (size_t)t * attn_out_stride(s) + (size_t)h * dv + col;
                 o[0] = acc[i][jj * 4 + 0] * f;
                 o[1] = acc[i][jj * 4 + 1] * f;
                 o[2] = acc[i][jj * 4 + 2] * f;
@@ -1019,16 +1084,38 @@ inline size_t attn_tiled_smem_bytes(int d, int dv, bool v_in_k = false) {
 }
 
 // ---- gated feed-forward: act(gate) * up over the fused projection output [gate | up] ------------------------------------
-enum { ACT_RELU = 0, ACT_SILU = 1, ACT_GELU_TANH = 2 };
+enum { ACT_RELU = 0, ACT_SILU = 1, ACT_GELU_TANH = 2, ACT_CLAMPED_SWISH = 4 };
 __device__ __forceinline__ float ff_act(float z, int act) {
     if (act == 0 /*ACT_RELU*/) return fmaxf(z, 0.f);
     if (act == 1 /*ACT_SILU*/) return z / (1.f + expf(-z));
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
-__global__ void glu_kernel(const float* gu, int ff, int act, float* y, size_t n) {
+// the gated feed-forward's inner value.  CLAMPED_SWISH: g = min(gate, limit), u = up cut to [-limit, limit], g sigmoid(1.702 g) (u + 1)
+__device__ __forceinline__ float glu_pair(float g, float u, int act, float limit) {
+    if (act == ACT_CLAMPED_SWISH) {
+        g = fminf(g, limit);
+        u = fminf(fmaxf(u, -limit), limit);
+        return g / (1.f + expf(-1.702f * g)) * (u + 1.f);
+    }
+    return ff_act(g, act) * u;
+}
+// rows of [gate | up] (row stride ld) -> y (row stride ldy); V = 4: four neighbouring columns a thread (ff, ld, ldy in fours, 16-byte bases)
+template <int V>
+__global__ void glu_kernel(const float* gu, int ld, int ff, int act, float limit, float* y, int ldy, int T) {
+    pdl_launch_dependents();
+    pdl_wait_prior_grid();
+    const int per = ff / V;
+    const size_t n = (size_t)T * per;
     for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = i / ff, c = i % ff;
-        y[i] = ff_act(gu[t * 2 * ff + c], act) * gu[t * 2 * ff + ff + c];
+        const size_t t = i / per, c = (i % per) * V;
+        const float *g = gu + t * ld + c, *u = g + ff;
+        float* o = y + t * ldy + c;
+        if constexpr (V == 4) {
+            const float4 a = *reinterpret_cast<const float4*>(g), b = *reinterpret_cast<const float4*>(u);
+            *reinterpret_cast<float4*>(o) = make_float4(glu_pair(a.x, b.x, act, limit), glu_pair(a.y, b.y, act, limit), glu_pair(a.z, b.z, act, limit), glu_pair(a.w, b.w, act, limit));
+        } else {
+            *o = glu_pair(*g, *u, act, limit);
+        }
     }
 }
 
@@ -1227,17 +1314,17 @@ __global__ void __launch_bounds__(32 * NW) wkv_scan_split_kernel(WkvArgs a, Step
 #pragma unroll
     for (int i = 0; i < RP; ++i) Sg[(size_t)(warp * RP + i) * D + j] = S[i];
 }
-// o[t, head] / rms(o[t, head]) * normw * gate, in place: one warp per (row, head).  d = the head's output size; normw is
+// o[t, head] / rms(o[t, head]) * normw * gate, in place: one warp per (row, head).  ldo = row stride of o; d = the head's output size; normw is
 // [heads][d] (w_heads = 1) or one [d] vector shared by the heads (w_heads = 0); gate (optional) has row stride gate_ld and is
 // used as it is (gate_silu = 0) or through z * sigmoid(z) (gate_silu = 1).
-__global__ void head_rmsnorm_gate_kernel(float* o, const float* gate, int gate_ld, int gate_silu, const float* normw, int w_heads, int T, int heads, int d,
+__global__ void head_rmsnorm_gate_kernel(float* o, int ldo, const float* gate, int gate_ld, int gate_silu, const float* normw, int w_heads, int T, int heads, int d,
                                          float eps) {
     pdl_launch_dependents();   // the kernel behind this one may be scheduled (and a few-row product may fetch its weights) ...
     pdl_wait_prior_grid();     // ... while this one waits here for the kernel before it, when it was launched ahead of its end
     const int warp = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
     if (warp >= T * heads) return;
     const int hd = warp % heads, t = warp / heads;
-    const size_t base = (size_t)t * heads * d + (size_t)hd * d;
+    const size_t base = (size_t)t * ldo + (size_t)hd * d;
     float ss = 0.f;
     for (int i = lane; i < d; i += 32) ss += o[base + i] * o[base + i];
     ss = warp_sum(ss);

@@ -38,7 +38,8 @@ struct LinScanArgs {
     float inv_tau;
     float qscale;
     float* state;                 // [slots][heads][dk][dv]
-    float* out;                   // [T][heads * dv]
+    float* out;                   // row t, head hd at [t * ldo + hd * dv]
+    int ldo;
     int heads, dk, dv;
 };
 
@@ -110,7 +111,7 @@ __global__ void __launch_bounds__(128) linear_scan_kernel(LinScanArgs a, StepMet
                         acc0 = fmaf(qs[i], sv, acc0);
                     }
                 }
-                if (own) a.out[(size_t)(tc + c) * (a.heads * dv) + (size_t)hd * dv + j] = acc0 + acc1;
+                if (own) a.out[(size_t)(tc + c) * a.ldo + (size_t)hd * dv + j] = acc0 + acc1;
             }
         }
     }
@@ -178,7 +179,7 @@ __global__ void __launch_bounds__(32 * NW) linear_scan_split_kernel(LinScanArgs 
                 float s = part[0][c][l];
 #pragma unroll
                 for (int w = 1; w < NW; ++w) s += part[w][c][l];
-                a.out[(size_t)(tc + c) * (a.heads * dv) + (size_t)hd * dv + col0 + l] = s;
+                a.out[(size_t)(tc + c) * a.ldo + (size_t)hd * dv + col0 + l] = s;
             }
         }
     };

@@ -20,12 +20,17 @@ reads folder/config.json and folder/model.safetensors.  Registered architectures
                   projections, half-split rotation with linearly scaled frequencies, unit-RMS values, a per-head score factor and a
                   zero-score sink, latent attention with low-rank queries, a sliding window and a per-head output gate, a gated
                   gelu feed-forward, and a block of layers that is run several times in a row; on the layered sequence engine too.
+  * "Sebudra"  -- layers with ONE norm whose output the mixer and the feed-forward both read: biased softmax attention with a window and
+                  turn-dependent frequencies side by side with a state-space recurrence, causal attention with sigmoid weights, capped
+                  scores and normed queries / keys, gated linear attention; a clamped gated feed-forward or squared-relu experts chosen by
+                  sigmoid scores inside the best groups; layers that use an earlier layer's tensors; on the layered sequence engine too.
   * "llama"    -- the quantized Llama-style decoder of the persistent decode kernel (turboinfer_b200.capi.Model); built from
                   {"hidden", "layers", "heads", "inter", "vocab"} and fp32 tensors under the reference's names.
 """
 from __future__ import annotations
 
 import json
+import math
 import os
 from typing import Callable, Dict, List, Tuple
 
@@ -298,6 +303,109 @@ def zopipel_descs(cfg: dict, mode: int, max_tokens: int, max_seqs: int, tensor_s
 def _load_zopipel(cfg: dict, weights: dict, dtype: str, max_tokens: int, max_seqs: int):
     mode = {"bfloat16": _seq.BF16, "float32": _seq.F32}[dtype]
     desc, layers = zopipel_descs(cfg, mode, max_tokens, max_seqs)
+    return _seq.SeqModel(desc, layers).load(weights)
+
+
+def _sebudra_attention(d: "_seq.LayerDesc", mx: dict, where: str) -> None:
+    """heads, sizes, rotation, window, scale and cap of either attention of a Sebudra layer (queries and keys normed before they turn)."""
+    d.mixer, d.qk_norm = _seq.MIXER_ATTENTION, _seq.QK_NORM_HEAD_GAIN
+    d.heads, d.kv_heads = int(_req(mx, "heads", where)), int(_req(mx, "kv_heads", where))
+    d.dim, d.vdim, d.scale = int(_req(mx, "dim", where)), int(_req(mx, "vdim", where)), float(_req(mx, "scale", where))
+    rot = mx.get("rot")
+    if rot:
+        d.rot_dims, d.rot_base, d.rot_half = int(_req(rot, "dims", where + " rot")), float(_req(rot, "base", where + " rot")), 1
+        sc = rot.get("scaling")
+        if sc:
+            d.rot_scaled = _seq.ROT_BY_TURNS
+            d.rot_factor, d.rot_original = float(_req(sc, "factor", where + " rot.scaling")), float(_req(sc, "original", where + " rot.scaling"))
+            d.rot_high, d.rot_low = float(_req(sc, "fast", where + " rot.scaling")), float(_req(sc, "slow", where + " rot.scaling"))
+            d.rot_amp = 0.1 * math.log(d.rot_factor) + 1.0
+    mask = mx.get("mask")
+    if mask:
+        d.window = int(_req(mask, "size", where + " mask"))
+        if d.window < 1:
+            raise ValueError(f"{where}: mask.size {d.window}")
+    d.softcap = float(mx.get("softcap") or 0.0)
+
+
+def sebudra_descs(cfg: dict, mode: int, max_tokens: int, max_seqs: int, tensor_shapes: Dict[str, Tuple[int, ...]] = None):
+    """config.json of a Sebudra model -> (ModelDesc, [LayerDesc]).  The inner size of the gla decay projection, which the configuration
+    does not carry, is the row count of the checkpoint's l<i>.mix.a1."""
+    shapes = tensor_shapes or {}
+    entries = _req(cfg, "layers", "the model")
+
+    def owner(i: int) -> int:   # the layer whose tensors layer i uses, through chains
+        seen = set()
+        while entries[i].get("weights_of") is not None:
+            seen.add(i)
+            i = int(entries[i]["weights_of"])
+            if not 0 <= i < len(entries) or i in seen:
+                raise ValueError(f"layer {min(seen)}: weights_of leads to no layer with tensors of its own")
+        return i
+
+    layers: List[_seq.LayerDesc] = []
+    for i, L in enumerate(entries):
+        where, own = f"layer {i}", owner(i)
+        mx = _req(L, "mixer", where)
+        d = _seq.LayerDesc()
+        kind = _req(L, "type", where)
+        if kind == "parallel":
+            _sebudra_attention(d, _req(mx, "left", where), where + " left")
+            d.proj_bias = _seq.BIAS_QKV
+            rt = _req(mx, "right", where)
+            d.ssm_heads, d.ssm_vdim = int(_req(rt, "heads", where + " right")), int(_req(rt, "vdim", where + " right"))
+            d.ssm_state, d.ssm_groups = int(_req(rt, "state", where + " right")), int(_req(rt, "groups", where + " right"))
+            d.ssm_taps, d.ssm_parts = int(_req(rt, "conv", where + " right")), int(_req(rt, "norm_groups", where + " right"))
+            d.left_scale, d.right_scale = float(_req(mx, "left_scale", where)), float(_req(mx, "right_scale", where))
+        elif kind == "attention":
+            _sebudra_attention(d, mx, where)
+            d.weights_kind = _seq.WEIGHTS_SIGMOID
+        elif kind == "gla":
+            d.mixer = _seq.MIXER_GLA
+            d.heads, d.dim, d.vdim = int(_req(mx, "heads", where)), int(_req(mx, "dim", where)), int(_req(mx, "vdim", where))
+            d.kv_heads, d.decay_tau = d.heads, float(_req(mx, "tau", where))
+            shape = shapes.get(f"l{own}.mix.a1")
+            if not shape:
+                raise ValueError(f"{where}: the decay projection l{own}.mix.a1 is missing from the checkpoint")
+            d.decay_rank = int(shape[0])
+        else:
+            raise ValueError(f"{where}: unknown mixer type '{kind}'")
+        mlp = L.get("mlp")
+        if mlp:
+            fk = _req(mlp, "kind", where + " mlp")
+            if fk == "dense":
+                d.ff_kind, d.ff_act = _seq.FF_GLU, _seq.ACT_CLAMPED_SWISH
+                d.ff, d.ff_limit = int(_req(mlp, "ff", where + " mlp")), float(_req(mlp, "limit", where + " mlp"))
+            elif fk == "moe":
+                r = _req(mlp, "router", where + " mlp")
+                d.ff_kind, d.ff = _seq.FF_EXPERTS, int(_req(_req(mlp, "expert", where + " mlp"), "ff", where + " mlp.expert"))
+                d.expert_form, d.route_kind = _seq.EXPERT_RELU2, _seq.ROUTE_SIGMOID
+                d.experts, d.top = int(_req(r, "experts", where + " router")), int(_req(r, "top", where + " router"))
+                d.route_scale = float(r.get("scale", 1.0))
+                g = r.get("groups") or {}
+                d.groups = int(g.get("count", 1))
+                d.groups_keep = int(g.get("keep", d.groups))
+                sh = mlp.get("shared")
+                d.shared_ff = int(_req(sh, "ff", where + " mlp.shared")) if sh else 0
+            else:
+                raise ValueError(f"{where}: unknown feed-forward kind '{fk}'")
+        d.weights_of = 0 if own == i else 1 + own
+        layers.append(d)
+    m = _seq.ModelDesc()
+    m.vocab, m.width, m.n_layers = int(_req(cfg, "vocab", "the model")), int(_req(cfg, "width", "the model")), len(layers)
+    m.norm_eps = float(_req(_req(cfg, "norm", "the model"), "eps", "norm"))
+    m.norm_kind, m.norm_place = _seq.NORM_VECTOR, _seq.NORMS_SHARED
+    m.embed_scale = float(_req(_req(cfg, "embedding", "the model"), "scale", "embedding"))
+    m.logit_scale = 1.0
+    m.mode, m.max_tokens, m.max_seqs = mode, int(max_tokens), int(max_seqs)
+    return m, layers
+
+
+@register("Sebudra")
+def _load_sebudra(cfg: dict, weights: dict, dtype: str, max_tokens: int, max_seqs: int):
+    mode = {"bfloat16": _seq.BF16, "float32": _seq.F32}[dtype]
+    shapes = {k: tuple(getattr(v, "shape", ())) for k, v in weights.items()}
+    desc, layers = sebudra_descs(cfg, mode, max_tokens, max_seqs, shapes)
     return _seq.SeqModel(desc, layers).load(weights)
 
 

@@ -11,14 +11,18 @@ import numpy as np
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 BF16, F32 = 0, 1
-MIXER_ATTENTION, MIXER_WKV, MIXER_GLA, MIXER_HGRN2, MIXER_LATENT = 0, 1, 2, 3, 4
-ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_XIELU = 0, 1, 2, 3
+MIXER_ATTENTION, MIXER_WKV, MIXER_GLA, MIXER_HGRN2, MIXER_LATENT, MIXER_SSM = 0, 1, 2, 3, 4, 5
+ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_XIELU, ACT_CLAMPED_SWISH = 0, 1, 2, 3, 4
 FF_GLU, FF_POLYNORM, FF_EXPERTS, FF_DENSE = 0, 1, 2, 3
 NORM_SCALAR, NORM_ONE_PLUS, NORM_VECTOR = 0, 1, 2
 SINK_NONE, SINK_LEARNED, SINK_ZERO = 0, 1, 2
-ROUTE_SOFTMAX_ALL, ROUTE_TOP_LOGITS = 0, 1
-QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_WHOLE = 0, 1, 2
-NORMS_AROUND, NORMS_BEHIND, NORMS_FRONT = 0, 1, 2
+ROUTE_SOFTMAX_ALL, ROUTE_TOP_LOGITS, ROUTE_SIGMOID = 0, 1, 2
+QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_WHOLE, QK_NORM_HEAD_GAIN = 0, 1, 2, 3
+NORMS_AROUND, NORMS_BEHIND, NORMS_FRONT, NORMS_SHARED = 0, 1, 2, 3
+WEIGHTS_SOFTMAX, WEIGHTS_SIGMOID = 0, 1
+BIAS_NONE, BIAS_QKVO, BIAS_QKV = 0, 1, 2
+EXPERT_GATED, EXPERT_RELU2 = 0, 1
+ROT_BY_WAVELENGTH, ROT_BY_TURNS = 1, 2
 
 
 class SeqError(RuntimeError):
@@ -36,7 +40,10 @@ class LayerDesc(C.Structure):
                 ("softcap", C.c_float), ("talk", C.c_int32), ("keep_first", C.c_int32), ("route_kind", C.c_int32),
                 ("shared_plain", C.c_int32), ("conv_taps", C.c_int32), ("layer_scale", C.c_int32), ("conv_ff", C.c_int32),
                 ("rot_half", C.c_int32), ("rot_linear", C.c_float), ("proj_bias", C.c_int32), ("v_norm", C.c_int32),
-                ("head_temp", C.c_int32), ("q_rank", C.c_int32)]
+                ("head_temp", C.c_int32), ("q_rank", C.c_int32), ("weights_kind", C.c_int32), ("rot_amp", C.c_float),
+                ("ssm_heads", C.c_int32), ("ssm_vdim", C.c_int32), ("ssm_state", C.c_int32), ("ssm_groups", C.c_int32), ("ssm_taps", C.c_int32),
+                ("ssm_parts", C.c_int32), ("left_scale", C.c_float), ("right_scale", C.c_float), ("ff_limit", C.c_float),
+                ("expert_form", C.c_int32), ("route_scale", C.c_float), ("weights_of", C.c_int32)]
 
     def __init__(self, *a, **kw):
         super().__init__(*a, **kw)
@@ -49,7 +56,7 @@ class ModelDesc(C.Structure):
                 ("loop_stop", C.c_int32), ("loop_times", C.c_int32), ("norm_eps", C.c_float), ("logit_scale", C.c_float),
                 ("mode", C.c_int32), ("max_tokens", C.c_int32), ("max_seqs", C.c_int32), ("norm_kind", C.c_int32),
                 ("logit_softcap", C.c_float), ("side_dim", C.c_int32), ("norm_place", C.c_int32), ("pos_base", C.c_float),
-                ("tied_head", C.c_int32), ("loop_plain", C.c_int32), ("streams", C.c_int32)]
+                ("tied_head", C.c_int32), ("loop_plain", C.c_int32), ("streams", C.c_int32), ("embed_scale", C.c_float)]
 
 
 _i32 = C.POINTER(C.c_int32)
