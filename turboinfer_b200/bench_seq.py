@@ -90,6 +90,27 @@ def zopipel_config_for(size: str) -> dict:
             "norm": {"eps": 1e-6}, "streams": 4, "vocab": z["vocab"], "width": z["width"]}
 
 
+def sebudra_config_for(size: str) -> dict:
+    """Seven layers in the order parallel, gla, attention, parallel, gla, attention, parallel (the last one on the first one's tensors).
+    Parallel: the size's heads over its window beside a state-space mixer with inner size = width (heads of 64, state 128, one group per
+    eight heads, four taps); gla: the size's heads with 64 key and 128 value channels; attention: the size's heads over all earlier
+    tokens.  Dense feed-forwards of the size's inner width, routed experts (8 of a quarter of it, 2 chosen from the best of 2 groups, a
+    shared expert of half of it) in the attention layers."""
+    z = SIZES[size]
+    D, H, d = z["width"], z["heads"], z["dim"]
+    left = {"heads": H, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "mask": {"size": z["window"]}, "scale": 1.0 / math.sqrt(d),
+            "rot": {"base": 10000.0, "dims": d, "scaling": {"factor": 8.0, "fast": 32.0, "slow": 1.0, "original": 4096}}}
+    right = {"heads": D // 64, "vdim": 64, "state": 128, "groups": max(1, D // 512), "conv": 4, "norm_groups": max(1, D // 512)}
+    att = {"heads": H, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "rot": {"base": 500000.0, "dims": d}, "scale": 1.0 / math.sqrt(d), "softcap": 50.0}
+    gla = {"heads": H, "dim": 64, "vdim": 128, "tau": 16.0}
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    moe = {"kind": "moe", "expert": {"ff": z["ff"] // 4}, "router": {"experts": 8, "top": 2, "scale": 2.5, "groups": {"count": 2, "keep": 1}},
+           "shared": {"ff": z["ff"] // 2}}
+    par = {"type": "parallel", "mlp": dense, "mixer": {"left": left, "right": right, "left_scale": 0.75, "right_scale": 1.25}}
+    order = [par, {"type": "gla", "mixer": gla, "mlp": dense}, {"type": "attention", "mixer": att, "mlp": moe}] * 2 + [dict(par, weights_of=0)]
+    return {"architecture": "Sebudra", "embedding": {"scale": math.sqrt(D)}, "layers": order, "norm": {"eps": 1e-6}, "vocab": z["vocab"], "width": D}
+
+
 def build_synthetic(cfg: dict, rank: int, dtype: str, max_tokens: int, max_seqs: int) -> seq.SeqModel:
     mode = {"bfloat16": seq.BF16, "float32": seq.F32}[dtype]
     if cfg["architecture"] == "Gulazen":
@@ -100,6 +121,9 @@ def build_synthetic(cfg: dict, rank: int, dtype: str, max_tokens: int, max_seqs:
         shapes = {f"l{i}.mix.a1": (rank, cfg["width"]) for i, L in enumerate(cfg["layers"]) if L["type"] == "gla"}
         shapes.update({f"l{i}.rg1": (cfg["width"], cfg["width"]) for i in range(len(cfg["layers"]))})
         desc, layers = models.tudasun_descs(cfg, mode, max_tokens, max_seqs, shapes)
+    elif cfg["architecture"] == "Sebudra":
+        shapes = {f"l{i}.mix.a1": (rank, cfg["width"]) for i, L in enumerate(cfg["layers"]) if L["type"] == "gla"}
+        desc, layers = models.sebudra_descs(cfg, mode, max_tokens, max_seqs, shapes)
     else:
         shapes = {f"l{i}.mix.w1": (rank, cfg["width"]) for i, L in enumerate(cfg["layers"]) if L["type"] == "wkv"}
         desc, layers = models.binusun_descs(cfg, mode, max_tokens, max_seqs, shapes)
@@ -112,6 +136,10 @@ def build_synthetic(cfg: dict, rank: int, dtype: str, max_tokens: int, max_seqs:
             amp, off = 0.25, 1.0   # plain gains and per-head score factors around one
         elif cfg["architecture"] == "Zopipel" and leaf == "b":
             amp, off = 0.1, 0.0
+        elif cfg["architecture"] == "Sebudra" and (leaf in ("norm1", "D") or leaf == "norm"):
+            amp, off = 0.25, 1.0   # plain gains around one
+        elif cfg["architecture"] == "Sebudra" and leaf in ("dt_bias", "A_log", "pb", "correction", "b"):
+            amp, off = 0.5, {"dt_bias": -3.0, "pb": -4.0}.get(leaf, 0.0)
         elif leaf in ("in", "out") and ".hc" in name:
             amp, off = 0.2, 0.6
         elif leaf == "mix" and ".hc" in name:
@@ -154,7 +182,7 @@ def prompt(n: int, vocab: int, offset: int = 0):
 
 def measure_seq(size: str, dtype: str, n_prompt: int, n_new: int, batch: int, steps: int, warmup: int, design: str = "Binusun") -> dict:
     cfg = {"Tudasun": tudasun_config_for, "Gulazen": gulazen_config_for, "BinusunAttention": binusun_attention_config_for,
-           "Zopipel": zopipel_config_for}.get(design, config_for)(size)
+           "Zopipel": zopipel_config_for, "Sebudra": sebudra_config_for}.get(design, config_for)(size)
     m = build_synthetic(cfg, SIZES[size]["rank"], dtype, max_tokens=(n_prompt + n_new + 64) * max(batch, 1) + 64, max_seqs=max(batch, 1))
     V = cfg["vocab"]
     launches0 = seq.launch_count()
@@ -186,7 +214,8 @@ def measure_seq(size: str, dtype: str, n_prompt: int, n_new: int, batch: int, st
     m.free()
     pre_ms, dec_ms = statistics.median(pre_dev), statistics.median(dec_dev)
     # routed experts: a decode step reads only the experts its rows chose; with one row that is at most `top` of them a layer
-    idle = sum((L["mlp"]["router"]["experts"] - min(L["mlp"]["router"]["top"], L["mlp"]["router"]["experts"])) * 3.0 * L["mlp"]["expert"]["ff"] * cfg["width"] * 2.0
+    mats = 2.0 if design == "Sebudra" else 3.0   # matrices of an expert
+    idle = sum((L["mlp"]["router"]["experts"] - min(L["mlp"]["router"]["top"], L["mlp"]["router"]["experts"])) * mats * L["mlp"]["expert"]["ff"] * cfg["width"] * 2.0
                for L in cfg["layers"] if L.get("mlp") and L["mlp"].get("kind") == "moe")
     extra = {}
     if idle and batch == 1:
@@ -244,6 +273,16 @@ def compare_zopipel(size: str, steps: int, warmup: int, n_prompt: int = 2048, n_
     """Zopipel next to the closest model of the library, seven Binusun attention layers on the same engine (bf16 weights both)."""
     out = {"size": size, "shape": SIZES[size], "prompt_tokens": n_prompt, "decode_steps": n_new}
     for design, key in (("Zopipel", "zopipel_bf16"), ("BinusunAttention", "binusun_attention_bf16")):
+        out[key] = measure_seq(size, "bfloat16", n_prompt, n_new, 1, steps, warmup, design)
+        out[key + "_batch4"] = {k: v for k, v in measure_seq(size, "bfloat16", 256, n_new, 4, 1, 1, design).items() if k.startswith("decode") or k == "batch"}
+    return out
+
+
+def compare_sebudra(size: str, steps: int, warmup: int, n_prompt: int = 2048, n_new: int = 64) -> dict:
+    """Sebudra next to the closest model of the library, Tudasun (gla, attention and routed experts) on the same engine (bf16 weights both)."""
+    out = {"size": size, "shape": SIZES[size], "prompt_tokens": n_prompt, "decode_steps": n_new}
+    for design in ("Sebudra", "Tudasun", "BinusunAttention"):
+        key = {"BinusunAttention": "binusun_attention"}.get(design, design.lower()) + "_bf16"
         out[key] = measure_seq(size, "bfloat16", n_prompt, n_new, 1, steps, warmup, design)
         out[key + "_batch4"] = {k: v for k, v in measure_seq(size, "bfloat16", 256, n_new, 4, 1, 1, design).items() if k.startswith("decode") or k == "batch"}
     return out
