@@ -219,10 +219,11 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
 
 // ---- decode rows with long windows: key chunks in parallel -----------------------------------------------------------------
 // grid (rows, heads, splits): split z of a (row, head) takes keys lo + z * chunk .. and leaves its partial (max, sum, o[dv]) in
-// `part`; attention_merge_kernel combines the splits and applies the gate.  chunk = ceil(visible keys / splits).
+// `part`; the block that finishes last (counted in `arrived` [rows][heads], zero between launches) combines the splits in ascending
+// order, whichever block that is, and applies the gate.  chunk = ceil(visible keys / splits); at most 32 splits.
 template <int PL>
 __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_split_kernel(const float* qkvg, StepMeta m, AttnShape s, const int* rows, int splits,
-                                                                                  const float* k_pool, const float* v_pool, float* part) {
+                                                                                  const float* k_pool, const float* v_pool, float* part, int* arrived, float* out) {
     pdl_launch_dependents();   // the kernel behind this one may be scheduled (and a few-row product may fetch its weights) ...
     pdl_wait_prior_grid();     // ... while this one waits here for the kernel before it, when it was launched ahead of its end
     extern __shared__ float sm[];
@@ -313,34 +314,35 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_split_kernel
         dst[0] = Mx;
         dst[1] = L;
     }
-}
-// one warp per (row, head): lane z holds split z's (max, sum); the output coordinates are spread over the lanes
-__global__ void attention_merge_kernel(const float* part, const float* qkvg, StepMeta m, AttnShape s, const int* rows, int n_rows, int splits, float* out) {
-    pdl_launch_dependents();   // the kernel behind this one may be scheduled (and a few-row product may fetch its weights) ...
-    pdl_wait_prior_grid();     // ... while this one waits here for the kernel before it, when it was launched ahead of its end
-    const int wid = (blockIdx.x * blockDim.x + threadIdx.x) >> 5, lane = threadIdx.x & 31;
-    if (wid >= n_rows * s.heads) return;
-    const int bx = wid / s.heads, h = wid % s.heads, t = rows ? rows[bx] : bx;
+    __shared__ int last;
+    __threadfence();
+    __syncthreads();
+    if (threadIdx.x == 0) {
+        int* cnt = arrived + (size_t)bx * s.heads + h;
+        last = atomicAdd(cnt, 1) == splits - 1;
+        if (last) *cnt = 0;
+    }
+    __syncthreads();
+    if (!last) return;
+    __threadfence();
+    // lane z holds split z's (max, sum); every warp works out the factors, the coordinates are spread over the block
     const size_t ps = (size_t)(s.vdim + 2);
     const float* p = part + ((size_t)bx * s.heads + h) * splits * ps;
-    const float mz = lane < splits ? p[(size_t)lane * ps] : -INFINITY;
-    const float lz = lane < splits ? p[(size_t)lane * ps + 1] : 0.f;
-    const float Mx = warp_max(mz);
-    const float fz = mz == -INFINITY ? 0.f : expf(mz - Mx);
-    const float L = warp_sum(lz * fz);
-    const float fin = attn_finish_factor(s, h, Mx, L) * attn_gate(s, qkvg, t, h);
-    // every split's factor in registers first, so that the loads of a coordinate's partials do not wait on one another
-    constexpr int kMaxSplits = 32;   // (a lane holds a split's statistics)
-    float fs[kMaxSplits];
+    const float mz = lane < splits ? __ldcg(p + (size_t)lane * ps) : -INFINITY;
+    const float lz = lane < splits ? __ldcg(p + (size_t)lane * ps + 1) : 0.f;
+    const float Mt = warp_max(mz);
+    const float fz = mz == -INFINITY ? 0.f : expf(mz - Mt);
+    const float fin = attn_finish_factor(s, h, Mt, warp_sum(lz * fz)) * attn_gate(s, qkvg, t, h);
+    constexpr int kMaxSplits = 32;
+    float fs[kMaxSplits];   // every split's factor in registers first, so that the loads of a coordinate's partials do not wait on one another
 #pragma unroll
-    for (int z = 0; z < kMaxSplits; ++z) fs[z] = __shfl_sync(0xFFFFFFFFu, fz, z);
-    for (int d0 = 0; d0 < s.vdim; d0 += 32) {
-        const int d = d0 + lane;
+    for (int q = 0; q < kMaxSplits; ++q) fs[q] = __shfl_sync(0xFFFFFFFFu, fz, q);
+    for (int d = threadIdx.x; d < s.vdim; d += blockDim.x) {
         float acc = 0.f;
 #pragma unroll
-        for (int z = 0; z < kMaxSplits; ++z)
-            if (z < splits && d < s.vdim) acc = fmaf(p[(size_t)z * ps + 2 + d], fs[z], acc);
-        if (d < s.vdim) out[(size_t)t * attn_out_stride(s) + (size_t)h * s.vdim + d] = acc * fin;
+        for (int q = 0; q < kMaxSplits; ++q)
+            if (q < splits) acc = fmaf(__ldcg(p + (size_t)q * ps + 2 + d), fs[q], acc);
+        out[(size_t)t * attn_out_stride(s) + (size_t)h * s.vdim + d] = acc * fin;
     }
 }
 

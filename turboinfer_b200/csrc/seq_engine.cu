@@ -38,8 +38,8 @@ cudaStream_t g_stream = nullptr;
 uint64_t g_launches = 0;
 size_t g_smem_optin = 0;
 bool g_use_tiled_attn = true;   // TURBOINFER_B200_SEQ_TILED_ATTN=0: every row goes through the row-at-a-time attention kernel
-constexpr int kAttnTiledMinRows = 8;
-constexpr int kAttnMaxSplits = 16;    // key chunks of a decode row's attention   // portions at least this long are cut into attention tiles
+constexpr int kAttnTiledMinRows = 8;   // portions at least this long are cut into attention tiles
+constexpr int kAttnMaxSplits = 16;    // key chunks of a decode row's attention
 bool g_use_pdl = true;  // TURBOINFER_B200_SEQ_PDL=0: the few-row products wait for their predecessor before they start (A/B measurements)
 bool g_use_row_mma = true;   // TURBOINFER_B200_SEQ_ROW_MMA=0: few-row products stay on the fp32 multiply-add kernel (A/B measurements)
 bool g_use_tc = true;   // TURBOINFER_B200_SEQ_TC=0: prompt-side products stay on the warp-level tensor path (A/B measurements)
@@ -264,6 +264,7 @@ struct Model {
     bool any_rgbuf = false;
     DevBuf<int> meta, picks;
     DevBuf<__nv_bfloat16> abf;   // bf16 copy of a product's activations for the tcgen05 path: [rows][max_k]
+    DevBuf<int> attn_arrived;    // split-key attention: finished splits of a (row, head), zero between launches
     DevBuf<float> attn_part;     // split-key attention partials: [rows][heads][splits][vdim + 2]
     DevBuf<float> mix_S, mix_den; // head-mixing attention: scores / weights [rows of a batch][heads][keys], 1 / denominators [rows][heads]
     bool any_mixed = false;
@@ -832,7 +833,11 @@ int ensure_scratch(Model& m, int rows, int want) {
         if (m.any_rgbuf) TRY(m.rgbuf.alloc(R * D));
         if (m.dbg) TRY(m.dbg_buf.alloc(m.runs.size() * R * D));
         if (m.d.mode == TI_SEQ_BF16 && g_use_tc) TRY(m.abf.alloc(R * (size_t)m.max_k));
-        if (m.max_heads_v) TRY(m.attn_part.alloc(R * (size_t)m.max_heads_v * kAttnMaxSplits));
+        if (m.max_heads_v) {
+            TRY(m.attn_part.alloc(R * (size_t)m.max_heads_v * kAttnMaxSplits));
+            TRY(m.attn_arrived.alloc(R * (size_t)m.max_heads_v));
+            CK(cudaMemsetAsync(m.attn_arrived.p, 0, m.attn_arrived.n * sizeof(int), g_stream));
+        }
         m.cap_rows = (int)R;
     }
     if (want > m.cap_want) {
@@ -1031,6 +1036,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
     LAUNCHED();
     const float eps = m.d.norm_eps;
     const int gv = m.gvec;
+    const int prepare_threads = T <= 2 * g_num_sms ? kPrepareFewThreads : 128;
     // the end of a sublayer: (identity experts) -> (gate) -> norm behind the sublayer -> residual sum (-> the next sublayer's input)
     auto post = [&](const float* gain, int gain_vec, const float* gain2, const float* gate, int gate_ld, const float* gate_bias, const float* idw) -> int {
         PostArgs a{};
@@ -1086,6 +1092,15 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         return 0;
     };
     // the short convolution in front of a sublayer: y = x + conv(x) over the sequence's last inputs; the slot then keeps the newest ones
+    auto conv_save = [&](const float* in, int ldx, int D, int taps, float* state) -> int {
+        bool many = false;   // (an entry of one row has shifted its state in the convolution kernel)
+        for (int e = 0; e < E; ++e) many = many || counts[e] > 1;
+        if (taps > 1 && many) {
+            TRY(launch_dep(short_conv_save_kernel, dim3(E, (D + nt - 1) / nt), dim3(nt), 0, in, ldx, sm, D, taps, state));
+            LAUNCHED();
+        }
+        return 0;
+    };
     auto conv = [&](const float* in, const ConvForm& cf, int D, const float* w, int taps, float* state, float* out) -> int {   // over D channels
         constexpr int kConvRows = 8;   // rows a block of the many-rows kernel takes
         const dim3 rows_grid((T + kConvRows - 1) / kConvRows, (D / 4 + 127) / 128);
@@ -1095,12 +1110,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         else if (v4) TRY(launch_dep(short_conv_kernel<4>, dim3(T), dim3(std::min(nt, (D / 4 + 31) / 32 * 32)), 0, in, cf, sm, D, taps, w, state, out));
         else TRY(launch_dep(short_conv_kernel<1>, dim3(T, T <= 64 ? (D + nt - 1) / nt : 1), dim3(nt), 0, in, cf, sm, D, taps, w, state, out));
         LAUNCHED();
-        bool many = false;   // (an entry of one row has shifted its state in the kernel above)
-        for (int e = 0; e < E; ++e) many = many || counts[e] > 1;
-        if (taps > 1 && many) {
-            TRY(launch_dep(short_conv_save_kernel, dim3(E, (D + nt - 1) / nt), dim3(nt), 0, in, cf.ldx, sm, D, taps, state));
-            LAUNCHED();
-        }
+        TRY(conv_save(in, cf.ldx, D, taps, state));
         return 0;
     };
     auto short_conv = [&](const float* in, const float* w, int taps, float* state, float* out) -> int {
@@ -1161,10 +1171,8 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             int splits = 1;
             if (span >= 32) splits = std::max(1, std::min({(span + 15) / 16, kAttnMaxSplits, (2 * g_num_sms) / std::max(1, n_rest * s.heads)}));
             if (splits > 1 && m.attn_part.p) {
-                if (wide) TRY(launch_dep(window_attention_split_kernel<kAttnWidePerLane>, dim3(n_rest, s.heads, splits), dim3(kAttnWarps * 32), smem, q, sm, s, rest, splits, kp, vp, m.attn_part.p));
-                else TRY(launch_dep(window_attention_split_kernel<kAttnMaxPerLane>, dim3(n_rest, s.heads, splits), dim3(kAttnWarps * 32), smem, q, sm, s, rest, splits, kp, vp, m.attn_part.p));
-                LAUNCHED();
-                TRY(launch_dep(attention_merge_kernel, dim3((n_rest * s.heads + 7) / 8), dim3(256), 0, (const float*)m.attn_part.p, q, sm, s, rest, n_rest, splits, out));
+                if (wide) TRY(launch_dep(window_attention_split_kernel<kAttnWidePerLane>, dim3(n_rest, s.heads, splits), dim3(kAttnWarps * 32), smem, q, sm, s, rest, splits, kp, vp, m.attn_part.p, m.attn_arrived.p, out));
+                else TRY(launch_dep(window_attention_split_kernel<kAttnMaxPerLane>, dim3(n_rest, s.heads, splits), dim3(kAttnWarps * 32), smem, q, sm, s, rest, splits, kp, vp, m.attn_part.p, m.attn_arrived.p, out));
                 LAUNCHED();
             } else {
                 if (wide) TRY(launch_dep(window_attention_kernel<kAttnWidePerLane>, dim3(n_rest, s.heads), dim3(kAttnWarps * 32), smem, q, sm, s, rest, kp, vp, out));
@@ -1277,6 +1285,19 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         LAUNCHED();
         return 0;
     };
+    auto moe_act = [&](const LayerW& L, int ld, const float* wdense, float* y, int ldy) -> int {
+        const ti_seq_layer_desc& d = L.d;
+        const int W = L.ff_width;
+        const bool v4 = d.ff % 4 == 0 && d.shared_ff % 4 == 0 && ld % 4 == 0 && ldy % 4 == 0 && (L.off_up < 0 || L.off_up % 4 == 0) && (L.off_sh < 0 || L.off_sh % 4 == 0) &&
+                        (reinterpret_cast<uintptr_t>(y) & 15) == 0;
+        const int per = v4 ? 4 : 1, want = (W / per + 255) / 256, groups = T <= 2 * g_num_sms ? want : std::min(want, 4);
+        if (v4) TRY(launch_dep(moe_act_kernel<4>, dim3(T, groups), dim3(256), 0, (const float*)m.proj.p, ld, L.off_up, d.experts, d.ff, wdense, L.off_sh, d.shared_ff, L.off_sg, y, ldy,
+                               d.expert_form, T));
+        else TRY(launch_dep(moe_act_kernel<1>, dim3(T, groups), dim3(256), 0, (const float*)m.proj.p, ld, L.off_up, d.experts, d.ff, wdense, L.off_sh, d.shared_ff, L.off_sg, y, ldy,
+                            d.expert_form, T));
+        LAUNCHED();
+        return 0;
+    };
     // one norm for both sublayers: x <- x + mixer(norm(x)) + ff(norm(x)).  ONE product in front (all mixers' and the feed-forward's input
     // matrices stacked; few rows: the norm in its prologue, the dense feed-forward's gating in its epilogue), the mixers and the
     // feed-forward each write their part of the rows of ONE product behind (output matrices side by side along K, residual sum in its epilogue)
@@ -1306,14 +1327,25 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         } else {
             TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, sparse ? L.off_up : L.n_front, D, EPI_NONE, 1.f, few ? &fn : nullptr));
         }
+        const int inner = d.ssm_heads * d.ssm_vdim;
+        const float* ssm_u = m.proj.p + std::max(L.off_in, 0);   // [z | x | B | C | dt]
+        ConvForm cf{};
+        cf.ldx = nf; cf.bias = L.ssm_conv_b; cf.silu = 1;
         if (d.mixer == TI_SEQ_MIXER_ATTENTION) {
             AttnShape s{};
             s.heads = d.heads; s.kv_heads = d.kv_heads; s.dim = d.dim; s.vdim = d.vdim; s.window = d.window; s.rot_dims = d.rot_dims; s.rot_half = d.rot_half;
             s.qk_norm = d.qk_norm == TI_SEQ_QK_NORM_HEAD ? 1 : 0; s.qgain = L.qgain; s.kgain = L.kgain; s.rot_amp = d.rot_amp > 0.f ? d.rot_amp : 1.f;
             s.scale = d.scale; s.eps = eps; s.ld = nf; s.sink = L.sink; s.softcap = d.softcap; s.v_norm = d.v_norm; s.bias = L.qkv_bias.p; s.temp = L.temp; s.pb = L.pb;
             s.out_ld = KB; s.out_scale = has_ssm(d) ? d.left_scale : 1.f;
-            TRY(launch_dep(attn_prepare_kernel, dim3(T), dim3(128), 0, m.proj.p, sm, s, L.inv_freq.p, R.k_pool.p, R.v_pool.p));
-            LAUNCHED();
+            if (few && has_ssm(d)) {   // with the state-space mixer's convolution in the same launch
+                TRY(launch_dep(attn_prepare_conv_kernel, dim3(T, 1 + (ssm_channels(d) + kPrepareFewThreads - 1) / kPrepareFewThreads), dim3(kPrepareFewThreads), 0, m.proj.p, sm, s,
+                               (const float*)L.inv_freq.p, R.k_pool.p, R.v_pool.p, ssm_u + inner, cf, ssm_channels(d), d.ssm_taps, L.ssm_conv, R.ssm_conv.p, m.aux2.p));
+                LAUNCHED();
+                TRY(conv_save(ssm_u + inner, nf, ssm_channels(d), d.ssm_taps, R.ssm_conv.p));
+            } else {
+                TRY(launch_dep(attn_prepare_kernel, dim3(T), dim3(prepare_threads), 0, m.proj.p, sm, s, L.inv_freq.p, R.k_pool.p, R.v_pool.p));
+                LAUNCHED();
+            }
             TRY(attention(s, m.proj.p, R.k_pool.p, R.v_pool.p, m.act.p));
         } else if (d.mixer == TI_SEQ_MIXER_GLA) {
             const int H = d.heads, C = H * d.dim;
@@ -1328,11 +1360,9 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             LAUNCHED();
         }
         if (has_ssm(d)) {
-            const int inner = d.ssm_heads * d.ssm_vdim, ch = ssm_channels(d);
-            const float* u = m.proj.p + L.off_in;   // [z | x | B | C | dt]
-            ConvForm cf{};
-            cf.ldx = nf; cf.bias = L.ssm_conv_b; cf.silu = 1;
-            TRY(conv(u + inner, cf, ch, L.ssm_conv, d.ssm_taps, R.ssm_conv.p, m.aux2.p));
+            const int ch = ssm_channels(d);
+            const float* u = ssm_u;
+            if (!few || d.mixer == TI_SEQ_MIXER_SSM) TRY(conv(u + inner, cf, ch, L.ssm_conv, d.ssm_taps, R.ssm_conv.p, m.aux2.p));
             SsmArgs a{};
             a.xbc = m.aux2.p; a.ld = ch; a.dt = u + inner + ch; a.ld_dt = nf; a.dt_bias = L.dt_bias; a.A_log = L.A_log; a.state = R.ssm_state.p;
             a.out = m.act.p + L.back_ssm; a.ldo = KB; a.heads = d.ssm_heads; a.N = d.ssm_state; a.dv = d.ssm_vdim; a.groups = d.ssm_groups;
@@ -1363,9 +1393,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
                 TRY(gemm(m, in, D, (const uint8_t*)L.front + (size_t)L.off_up * D * m.wsize, m.proj.p + L.off_up, nf, T, L.n_front - L.off_up, D, EPI_NONE, 1.f, &f));
                 fk.kskip = ExpertSkip{used, L.back_ff, F, Ex};
             }
-            TRY(launch_dep(moe_act_kernel, dim3(grid_for((size_t)T * L.ff_width)), dim3(256), 0, (const float*)m.proj.p, nf, L.off_up, Ex, F, (const float*)wdense, L.off_sh,
-                           d.shared_ff, L.off_sg, ffo, KB, d.expert_form, T));
-            LAUNCHED();
+            TRY(moe_act(L, nf, wdense, ffo, KB));
         }
         return gemm(m, m.act.p, KB, L.back, m.x.p, D, T, D, KB, EPI_ADD, 1.f, &fk);
     };
@@ -1429,7 +1457,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             s.rot_half = L.d.rot_half; s.v_norm = L.d.v_norm; s.bias = L.qkv_bias.p; s.temp = L.temp;
             s.qgain = L.qgain; s.kgain = L.kgain; s.rot_amp = L.d.rot_amp > 0.f ? L.d.rot_amp : 1.f; s.pb = L.pb;
             if (L.d.qk_norm == TI_SEQ_QK_NORM_WHOLE) TRY(launch_dep(attn_prepare_whole_kernel, dim3(T), dim3(256), 0, m.proj.p, sm, s, L.qnorm, L.knorm, R.k_pool.p, R.v_pool.p));
-            else TRY(launch_dep(attn_prepare_kernel, dim3(T), dim3(128), 0, m.proj.p, sm, s, L.inv_freq.p, R.k_pool.p, R.v_pool.p));
+            else TRY(launch_dep(attn_prepare_kernel, dim3(T), dim3(prepare_threads), 0, m.proj.p, sm, s, L.inv_freq.p, R.k_pool.p, R.v_pool.p));
             LAUNCHED();
             if (L.mix_HP > 0) TRY(mixed_attention(s, L, m.proj.p, R.k_pool.p, R.v_pool.p, m.att.p));
             else TRY(attention(s, m.proj.p, R.k_pool.p, R.v_pool.p, m.att.p));
@@ -1591,9 +1619,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
                     TRY(route(r, rper, nfw, L, wdense, idw_buf, nullptr));
                 }
                 if (L.ff_width > 0) {
-                    TRY(launch_dep(moe_act_kernel, dim3(grid_for((size_t)T * L.ff_width)), dim3(256), 0, (const float*)m.proj.p, nfw, L.off_up, Ex, F, (const float*)wdense, L.off_sh,
-                                   L.d.shared_ff, L.off_sg, m.act.p, L.ff_width, L.d.expert_form, T));
-                    LAUNCHED();
+                    TRY(moe_act(L, nfw, wdense, m.act.p, L.ff_width));
                 }
                 if (sparse) {
                     Fuse f;
@@ -1712,6 +1738,20 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
     std::vector<int*> at;            // where the offset of every front part goes (null: nowhere)
     std::vector<std::string> used;   // tensors that live on inside the two matrices
     const auto add = [&](const std::string& nm, int* off) { fr.push_back(T(nm)); at.push_back(off); used.push_back(nm); };
+    std::vector<std::unique_ptr<Tensor>> zeros;   // rows of zeros that let the part behind them start on a multiple of four columns
+    const auto align = [&]() -> int {
+        int64_t rows = 0;
+        for (const Tensor* t : fr) rows += t->shape[0];
+        if (rows % 4 == 0) return 0;
+        zeros.push_back(std::make_unique<Tensor>());
+        Tensor& z = *zeros.back();
+        z.shape = {4 - rows % 4, (int64_t)m.d.width};
+        TRY(z.data.alloc(z.count() * m.wsize));
+        CK(cudaMemset(z.data.p, 0, z.data.n));
+        fr.push_back(&z);
+        at.push_back(nullptr);
+        return 0;
+    };
     const auto add_back = [&](const std::string& nm) { bk.push_back(T(nm)); used.push_back(nm); };
     int width = 0;
     const std::string pl = p + mix_prefix(d, false), pr = p + mix_prefix(d, true);
@@ -1732,6 +1772,7 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
     if (d.ff > 0) {
         L.back_ff = width;
         if (d.ff_kind == TI_SEQ_FF_GLU) {
+            TRY(align());
             add(p + "mlp.gate", &L.off_up); add(p + "mlp.up", nullptr);
             add_back(p + "mlp.down");
             L.ff_width = d.ff;
@@ -1743,6 +1784,7 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
                 else add(q + "up", off);
                 add_back(q + "down");
             };
+            TRY(align());
             for (int e = 0; e < d.experts; ++e) expert(p + "mlp.e" + std::to_string(e) + ".", e == 0 ? &L.off_up : nullptr);
             if (d.shared_ff > 0) expert(p + "mlp.shared.", &L.off_sh);
             L.ff_width = d.experts * d.ff + d.shared_ff;

@@ -180,38 +180,48 @@ __global__ void moe_route_kernel(const float* proj, int ld, int off, RouteShape 
 // Expert e's [gate | up] block starts at proj column off_gu + e * 2F, the shared expert's at off_sh.  form EXPERT_RELU2: an expert has no
 // gate, its inner value is max(up, 0)^2 and its block is F wide.  lda = row stride of act.
 enum { EXPERT_GATED = 0, EXPERT_RELU2 = 1 };
+// One row a block (blockIdx.y: column groups); V = 4: four neighbouring columns a thread (F, Fs, the offsets and strides in fours).
+template <int V>
 __global__ void moe_act_kernel(const float* proj, int ld, int off_gu, int E, int F, const float* wdense, int off_sh, int Fs, int off_sg, float* act, int lda, int form, int T) {
     pdl_launch_dependents();
     pdl_wait_prior_grid();
     const int W = E * F + Fs;
-    const size_t n = (size_t)T * W;
-    for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
-        const size_t t = i / W;
-        const int x = (int)(i % W);
-        const float* row = proj + t * ld;
-        float v = 0.f;
-        if (x < E * F) {
-            const int e = x / F, c = x % F;
-            const float w = wdense[t * E + e];
-            if (w != 0.f && form == EXPERT_RELU2) {
-                const float u = fmaxf(row[off_gu + (size_t)e * F + c], 0.f);
-                v = w * u * u;
-            } else if (w != 0.f) {
-                const float g = row[off_gu + (size_t)e * 2 * F + c], u = row[off_gu + (size_t)e * 2 * F + F + c];
-                v = w * (g / (1.f + expf(-g))) * u;
-            }
-        } else {
-            const int c = x - E * F;
-            if (form == EXPERT_RELU2) {
-                const float u = fmaxf(row[off_sh + c], 0.f);
-                v = u * u;
+    const size_t t = blockIdx.x;
+    const float* row = proj + t * ld;
+    const float* wr = wdense + t * E;
+    for (int x = (blockIdx.y * blockDim.x + threadIdx.x) * V; x < W; x += gridDim.y * blockDim.x * V) {
+        const bool routed = x < E * F;
+        const int e = routed ? x / F : 0, c = routed ? x - e * F : x - E * F, wide = routed ? F : Fs;
+        const float* g = row + (routed ? off_gu + (size_t)e * (form == EXPERT_RELU2 ? F : 2 * F) : (size_t)off_sh) + c;
+        const float w = routed ? wr[e] : off_sg >= 0 ? 1.f / (1.f + expf(-row[off_sg])) : 1.f;
+        float v[V];
+#pragma unroll
+        for (int q = 0; q < V; ++q) v[q] = 0.f;
+        if (w != 0.f) {   // (an expert the row did not choose is not read)
+            float a[V], b[V];
+            if constexpr (V == 4) {
+                const float4 p = *reinterpret_cast<const float4*>(g);
+                a[0] = p.x; a[1] = p.y; a[2] = p.z; a[3] = p.w;
+                if (form != EXPERT_RELU2) {
+                    const float4 u = *reinterpret_cast<const float4*>(g + wide);
+                    b[0] = u.x; b[1] = u.y; b[2] = u.z; b[3] = u.w;
+                }
             } else {
-                const float g = row[off_sh + c], u = row[off_sh + Fs + c];
-                v = (g / (1.f + expf(-g))) * u;
+                a[0] = g[0];
+                if (form != EXPERT_RELU2) b[0] = g[wide];
             }
-            if (off_sg >= 0) v /= 1.f + expf(-row[off_sg]);
+#pragma unroll
+            for (int q = 0; q < V; ++q) {
+                if (form == EXPERT_RELU2) {
+                    const float u = fmaxf(a[q], 0.f);
+                    v[q] = w * u * u;
+                } else {
+                    v[q] = w * (a[q] / (1.f + expf(-a[q]))) * b[q];
+                }
+            }
         }
-        act[t * lda + x] = v;
+        if constexpr (V == 4) *reinterpret_cast<float4*>(act + t * lda + x) = make_float4(v[0], v[1], v[2], v[3]);
+        else act[t * lda + x] = v[0];
     }
 }
 

@@ -57,15 +57,14 @@ template <int V> __device__ __forceinline__ void conv_store(float* p, const floa
     else *p = v[0];
 }
 // V = 4: a thread takes four neighbouring coordinates with 16-byte loads and stores (D in whole fours); V = 1: one coordinate at a time.
+// (row t; the threads first, first + step, ... take the coordinates)
 template <int V>
-__global__ void short_conv_kernel(const float* x, ConvForm f, StepMeta m, int D, int taps, const float* w, float* state, float* y) {
-    pdl_launch_dependents();
-    pdl_wait_prior_grid();
+__device__ __forceinline__ void short_conv_row(int t, int first, int step, const float* x, const ConvForm& f, const StepMeta& m, int D, int taps, const float* w, float* state, float* y) {
     constexpr int CH = V == 4 ? 4 : 8;   // taps whose inputs are requested together
-    const int t = blockIdx.x, e = m.row_ent[t], i = t - m.ent_row0[e], pos0 = m.ent_pos0[e];
+    const int e = m.row_ent[t], i = t - m.ent_row0[e], pos0 = m.ent_pos0[e];
     float* st = state + (size_t)m.ent_slot[e] * (taps - 1) * D;
     const bool alone = m.ent_row0[e + 1] - m.ent_row0[e] == 1;
-    for (int d = (blockIdx.y * blockDim.x + threadIdx.x) * V; d < D; d += gridDim.y * blockDim.x * V) {
+    for (int d = first * V; d < D; d += step * V) {
         float xv[V], acc[V];
         conv_load<V>(x + (size_t)t * f.ldx + d, xv);
         conv_start<V>(f, d, xv, acc);
@@ -103,6 +102,12 @@ __global__ void short_conv_kernel(const float* x, ConvForm f, StepMeta m, int D,
             if (taps > 1) conv_store<V>(st + (size_t)(taps - 2) * D + d, xv);
         }
     }
+}
+template <int V>
+__global__ void short_conv_kernel(const float* x, ConvForm f, StepMeta m, int D, int taps, const float* w, float* state, float* y) {
+    pdl_launch_dependents();
+    pdl_wait_prior_grid();
+    short_conv_row<V>(blockIdx.x, blockIdx.y * blockDim.x + threadIdx.x, gridDim.y * blockDim.x, x, f, m, D, taps, w, state, y);
 }
 // Many rows (prompt portions): a block takes R consecutive rows and a thread four neighbouring coordinates (D in whole fours), whose
 // weights (taps <= KT) it reads ONCE and keeps in registers, the tap that reaches `back` rows back in entry KT - 1 - back.

@@ -488,20 +488,23 @@ __global__ void __launch_bounds__(kRowGemvThreads) gemv_heads_rows_kernel(const 
 constexpr int kMmaCols = 16;
 // Routed experts on few rows: the stacked matrices hold every expert's rows, the step's tokens chose only some.  Output columns
 // (front product) or k (down product) in [first + e * group, first + (e + 1) * group) belong to expert e < count; a column tile or
-// k chunk whose experts were chosen by no row is not read (its outputs are never used / its activations are exactly zero).
+// k chunk whose experts were chosen by no row is not read (its outputs are never used / its activations are exactly zero).  The k chunks
+// that stay are listed first: only their part of the rows is staged, and the warps deal the list out among themselves.  Column tiles in
+// use are dealt out to the blocks the same way when every expert has whole tiles.
 struct ExpertSkip {
     const int* used;   // [count] 0 / 1; null: nothing is skipped
     int first, group, count;
 };
-__device__ __forceinline__ bool expert_range_used(const ExpertSkip& s, int lo, int hi) {   // does [lo, hi] touch a used expert or leave the experts' range?
-    if (!s.used) return true;
+constexpr int kSkipMaxExperts = 1024;
+// does [lo, hi] touch a used expert (bit e of `bits`) or leave the experts' range?
+__device__ __forceinline__ bool expert_range_used(const ExpertSkip& s, const uint32_t* bits, int lo, int hi) {
     if (lo < s.first) return true;
     const int e0 = (lo - s.first) / s.group, e1 = (hi - s.first) / s.group;
     for (int e = e0; e <= e1; ++e)
-        if (e >= s.count || s.used[e]) return true;
+        if (e >= s.count || (bits[e >> 5] >> (e & 31) & 1u)) return true;
     return false;
 }
-__host__ __device__ inline size_t gemv_mma_smem_bytes(int M, int K) { return (size_t)M * (K + 32) * 2 + 8 * 2 * 128 * sizeof(float); }
+__host__ __device__ inline size_t gemv_mma_smem_bytes(int M, int K) { return (size_t)M * (K + 32) * 2 + 8 * 2 * 128 * sizeof(float) + (size_t)(K / 32) * 2 /* k chunk list */; }
 __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
     asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
@@ -515,8 +518,17 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
     const int Kp = K + 32;
     __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smraw);                       // [M][Kp]
     float* red = reinterpret_cast<float*>(smraw + (size_t)M * Kp * 2);                  // [8 warps][2][128]
+    uint16_t* klist = reinterpret_cast<uint16_t*>(red + 8 * 2 * 128);                   // [K / 32] chunks in use, ascending
     __shared__ float rss[kRowGemvMaxRows][8];
+    __shared__ int kcount[8];
+    __shared__ uint32_t ubits[kSkipMaxExperts / 32];   // experts some row chose
+    __shared__ uint16_t ulist[kSkipMaxExperts];        // the same as a list
+    __shared__ int ucount;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const bool skip = kskip.used && !norm_gain && kskip.count <= kSkipMaxExperts;   // (a norm in front needs the whole row)
+    const bool nskips = !GLU && nskip.used && nskip.count <= kSkipMaxExperts;
+    const int per_expert = nskip.group / kMmaCols;
+    const bool dealt = nskips && nskip.first == 0 && nskip.group % kMmaCols == 0;   // every expert's columns are whole tiles
     const int NC = K / 32, c_begin = warp * NC / 8, c_end = (warp + 1) * NC / 8;   // this warp's 32-k chunks
     // column tiles: the plain columns in sixteens, then (GLU) the gated ones
     const int plain_cols = GLU ? glu.first : N, plain_tiles = (plain_cols + kMmaCols - 1) / kMmaCols;
@@ -526,13 +538,55 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
         const bool gated = GLU && (int)blockIdx.x >= plain_tiles;
         const int n = gated ? min(plain_cols + ((int)blockIdx.x - plain_tiles) * kMmaCols + (lane & 15), N - 1) : min((int)blockIdx.x * kMmaCols + (lane & 15), plain_cols - 1);
         const char* w = reinterpret_cast<const char*>(W + (size_t)n * K + (size_t)c_begin * 32);
-        const size_t bytes = (size_t)(c_end - c_begin) * 64;
+        // (what the step's rows chose is not known yet: nothing of the experts is asked for)
+        const bool expert_tile = nskips && (int)blockIdx.x * kMmaCols >= nskip.first && (int)blockIdx.x * kMmaCols < nskip.first + nskip.group * nskip.count;
+        const int p_end = skip ? min(c_end, kskip.first / 32) : c_end;
+        const size_t bytes = p_end > c_begin && !expert_tile ? (size_t)(p_end - c_begin) * 64 : 0;
         for (size_t o = (size_t)(lane >> 4) * 128; o < bytes; o += 256) {
             asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
             if (gated) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o + (size_t)glu.ff * K * 2));
         }
     }
     pdl_wait_prior_grid();
+    if (skip || nskips) {
+        const ExpertSkip& s = skip ? kskip : nskip;
+        for (int e0 = 32 * warp; e0 < s.count; e0 += 256) {
+            const uint32_t b = __ballot_sync(0xFFFFFFFFu, e0 + lane < s.count && s.used[e0 + lane]);
+            if (lane == 0) ubits[e0 >> 5] = b;
+        }
+        __syncthreads();
+        if (dealt && warp == 0) {
+            int n = 0;
+            for (int e0 = 0; e0 < s.count; e0 += 32) {
+                const uint32_t b = ubits[e0 >> 5];
+                if (b >> lane & 1u) ulist[n + __popc(b & ((1u << lane) - 1u))] = (uint16_t)(e0 + lane);
+                n += __popc(b);
+            }
+            if (lane == 0) ucount = n;
+        }
+        __syncthreads();
+    }
+    const int used_tiles = dealt ? ucount * per_expert : 0, turns = dealt ? used_tiles + tiles - nskip.count * per_expert : tiles;
+    int NA = NC;   // chunks in use
+    if (skip) {    // every warp lists its share of the chunks behind those of the warps before it
+        int n = 0;
+        for (int c0 = c_begin; c0 < c_end; c0 += 32) n += __popc(__ballot_sync(0xFFFFFFFFu, c0 + lane < c_end && expert_range_used(kskip, ubits, (c0 + lane) * 32, (c0 + lane) * 32 + 31)));
+        if (lane == 0) kcount[warp] = n;
+        __syncthreads();
+        int at = 0;
+        NA = 0;
+        for (int w = 0; w < 8; ++w) {
+            if (w < warp) at += kcount[w];
+            NA += kcount[w];
+        }
+        for (int c0 = c_begin; c0 < c_end; c0 += 32) {
+            const bool on = c0 + lane < c_end && expert_range_used(kskip, ubits, (c0 + lane) * 32, (c0 + lane) * 32 + 31);
+            const uint32_t mask = __ballot_sync(0xFFFFFFFFu, on);
+            if (on) klist[at + __popc(mask & ((1u << lane) - 1u))] = (uint16_t)(c0 + lane);
+            at += __popc(mask);
+        }
+        __syncthreads();
+    }
     // rows -> shared memory as bf16, behind the scalar-gain RMS norm when one is fused in front; 16-byte loads, several in flight
     // (every block stages all rows, so this prologue is on the critical path of the launch)
     const bool v4 = (lda % 4 == 0) && ((reinterpret_cast<uintptr_t>(A) & 15) == 0);   // K is a multiple of 32
@@ -564,7 +618,21 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
         const bool gv = norm_gain && gvec;
         const float* ar = A + (size_t)r * lda;
         __nv_bfloat16* xr = xs + (size_t)r * Kp;
-        if (v4) {
+        if (skip) {
+            if (v4) {
+#pragma unroll 4
+                for (int i = threadIdx.x * 4; i < NA * 32; i += 1024) {
+                    const float4 v = *reinterpret_cast<const float4*>(ar + (int)klist[i >> 5] * 32 + (i & 31));
+                    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+                    uint2 pk;
+                    pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+                    pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+                    *reinterpret_cast<uint2*>(xr + i) = pk;
+                }
+            } else {
+                for (int i = threadIdx.x; i < NA * 32; i += 256) xr[i] = __float2bfloat16_rn(ar[(int)klist[i >> 5] * 32 + (i & 31)]);
+            }
+        } else if (v4) {
 #pragma unroll 4
             for (int k = threadIdx.x * 4; k < K; k += 1024) {
                 float4 v = *reinterpret_cast<const float4*>(ar + k);
@@ -584,26 +652,25 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
     }
     __syncthreads();
     constexpr int UNR = GLU ? 4 : 8;   // chunks whose weight loads are in flight together (16-byte loads a lane: 2 or 4 a chunk)
-    // when chunks may be skipped the warps take the chunks in turn (every warp gets its share of every expert) instead of one range each
-    const int cstep = kskip.used ? 8 : 1, c0 = kskip.used ? warp : c_begin, c1 = kskip.used ? NC : c_end;
-    for (int tile = blockIdx.x; tile < tiles; tile += gridDim.x) {
+    // positions in the chunk list (the chunks themselves when nothing is skipped): a range for every warp
+    const int c0 = skip ? warp * NA / 8 : c_begin, c1 = skip ? (warp + 1) * NA / 8 : c_end;
+    for (int turn = blockIdx.x; turn < turns; turn += gridDim.x) {
+        const int tile = !dealt ? turn : turn < used_tiles ? (int)ulist[turn / per_expert] * per_expert + turn % per_expert : nskip.count * per_expert + turn - used_tiles;
         const bool gated = GLU && tile >= plain_tiles;
         const int n0 = gated ? plain_cols + (tile - plain_tiles) * kMmaCols : tile * kMmaCols, end = gated ? N : plain_cols;
-        if (!expert_range_used(nskip, n0, min(n0 + kMmaCols, end) - 1)) continue;   // (uniform over the block)
+        if (nskips && !dealt && !expert_range_used(nskip, ubits, n0, min(n0 + kMmaCols, end) - 1)) continue;   // (uniform over the block)
         float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
         const __nv_bfloat16* w0 = W + (size_t)min(n0 + g, end - 1) * K + 8 * t;
         const __nv_bfloat16* w1 = W + (size_t)min(n0 + g + 8, end - 1) * K + 8 * t;
         const size_t up = (size_t)glu.ff * K;
         const __nv_bfloat16* xr = xs + (size_t)g * Kp + 8 * t;
-        for (int c = c0; c < c1; c += UNR * cstep) {
+        for (int c = c0; c < c1; c += UNR) {
             uint4 ra[UNR], rb[UNR], ua[GLU ? UNR : 1], ub[GLU ? UNR : 1];
-            bool on[UNR];
 #pragma unroll
             for (int q = 0; q < UNR; ++q) {
-                const int cc = c + q * cstep;
-                on[q] = cc < c1 && expert_range_used(kskip, cc * 32, cc * 32 + 31);
-                if (on[q]) {
-                    const int k = cc * 32;
+                const int cc = c + q;
+                if (cc < c1) {
+                    const int k = (skip ? (int)klist[cc] : cc) * 32;
                     ra[q] = *reinterpret_cast<const uint4*>(w0 + k);
                     rb[q] = *reinterpret_cast<const uint4*>(w1 + k);
                     if (gated) {
@@ -614,9 +681,9 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
             }
 #pragma unroll
             for (int q = 0; q < UNR; ++q)
-                if (on[q]) {
+                if (c + q < c1) {
                     uint4 x = make_uint4(0u, 0u, 0u, 0u);
-                    if (g < M) x = *reinterpret_cast<const uint4*>(xr + (c + q * cstep) * 32);
+                    if (g < M) x = *reinterpret_cast<const uint4*>(xr + (c + q) * 32);
                     mma_bf16_16816(acc, ra[q].x, rb[q].x, ra[q].y, rb[q].y, x.x, x.y);
                     mma_bf16_16816(acc, ra[q].z, rb[q].z, ra[q].w, rb[q].w, x.z, x.w);
                     if (gated) {
@@ -774,10 +841,7 @@ __device__ __forceinline__ float attn_finish_factor(const AttnShape& s, int h, f
 // Biases, the per-head norm with a gain, rotation of q and k, unit RMS per head, the per-head query factor, unit-RMS values and the
 // cache append: one block per row.  q is rewritten in place; k and v go to the row's page.  inv_freq[rot_dims / 2] holds the (scaled) frequencies; the angle is
 // position * frequency in fp32.  Pair i of the rotated coordinates is (2 i, 2 i + 1) or, with rot_half, (i, i + rot_dims / 2).
-__global__ void attn_prepare_kernel(float* qkvg, StepMeta m, AttnShape s, const float* inv_freq, float* k_pool, float* v_pool) {
-    pdl_launch_dependents();   // the kernel behind this one may be scheduled (and a few-row product may fetch its weights) ...
-    pdl_wait_prior_grid();     // ... while this one waits here for the kernel before it, when it was launched ahead of its end
-    const int t = blockIdx.x;
+__device__ __forceinline__ void attn_prepare_row(int t, float* qkvg, const StepMeta& m, const AttnShape& s, const float* inv_freq, float* k_pool, float* v_pool) {
     const int pos = m.row_pos[t];
     const int slot = m.ent_slot[m.row_ent[t]];
     const int page = m.page_table[(size_t)slot * m.table_stride + pos / kPageTokens];
@@ -849,6 +913,12 @@ __global__ void attn_prepare_kernel(float* qkvg, StepMeta m, AttnShape s, const 
     } else {
         for (int i = threadIdx.x; i < s.kv_heads * s.vdim; i += blockDim.x) vd[i] = vs[i] + (vb ? vb[i] : 0.f);
     }
+}
+constexpr int kPrepareFewThreads = 512;   // few rows: more of a row's heads at once
+__global__ void __launch_bounds__(kPrepareFewThreads) attn_prepare_kernel(float* qkvg, StepMeta m, AttnShape s, const float* inv_freq, float* k_pool, float* v_pool) {
+    pdl_launch_dependents();   // the kernel behind this one may be scheduled (and a few-row product may fetch its weights) ...
+    pdl_wait_prior_grid();     // ... while this one waits here for the kernel before it, when it was launched ahead of its end
+    attn_prepare_row(blockIdx.x, qkvg, m, s, inv_freq, k_pool, v_pool);
 }
 
 // Softmax attention of one (row, query head) over the keys its window allows, read from the paged cache: 4 warps share the

@@ -8,12 +8,23 @@
 //
 // ssm_scan_kernel runs the recurrence token by token; the other kernels finish a row.  Everything is fp32 in both compute modes.
 #pragma once
+#include "seq_headmix.cuh"
 #include "seq_kernels.cuh"
 
 namespace tib {
 namespace seq {
 
 __device__ __forceinline__ float softplus_f32(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+// Few rows, attention and a state-space mixer side by side: the attention's preparation of row blockIdx.x (blockIdx.y 0) and the
+// convolution in front of the state-space recurrence (the other blockIdx.y) in one launch -- both only read the front product.
+__global__ void __launch_bounds__(kPrepareFewThreads) attn_prepare_conv_kernel(float* qkvg, StepMeta m, AttnShape s, const float* inv_freq, float* k_pool, float* v_pool,
+                                                                              const float* x, ConvForm f, int channels, int taps, const float* w, float* state, float* y) {
+    pdl_launch_dependents();
+    pdl_wait_prior_grid();
+    if (blockIdx.y == 0) attn_prepare_row(blockIdx.x, qkvg, m, s, inv_freq, k_pool, v_pool);
+    else short_conv_row<1>(blockIdx.x, (blockIdx.y - 1) * blockDim.x + threadIdx.x, (gridDim.y - 1) * blockDim.x, x, f, m, channels, taps, w, state, y);
+}
 
 struct SsmArgs {
     const float* xbc;             // [T][ld]: x [heads * dv], B [groups * N], C [groups * N] behind the convolution
