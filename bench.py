@@ -284,7 +284,9 @@ def main():
                     help="with --arch-compare: the design that is measured.  Tudasun (gated linear recurrences, latent attention, routed experts; bf16) "
                          "is put next to the Binusun hybrid on the same engine at equal width and depth; Gulazen (capped head-mixed window attention "
                          "behind a short convolution, xIELU / routed feed-forward; bf16) and Zopipel (hyper-connections, attention with a zero sink and "
-                         "windowed latent attention behind short convolutions; bf16) next to seven Binusun attention layers of the same sizes")
+                         "windowed latent attention behind short convolutions; bf16) next to seven Binusun attention layers of the same sizes; Sebudra (one norm for "
+                         "both sublayers, state space beside attention, gla, sigmoid-weighted attention, routed experts; bf16) next to Tudasun and to the "
+                         "Binusun attention layers")
     ap.add_argument("--layers", type=int, default=0, help="debug: truncate depth (the number is then NOT a bench value)")
     args = ap.parse_args()
 

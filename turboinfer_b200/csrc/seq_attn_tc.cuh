@@ -120,11 +120,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
         const int qp0 = pos0 + r0, qp1 = pos0 + r1;
         const int w = s.window > 0 ? s.window : 0x3FFFFFFF;
         float mx0 = -INFINITY, mx1 = -INFINITY;
-        if (s.softcap > 0.f) {   // (a multiplication by the scale commutes with nothing here: the cap takes the scaled score)
+        if (s.softcap > 0.f) {
+            const float pre = s.scale / s.softcap;
 #pragma unroll
             for (int j = 0; j < kTcKT / 8; ++j)
 #pragma unroll
-                for (int i = 0; i < 4; ++i) sc[j][i] = s.softcap * tanhf(sc[j][i] * s.scale / s.softcap);
+                for (int i = 0; i < 4; ++i) sc[j][i] = s.softcap * tanhf(sc[j][i] * pre);
         } else {
 #pragma unroll
             for (int j = 0; j < kTcKT / 8; ++j)

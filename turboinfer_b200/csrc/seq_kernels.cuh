@@ -821,7 +821,7 @@ __device__ __forceinline__ float attn_score(const AttnShape& s, float dot) {
     const float v = dot * s.scale;
     return s.softcap > 0.f ? s.softcap * tanhf(v / s.softcap) : v;
 }
-__device__ __forceinline__ float attn_sigmoid(float score, float pb) { return 1.f / (1.f + expf(-(score + pb))); }
+__device__ __forceinline__ float attn_sigmoid(float score, float pb) { return __fdividef(1.f, 1.f + expf(-(score + pb))); }
 // sigmoid output gate of (row t, head h), 1 without a gate
 __device__ __forceinline__ float attn_gate(const AttnShape& s, const float* qkvg, int t, int h) {
     if (!s.out_gate) return 1.f;
