@@ -148,28 +148,28 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
 #pragma unroll
                 for (int i = 0; i < 4; ++i) sc[j][i] = sc[j][i] == -INFINITY ? 0.f : attn_sigmoid(sc[j][i], pb);
         } else {
-        mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1)); mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
-        mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1)); mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
-        const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
-        float rs0 = 0.f, rs1 = 0.f;
+            mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 1)); mx0 = fmaxf(mx0, __shfl_xor_sync(0xffffffffu, mx0, 2));
+            mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 1)); mx1 = fmaxf(mx1, __shfl_xor_sync(0xffffffffu, mx1, 2));
+            const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
+            float rs0 = 0.f, rs1 = 0.f;
 #pragma unroll
-        for (int j = 0; j < kTcKT / 8; ++j) {
-            sc[j][0] = mn0 == -INFINITY ? 0.f : expf(sc[j][0] - mn0);
-            sc[j][1] = mn0 == -INFINITY ? 0.f : expf(sc[j][1] - mn0);
-            sc[j][2] = mn1 == -INFINITY ? 0.f : expf(sc[j][2] - mn1);
-            sc[j][3] = mn1 == -INFINITY ? 0.f : expf(sc[j][3] - mn1);
-            rs0 += sc[j][0] + sc[j][1];
-            rs1 += sc[j][2] + sc[j][3];
-        }
-        rs0 += __shfl_xor_sync(0xffffffffu, rs0, 1); rs0 += __shfl_xor_sync(0xffffffffu, rs0, 2);
-        rs1 += __shfl_xor_sync(0xffffffffu, rs1, 1); rs1 += __shfl_xor_sync(0xffffffffu, rs1, 2);
-        const float c0 = mn0 == -INFINITY ? 1.f : expf(m0 - mn0), c1 = mn1 == -INFINITY ? 1.f : expf(m1 - mn1);
-        l0 = l0 * c0 + rs0;
-        l1 = l1 * c1 + rs1;
-        m0 = mn0;
-        m1 = mn1;
+            for (int j = 0; j < kTcKT / 8; ++j) {
+                sc[j][0] = mn0 == -INFINITY ? 0.f : expf(sc[j][0] - mn0);
+                sc[j][1] = mn0 == -INFINITY ? 0.f : expf(sc[j][1] - mn0);
+                sc[j][2] = mn1 == -INFINITY ? 0.f : expf(sc[j][2] - mn1);
+                sc[j][3] = mn1 == -INFINITY ? 0.f : expf(sc[j][3] - mn1);
+                rs0 += sc[j][0] + sc[j][1];
+                rs1 += sc[j][2] + sc[j][3];
+            }
+            rs0 += __shfl_xor_sync(0xffffffffu, rs0, 1); rs0 += __shfl_xor_sync(0xffffffffu, rs0, 2);
+            rs1 += __shfl_xor_sync(0xffffffffu, rs1, 1); rs1 += __shfl_xor_sync(0xffffffffu, rs1, 2);
+            const float c0 = mn0 == -INFINITY ? 1.f : expf(m0 - mn0), c1 = mn1 == -INFINITY ? 1.f : expf(m1 - mn1);
+            l0 = l0 * c0 + rs0;
+            l1 = l1 * c1 + rs1;
+            m0 = mn0;
+            m1 = mn1;
 #pragma unroll
-        for (int n = 0; n < NT; ++n) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
+            for (int n = 0; n < NT; ++n) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
         }
 #pragma unroll
         for (int jp = 0; jp < kTcKT / 16; ++jp) {

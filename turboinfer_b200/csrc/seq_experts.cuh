@@ -71,22 +71,22 @@ __global__ void moe_route_kernel(const float* proj, int ld, int off, RouteShape 
             ch[i] = v + correction[i];
         }
     } else {
-    float mx = -INFINITY;
-    for (int i = lane; i < n; i += 32) mx = fmaxf(mx, z[i] + (r.kind == ROUTE_LOGITS ? correction[i] : 0.f));
-    mx = warp_max(mx);
-    float sum = 0.f;
-    for (int i = lane; i < n; i += 32) {
-        const float e = expf(z[i] + (r.kind == ROUTE_LOGITS ? correction[i] : 0.f) - mx);
-        s[i] = e;
-        sum += e;
-    }
-    sum = warp_sum(sum);
-    for (int i = lane; i < n; i += 32) {
-        // by logits: the choice is made among the biased logits, and exp(. - max) of a chosen one over the chosen ones' sum is the
-        // softmax over the chosen logits (the largest logit is always among them, so nothing underflows that matters)
-        if (r.kind == ROUTE_LOGITS) { ch[i] = z[i] + correction[i]; s[i] = fmaxf(s[i], 1e-37f); }
-        else { s[i] = s[i] / sum; ch[i] = s[i] + correction[i]; }
-    }
+        float mx = -INFINITY;
+        for (int i = lane; i < n; i += 32) mx = fmaxf(mx, z[i] + (r.kind == ROUTE_LOGITS ? correction[i] : 0.f));
+        mx = warp_max(mx);
+        float sum = 0.f;
+        for (int i = lane; i < n; i += 32) {
+            const float e = expf(z[i] + (r.kind == ROUTE_LOGITS ? correction[i] : 0.f) - mx);
+            s[i] = e;
+            sum += e;
+        }
+        sum = warp_sum(sum);
+        for (int i = lane; i < n; i += 32) {
+            // by logits: the choice is made among the biased logits, and exp(. - max) of a chosen one over the chosen ones' sum is the
+            // softmax over the chosen logits (the largest logit is always among them, so nothing underflows that matters)
+            if (r.kind == ROUTE_LOGITS) { ch[i] = z[i] + correction[i]; s[i] = fmaxf(s[i], 1e-37f); }
+            else { s[i] = s[i] / sum; ch[i] = s[i] + correction[i]; }
+        }
     }
     __syncwarp();
     const int size = n / r.groups;
