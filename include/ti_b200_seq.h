@@ -29,10 +29,12 @@ enum {
     TI_SEQ_MIXER_GLA = 2,       /* gated linear attention: S <- diag(a) S + k v^T, o = S^T q, a = sigmoid(.)^(1/tau) per key channel */
     TI_SEQ_MIXER_HGRN2 = 3,     /* the same recurrence with the forget gate f as decay and 1 - f as the written key */
     TI_SEQ_MIXER_SSM = 5,       /* state space: S <- exp(-exp(A) dt) S + dt B x^T, y = S^T C + D x, behind a short convolution (the ssm_* numbers below) */
+    TI_SEQ_MIXER_DELTA = 6,     /* gated delta rule: S <- g S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q; short convolutions over q, k and v, unit q and k */
     TI_SEQ_MIXER_LATENT = 4     /* softmax attention whose keys / values are linear images of a cached low-rank vector + one shared rotated key part */
 };
 enum {
     TI_SEQ_ACT_RELU = 0, TI_SEQ_ACT_SILU = 1, TI_SEQ_ACT_GELU_TANH = 2,
+    TI_SEQ_ACT_GELU = 5,          /* 0.5 z (1 + erf(z / sqrt(2))) */
     TI_SEQ_ACT_CLAMPED_SWISH = 4, /* gated form only: g = min(gate h, limit), u = up h cut to [-limit, limit], g sigmoid(1.702 g) (u + 1) */
     TI_SEQ_ACT_XIELU = 3 /* a z^2 + z / 2 for z > 0, b (exp(z) - 1 - z) + z / 2 otherwise; a = softplus(act[0]), b = 1/2 + softplus(act[1]) */
 };
@@ -61,6 +63,11 @@ enum {
     TI_SEQ_NORMS_SHARED = 3  /* one norm a layer ("norm1") whose output both sublayers read: x <- x + mixer(norm(x)) + ff(norm(x)) */
 };
 enum { TI_SEQ_WEIGHTS_SOFTMAX = 0, TI_SEQ_WEIGHTS_SIGMOID = 1 /* a visible key's weight is sigmoid(score + "mix.pb"[head]), not normalised */ };
+enum {
+    TI_SEQ_GATE_NONE = 0,
+    TI_SEQ_GATE_HEAD = 1,   /* one sigmoid a head ("mix.g" [heads][width]) */
+    TI_SEQ_GATE_ELEMENT = 2 /* latent attention: one sigmoid a coordinate of the concatenated heads ("mix.g" [heads * vdim][width]) */
+};
 enum { TI_SEQ_BIAS_NONE = 0, TI_SEQ_BIAS_QKVO = 1, TI_SEQ_BIAS_QKV = 2 };
 enum { TI_SEQ_EXPERT_GATED = 0 /* down(silu(gate h) * up h) */, TI_SEQ_EXPERT_RELU2 = 1 /* down(max(up h, 0)^2) */ };
 enum {
@@ -86,7 +93,7 @@ typedef struct ti_seq_layer_desc {
                                 ramp over the pair index between) */
     float rot_factor, rot_low, rot_high, rot_original;
     int32_t qk_norm;         /* TI_SEQ_QK_NORM_* */
-    int32_t out_gate;        /* 1: head output times sigmoid of a per-head projection of the mixer input */
+    int32_t out_gate;        /* TI_SEQ_GATE_*: the heads' output times sigmoid of a projection of the mixer input */
     float scale;             /* attention score scale */
     int32_t decay_rank;      /* wkv: inner size of the decay's two-matrix projection */
     int32_t ff;              /* feed-forward inner size, 0 = the layer has no feed-forward */
@@ -126,7 +133,7 @@ typedef struct ti_seq_layer_desc {
     int32_t proj_bias;       /* TI_SEQ_BIAS_*: the q, k, v (and output) projections add biases ("mix.q.b", "mix.k.b", "mix.v.b", "mix.o.b") */
     int32_t v_norm;          /* 1: every value head is divided by its RMS (no weight) before it is cached */
     int32_t head_temp;       /* 1: the scaled score of query head h is multiplied by "mix.temp"[h] */
-    /* -- latent attention (`window` and `out_gate` above apply to it as well: "mix.g" [heads][width]) -- */
+    /* -- latent attention (`window`, `chunk` and `out_gate` apply to it as well) -- */
     int32_t q_rank;          /* > 0: queries through a low-rank vector: q = Uq norm(Dq h) ("mix.dq" [q_rank][width], "mix.dq.norm",
                                 "mix.uq" [heads * (dim + rot_dims)][q_rank]); 0: "mix.q" */
     /* -- attention -- */
@@ -144,6 +151,11 @@ typedef struct ti_seq_layer_desc {
     float route_scale;       /* > 0: factor on the routing weights */
     /* -- the whole layer -- */
     int32_t weights_of;      /* 1 + j: the layer has no tensors of its own and uses layer j's, with a cache / state of its own; 0: own tensors */
+    /* -- attention and latent attention: which keys a row sees -- */
+    int32_t chunk;           /* > 0: position i sees j <= i only if i / chunk == j / chunk (whole-number division, positions of the sequence) */
+    /* -- delta rule: heads, kv_heads (q and k heads; head h reads q / k head h / (heads / kv_heads)), dim, vdim above -- */
+    int32_t mix_taps;        /* taps of the convolutions over q, k and v ("mix.q.conv" [kv_heads * dim][taps] ..., silu); the last taps - 1
+                                inputs are sequence state */
 } ti_seq_layer_desc;
 
 typedef struct ti_seq_model_desc {
@@ -156,7 +168,7 @@ typedef struct ti_seq_model_desc {
     int32_t max_tokens;      /* tokens the page pool holds (each sequence's count rounds up to whole pages) */
     int32_t max_seqs;        /* state slots = sequences that can be live at once */
     int32_t norm_kind;       /* TI_SEQ_NORM_* of the norms around the sublayers and in front of the head */
-    float logit_softcap;     /* > 0: logits <- cap * tanh(logits / cap) */
+    float logit_softcap;     /* > 0: logits <- cap * tanh(logits / cap), behind logit_scale */
     int32_t side_dim;        /* > 0: after every layer a per-token side input is added: side.embed[token][layer * side_dim ...] gated by
                                 gelu_tanh(side.gate x), projected back and RMS-normed with a plain per-coordinate weight */
     int32_t norm_place;      /* TI_SEQ_NORMS_* */

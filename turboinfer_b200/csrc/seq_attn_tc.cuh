@@ -2,7 +2,7 @@
 // accuracy: the split-half scheme of the library's prefill attention (prefill.cuh: every fp32 operand x = hi + lo with two fp16
 // halves, 22 mantissa bits, and hi*hi + hi*lo + lo*hi accumulated in fp32 by mma.sync m16n8k16), generalised to
 //   - ragged steps: a block owns up to 128 consecutive rows of ONE sequence (tiles[2 i] = first row, tiles[2 i + 1] = count),
-//   - grouped key/value heads, a sliding window (only the pages the tile's rows can see are visited),
+//   - grouped key/value heads, a sliding window or chunks of positions (only the pages the tile's rows can see are visited),
 //   - the per-head sigmoid output gate and the sink term of the softmax denominator.
 // Scores, softmax and the running sums are fp32.  Query/key and value sizes up to 128 in fours, each padded with zeros to 64 or 128 (the
 // template's sizes; SIZED: they are the layer's own); other shapes use the fp32 tiled kernel.
@@ -56,9 +56,9 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
     for (int n = 0; n < NT; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     const int last_pos = pos0 + M - 1;
-    const int lo = (s.window > 0 && pos0 - s.window + 1 > 0) ? pos0 - s.window + 1 : 0;
+    const int lo = attn_first_key(s, pos0);
     const int warp_first = pos0 + 16 * warp, warp_last = pos0 + min(16 * warp + 15, M - 1);
-    const int warp_lo = (s.window > 0 && warp_first - s.window + 1 > 0) ? warp_first - s.window + 1 : 0;
+    const int warp_lo = attn_first_key(s, warp_first), lo0 = attn_first_key(s, pos0 + r0), lo1 = attn_first_key(s, pos0 + r1);   // (lo0, lo1: of the lane's two rows)
     const uint32_t* qh_row = reinterpret_cast<const uint32_t*>(Qh + (16 * warp + g) * LD) + t;
     const uint32_t* ql_row = reinterpret_cast<const uint32_t*>(Ql + (16 * warp + g) * LD) + t;
     const int lm = lane >> 3, lr = lane & 7;
@@ -118,7 +118,6 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
             }
         }
         const int qp0 = pos0 + r0, qp1 = pos0 + r1;
-        const int w = s.window > 0 ? s.window : 0x3FFFFFFF;
         float mx0 = -INFINITY, mx1 = -INFINITY;
         if (s.softcap > 0.f) {
             const float pre = s.scale / s.softcap;
@@ -135,10 +134,10 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
 #pragma unroll
         for (int j = 0; j < kTcKT / 8; ++j) {
             const int key = t0 + 8 * j + 2 * t;
-            sc[j][0] = (key <= qp0 && key > qp0 - w && r0 < M) ? sc[j][0] : -INFINITY;
-            sc[j][1] = (key + 1 <= qp0 && key + 1 > qp0 - w && r0 < M) ? sc[j][1] : -INFINITY;
-            sc[j][2] = (key <= qp1 && key > qp1 - w && r1 < M) ? sc[j][2] : -INFINITY;
-            sc[j][3] = (key + 1 <= qp1 && key + 1 > qp1 - w && r1 < M) ? sc[j][3] : -INFINITY;
+            sc[j][0] = (key <= qp0 && key >= lo0 && r0 < M) ? sc[j][0] : -INFINITY;
+            sc[j][1] = (key + 1 <= qp0 && key + 1 >= lo0 && r0 < M) ? sc[j][1] : -INFINITY;
+            sc[j][2] = (key <= qp1 && key >= lo1 && r1 < M) ? sc[j][2] : -INFINITY;
+            sc[j][3] = (key + 1 <= qp1 && key + 1 >= lo1 && r1 < M) ? sc[j][3] : -INFINITY;
             mx0 = fmaxf(mx0, fmaxf(sc[j][0], sc[j][1]));
             mx1 = fmaxf(mx1, fmaxf(sc[j][2], sc[j][3]));
         }
@@ -241,7 +240,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_split_kernel
         qr[i] = d < s.dim ? q[d] : 0.f;
         o[i] = 0.f;
     }
-    const int lo = (s.window > 0 && pos - s.window + 1 > 0) ? pos - s.window + 1 : 0;
+    const int lo = attn_first_key(s, pos);
     const int chunk = (pos - lo + 1 + splits - 1) / splits;
     const int j0 = lo + z * chunk, j1 = min(pos, j0 + chunk - 1);
     float mx = s.pb ? 0.f : -INFINITY, l = 0.f;   // (weights without a softmax: the running maximum stays 0)

@@ -25,6 +25,7 @@
 #include "seq_headmix.cuh"
 #include "seq_hyper.cuh"
 #include "seq_ssm.cuh"
+#include "seq_delta.cuh"
 #include "sampling.cuh"
 
 using namespace tib;
@@ -184,7 +185,7 @@ struct LayerW {
     // the mixer has), its width and the column where each part starts (-1: the mixer has no such part)
     const void* front = nullptr;
     DevBuf<uint8_t> front_buf;
-    int n_front = 0, off_q = -1, off_k = -1, off_v = -1, off_g = -1, off_a1 = -1, off_dkv = -1, off_rg1 = -1;
+    int n_front = 0, off_q = -1, off_k = -1, off_v = -1, off_g = -1, off_a1 = -1, off_dkv = -1, off_rg1 = -1, off_b = -1;
     const void *a2 = nullptr, *uv = nullptr;
     DevBuf<uint8_t> ukT;                       // latent attention: per head the transpose of the key up-projection [heads][rank][dim]
     const float *a2b = nullptr, *fb = nullptr, *lower = nullptr, *cnorm = nullptr, *sink = nullptr;
@@ -204,6 +205,7 @@ struct LayerW {
     float act_a = 0.f, act_b = 0.f;
     // attention with biased projections / a per-head score factor / a fixed sink; latent attention with low-rank queries; a second
     // convolution in front of the feed-forward; hyper-connections (index 0: mixer, 1: feed-forward)
+    DevBuf<float> delta_conv;                  // delta rule: the convolutions' weights over q, k and v side by side [channels][taps]
     DevBuf<float> qkv_bias, sink_zero;         // biases of the fused [q | k | v] product side by side; zeros [heads]
     const float *o_bias = nullptr, *temp = nullptr, *canon2 = nullptr, *dqnorm = nullptr;
     const void* uq = nullptr;
@@ -224,8 +226,8 @@ struct Run {
     int layer = 0;
     bool enters_pass = false;   // the looped block's input projection comes right before this run
     DevBuf<float> k_pool, v_pool;          // attention: [pages * 64][G * d], [pages * 64][G * dv]; latent attention: k_pool [pages * 64][rank + rot]
-    DevBuf<float> state, prev;             // wkv: [slots][H][d][d], [slots][D]; gla / hgrn2: state [slots][H][dk][dv]
-    DevBuf<float> ssm_state, ssm_conv;     // state space: [slots][H][N][dv], and its convolution's [slots][taps - 1][channels]
+    DevBuf<float> state, prev;             // wkv: [slots][H][d][d], [slots][D]; gla / hgrn2: state [slots][H][dk][dv]; delta rule: state [slots][H][dv][dk]
+    DevBuf<float> ssm_state, mix_conv;     // state space: [slots][H][N][dv]; its or the delta rule's convolution: [slots][taps - 1][channels]
     int kv_run = -1;                       // latent attention reading another layer's cache: the run that owns it
     DevBuf<float> conv_state;              // short convolution: [slots][taps - 1][D], the last inputs of every sequence
     DevBuf<float> conv_state2;             // the same for the convolution in front of the feed-forward
@@ -307,6 +309,7 @@ void require(Model& m, const std::string& name, std::vector<int64_t> shape, bool
 bool has_ssm(const ti_seq_layer_desc& L) { return L.ssm_heads > 0; }
 int ssm_channels(const ti_seq_layer_desc& L) { return L.ssm_heads * L.ssm_vdim + 2 * L.ssm_groups * L.ssm_state; }
 int ssm_in_rows(const ti_seq_layer_desc& L) { return L.ssm_heads * L.ssm_vdim + ssm_channels(L) + L.ssm_heads; }
+int delta_channels(const ti_seq_layer_desc& L) { return 2 * L.kv_heads * L.dim + L.heads * L.vdim; }   // q, k and v behind the delta rule's convolutions
 // tensors of the two mixers of a layer: "mix." when there is one, "mix.left." / "mix.right." when there are two
 std::string mix_prefix(const ti_seq_layer_desc& L, bool second) {
     if (!has_ssm(L) || L.mixer == TI_SEQ_MIXER_SSM) return "mix.";
@@ -335,12 +338,17 @@ int describe_tensors(Model& m) {
             continue;
         }
         if (L.ssm_heads < 0 || (L.mixer == TI_SEQ_MIXER_SSM && !has_ssm(L))) return fail("layer %d: %d state-space heads", i, L.ssm_heads);
-        if (shared && ((L.mixer != TI_SEQ_MIXER_ATTENTION && L.mixer != TI_SEQ_MIXER_GLA && L.mixer != TI_SEQ_MIXER_SSM) || L.res_gate || L.layer_scale || L.conv_taps || L.out_gate ||
+        const bool dense_ok = L.ff_kind == TI_SEQ_FF_DENSE && L.ff_act != TI_SEQ_ACT_XIELU;
+        if (shared && ((L.mixer != TI_SEQ_MIXER_ATTENTION && L.mixer != TI_SEQ_MIXER_GLA && L.mixer != TI_SEQ_MIXER_SSM && L.mixer != TI_SEQ_MIXER_LATENT && L.mixer != TI_SEQ_MIXER_DELTA) ||
+                       L.res_gate || L.layer_scale || L.conv_taps || (L.out_gate && L.mixer != TI_SEQ_MIXER_LATENT) || (L.mixer == TI_SEQ_MIXER_LATENT && L.kv_from >= 0) ||
                        L.talk || L.keep_first > 0 || L.qk_norm == TI_SEQ_QK_NORM_WHOLE || L.proj_bias == TI_SEQ_BIAS_QKVO || L.identity > 0 ||
-                       (L.ff > 0 && L.ff_kind != TI_SEQ_FF_GLU && L.ff_kind != TI_SEQ_FF_EXPERTS)))
-            return fail("layer %d: one norm for both sublayers is built for attention, gla and state-space mixers without output / residual gates, mixed heads, kept keys, short "
-                        "convolutions, output bias and layer scale, and for the gated and the routed feed-forward", i);
-        if (!shared && (has_ssm(L) || L.mixer == TI_SEQ_MIXER_SSM)) return fail("layer %d: the state-space mixer is built with one norm for both sublayers", i);
+                       (L.ff > 0 && L.ff_kind != TI_SEQ_FF_GLU && L.ff_kind != TI_SEQ_FF_EXPERTS && !dense_ok)))
+            return fail("layer %d: one norm for both sublayers is built for attention, latent attention with a cache of its own, gla, delta-rule and state-space mixers without residual "
+                        "gates, attention output gates, mixed heads, kept keys, short convolutions, output bias and layer scale, and for the gated, the routed and the dense feed-forward", i);
+        if (!shared && (has_ssm(L) || L.mixer == TI_SEQ_MIXER_SSM || L.mixer == TI_SEQ_MIXER_DELTA)) return fail("layer %d: the state-space and the delta-rule mixer are built with one norm for both sublayers", i);
+        if (L.chunk < 0 || (L.chunk > 0 && ((L.mixer != TI_SEQ_MIXER_ATTENTION && L.mixer != TI_SEQ_MIXER_LATENT) || L.talk || L.keep_first > 0)))
+            return fail("layer %d: chunks of %d positions (built for attention and latent attention without mixed heads and kept keys)", i, L.chunk);
+        if (L.out_gate < TI_SEQ_GATE_NONE || L.out_gate > TI_SEQ_GATE_ELEMENT || (L.out_gate == TI_SEQ_GATE_ELEMENT && L.mixer != TI_SEQ_MIXER_LATENT)) return fail("layer %d: output gate %d", i, L.out_gate);
         if (!shared && (L.ff_act == TI_SEQ_ACT_CLAMPED_SWISH || L.expert_form != TI_SEQ_EXPERT_GATED) && L.ff > 0 && L.ff_kind != TI_SEQ_FF_GLU && L.ff_kind != TI_SEQ_FF_EXPERTS)
             return fail("layer %d: activation %d / expert form %d", i, L.ff_act, L.expert_form);
         require(m, p + "norm1", gain_shape, false);
@@ -459,7 +467,7 @@ int describe_tensors(Model& m) {
                 require(m, p + "mix.q", {(int64_t)L.heads * (L.dim + L.rot_dims), D}, true);
             } else return fail("layer %d: query rank %d", i, L.q_rank);
             if (L.window < 0) return fail("layer %d: window %d", i, L.window);
-            if (L.out_gate) require(m, p + "mix.g", {(int64_t)L.heads, D}, true);
+            if (L.out_gate) require(m, p + "mix.g", {(int64_t)L.heads * (L.out_gate == TI_SEQ_GATE_ELEMENT ? L.vdim : 1), D}, true);
             if (L.kv_from < 0) {
                 require(m, p + "mix.dkv", {(int64_t)L.kv_rank + L.rot_dims, D}, true);
                 require(m, p + "mix.dkv.norm", {(int64_t)L.kv_rank}, false);
@@ -468,6 +476,20 @@ int describe_tensors(Model& m) {
             require(m, p + "mix.uv", {(int64_t)L.heads * L.vdim, (int64_t)L.kv_rank}, true);
             if (L.sink == TI_SEQ_SINK_LEARNED) require(m, p + "mix.sink", {(int64_t)L.heads}, false);
             require(m, p + "mix.o", {D, (int64_t)L.heads * L.vdim}, true);
+        } else if (L.mixer == TI_SEQ_MIXER_DELTA) {
+            if (L.heads <= 0 || L.kv_heads <= 0 || L.heads % L.kv_heads || L.dim <= 0 || L.dim > kDeltaMaxKey || L.vdim <= 0 || L.vdim > 65535 * kDeltaCols || L.mix_taps < 1)
+                return fail("layer %d: delta rule with heads %d / %d, sizes %d (at most %d) / %d, taps %d", i, L.heads, L.kv_heads, L.dim, kDeltaMaxKey, L.vdim, L.mix_taps);
+            const int64_t C = (int64_t)L.kv_heads * L.dim, Cv = (int64_t)L.heads * L.vdim;
+            for (const char* s : {"q", "k", "v"}) {
+                const int64_t n = s[0] == 'v' ? Cv : C;
+                require(m, p + "mix." + s, {n, D}, true);
+                require(m, p + "mix." + s + ".conv", {n, (int64_t)L.mix_taps}, false);
+            }
+            for (const char* s : {"b", "a"}) require(m, p + "mix." + s, {(int64_t)L.heads, D}, true);
+            for (const char* s : {"A_log", "dt_bias"}) require(m, p + "mix." + s, {(int64_t)L.heads}, false);
+            require(m, p + "mix.norm", {(int64_t)L.vdim}, false);
+            require(m, p + "mix.g", {Cv, D}, true);
+            require(m, p + "mix.o", {D, Cv}, true);
         } else if (L.mixer != TI_SEQ_MIXER_SSM) {
             return fail("layer %d: unknown mixer %d", i, L.mixer);
         }
@@ -493,7 +515,7 @@ int describe_tensors(Model& m) {
             if (!behind && !front && !shared) require(m, p + "norm2b", gain_shape, false);
             if (behind && L.ff_kind != TI_SEQ_FF_DENSE && L.ff_kind != TI_SEQ_FF_EXPERTS) return fail("layer %d: norms behind the sublayers only are built for the dense and the routed feed-forward", i);
             if (L.ff_kind == TI_SEQ_FF_DENSE) {
-                if (L.ff_act != TI_SEQ_ACT_XIELU && L.ff_act != TI_SEQ_ACT_RELU && L.ff_act != TI_SEQ_ACT_SILU && L.ff_act != TI_SEQ_ACT_GELU_TANH)
+                if (L.ff_act != TI_SEQ_ACT_XIELU && L.ff_act != TI_SEQ_ACT_RELU && L.ff_act != TI_SEQ_ACT_SILU && L.ff_act != TI_SEQ_ACT_GELU_TANH && L.ff_act != TI_SEQ_ACT_GELU)
                     return fail("layer %d: activation %d", i, L.ff_act);
                 require(m, p + "mlp.up", {(int64_t)L.ff, D}, true);
                 require(m, p + "mlp.down", {D, (int64_t)L.ff}, true);
@@ -708,6 +730,7 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
     // bf16 weights with K in whole 32-element chunks: the tensor-core form (a weight byte costs the same for 1 and for 8 rows; rows staged as bf16)
     const bool mma_ok = M <= kRowGemvMaxRows && m.d.mode == TI_SEQ_BF16 && g_use_row_mma && K % 32 == 0 && K >= 256 && (reinterpret_cast<uintptr_t>(W) & 15) == 0 &&
                         mma_bytes <= g_smem_optin;
+    const bool single = fuse && fuse->glu.ff > 0 && fuse->glu.single;   // activation columns without a partner: every path takes them
     const bool plain = !fuse || (!fuse->norm_gain && !fuse->glu.ff);   // (a request to skip unused experts' rows is only a permission)
     if (plain && M > 1 && M <= kRowGemvMaxRows && !mma_ok && !few_rows(M, K) && few_rows(1, K)) {
         const int half = M / 2;
@@ -735,11 +758,14 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
             attr[0].val.programmaticStreamSerializationAllowed = 1;
             cfg.attrs = attr;
             cfg.numAttrs = g_use_pdl ? 1 : 0;
-            if (f.glu.ff > 0)
-                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<true>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
+            if (single)
+                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<COLS_SINGLE>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
+                                      f.gvec, f.nskip, f.kskip));
+            else if (f.glu.ff > 0)
+                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<COLS_PAIR>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
                                       f.gvec, f.nskip, f.kskip));
             else
-                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<false>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
+                CK(cudaLaunchKernelEx(&cfg, gemv_rows_mma_kernel<COLS_PLAIN>, A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, f.norm_gain, f.eps, f.glu,
                                       f.gvec, f.nskip, f.kskip));
             LAUNCHED();
             return 0;
@@ -763,7 +789,7 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
         LAUNCHED();
         return 0;
     }
-    if (!plain) return fail("internal: a fused product was asked for on the many-row path");
+    if (!plain && (!single || fuse->norm_gain)) return fail("internal: a fused product was asked for on the many-row path");
     // prompt-sized products in bf16 mode: tcgen05 (TMA wants 16-byte row pitches and bases)
     if (m.d.mode == TI_SEQ_BF16 && g_use_tc && M > 32 && N >= 64 && K >= 64 && K % 8 == 0 && (reinterpret_cast<uintptr_t>(W) & 15) == 0 && m.abf.p &&
         (size_t)M * K <= m.abf.n) {
@@ -774,26 +800,36 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
         TRY(make_tmap_bf16(&mw, W, (uint64_t)K, (uint64_t)N));
         TcArgs g{};
         g.M = M; g.N = N; g.K = K; g.C = C; g.ldc = ldc; g.epi = epi; g.alpha = alpha; g.beta = beta; g.err = m.err.p;
+        if (single) g.cols = fuse->glu;
         gemm_bf16_tc_kernel<<<dim3((N + kSgBN - 1) / kSgBN, (M + kSgBM - 1) / kSgBM), kSgThreads, kSgSmemBytes, g_stream>>>(ma, mw, g);
         LAUNCHED();
         return 0;
     }
     dim3 grid((N + 63) / 64, (M + 63) / 64);
-    if (m.d.mode == TI_SEQ_BF16) gemm_bf16_kernel<<<grid, 128, 0, g_stream>>>(A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, 0, 0, 0);
-    else gemm_f32_kernel<<<grid, 256, 0, g_stream>>>(A, lda, (const float*)W, C, ldc, M, N, K, epi, alpha, beta, 0, 0, 0);
+    if (m.d.mode == TI_SEQ_BF16) gemm_bf16_kernel<<<grid, 128, 0, g_stream>>>(A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, 0, 0, 0, nullptr, 0);
+    else gemm_f32_kernel<<<grid, 256, 0, g_stream>>>(A, lda, (const float*)W, C, ldc, M, N, K, epi, alpha, beta, 0, 0, 0, nullptr, 0);
     LAUNCHED();
+    if (single) {   // (C has room for these columns too)
+        const GluCols& u = fuse->glu;
+        const float* src = C + u.first;
+        const bool v4 = u.ff % 4 == 0 && ldc % 4 == 0 && u.ld % 4 == 0 && ((reinterpret_cast<uintptr_t>(src) | reinterpret_cast<uintptr_t>(u.out)) & 15) == 0;
+        if (v4) TRY(launch_dep(act_kernel<4>, dim3(grid_for((size_t)M * u.ff / 4)), dim3(256), 0, src, ldc, u.ff, u.act, u.out, u.ld, M));
+        else TRY(launch_dep(act_kernel<1>, dim3(grid_for((size_t)M * u.ff)), dim3(256), 0, src, ldc, u.ff, u.act, u.out, u.ld, M));
+        LAUNCHED();
+    }
     return 0;
 }
 
-// one small product per head: C[r][h * c_stride + n] = sum_k A[r][h * a_stride + k] W[h][n][k]; few rows in one launch, else a product per head
-int gemm_heads(Model& m, const float* A, int lda, int a_stride, const void* W, float* C, int ldc, int c_stride, int heads, int M, int N, int K) {
+// one small product per head: C[r][h * c_stride + n] = sum_k A[r][h * a_stride + k] W[h][n][k] (times sigmoid(gate[r * ldg + h * c_stride + n]))
+int gemm_heads(Model& m, const float* A, int lda, int a_stride, const void* W, float* C, int ldc, int c_stride, int heads, int M, int N, int K, const float* gate = nullptr,
+               int ldg = 0) {
     if (M <= kRowGemvMaxRows && (size_t)M * K * sizeof(float) <= 48 * 1024) {
         const int warps = kRowGemvThreads / 32;
         const dim3 grid(std::max(1, std::min((N + warps - 1) / warps, std::max(1, 4 * g_num_sms / heads))), heads);
         if (m.d.mode == TI_SEQ_BF16)
-            TRY(launch_dep(gemv_heads_rows_kernel<__nv_bfloat16>, grid, dim3(kRowGemvThreads), (size_t)M * K * sizeof(float), A, lda, a_stride, (const __nv_bfloat16*)W, C, ldc, c_stride, M, N, K));
+            TRY(launch_dep(gemv_heads_rows_kernel<__nv_bfloat16>, grid, dim3(kRowGemvThreads), (size_t)M * K * sizeof(float), A, lda, a_stride, (const __nv_bfloat16*)W, C, ldc, c_stride, M, N, K, gate, ldg));
         else
-            TRY(launch_dep(gemv_heads_rows_kernel<float>, grid, dim3(kRowGemvThreads), (size_t)M * K * sizeof(float), A, lda, a_stride, (const float*)W, C, ldc, c_stride, M, N, K));
+            TRY(launch_dep(gemv_heads_rows_kernel<float>, grid, dim3(kRowGemvThreads), (size_t)M * K * sizeof(float), A, lda, a_stride, (const float*)W, C, ldc, c_stride, M, N, K, gate, ldg));
         LAUNCHED();
         return 0;
     }
@@ -801,12 +837,13 @@ int gemm_heads(Model& m, const float* A, int lda, int a_stride, const void* W, f
     const dim3 grid((N + 63) / 64, (M + 63) / 64, heads);
     if (heads <= 65535 && grid.y <= 65535) {
         if (m.d.mode == TI_SEQ_BF16)
-            gemm_bf16_kernel<<<grid, 128, 0, g_stream>>>(A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, EPI_NONE, 1.f, 0.f, (size_t)a_stride, (size_t)N * K, (size_t)c_stride);
+            gemm_bf16_kernel<<<grid, 128, 0, g_stream>>>(A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, EPI_NONE, 1.f, 0.f, (size_t)a_stride, (size_t)N * K, (size_t)c_stride, gate, ldg);
         else
-            gemm_f32_kernel<<<grid, 256, 0, g_stream>>>(A, lda, (const float*)W, C, ldc, M, N, K, EPI_NONE, 1.f, 0.f, (size_t)a_stride, (size_t)N * K, (size_t)c_stride);
+            gemm_f32_kernel<<<grid, 256, 0, g_stream>>>(A, lda, (const float*)W, C, ldc, M, N, K, EPI_NONE, 1.f, 0.f, (size_t)a_stride, (size_t)N * K, (size_t)c_stride, gate, ldg);
         LAUNCHED();
         return 0;
     }
+    if (gate) return fail("internal: %d heads of %d rows exceed a launch", heads, M);
     for (int h = 0; h < heads; ++h)
         TRY(gemm(m, A + (size_t)h * a_stride, lda, (const uint8_t*)W + (size_t)h * N * K * m.wsize, C + (size_t)h * c_stride, ldc, M, N, K));
     return 0;
@@ -1136,15 +1173,24 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         // bf16 mode, head sizes up to 128 in fours: the split-half tensor-core kernel (fp32-accurate); fp32 mode keeps true fp32 arithmetic
         const bool h3_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles128 > 0 && s.dim <= 128 && s.vdim <= 128 && s.dim % 4 == 0 && s.vdim % 4 == 0 && s.v_ld == 0;
         // bf16 mode, a shared key/value head with the values inside the key rows (latent attention), instantiated sizes: tensor cores
-        const bool lat_size = (s.dim == 320 && s.vdim == 256) || (s.dim == 192 && s.vdim == 128) || (s.dim == 160 && s.vdim == 128);
+        const bool lat_size = (s.dim == 320 && s.vdim == 256) || (s.dim == 192 && s.vdim == 128) || (s.dim == 160 && s.vdim == 128) || (s.dim == s.vdim && s.dim % 4 == 0 && s.dim <= 512);
         const bool lat_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles > 0 && v_in_k && (!s.out_gate || s.gate) && !s.qk_norm && lat_size;
         const int* rest = (tiled_ok || h3_ok || lat_ok) ? d_small : nullptr;
         const int n_rest = (tiled_ok || h3_ok || lat_ok) ? n_small : T;
         if (lat_ok) {
             const dim3 grid(n_tiles, s.heads);
-            if (s.dim == 320) latent_attention_h3_kernel<320, 256><<<grid, 256, latent_h3_smem_bytes<320>(), g_stream>>>(q, sm, s, d_tiles, kp, out);
-            else if (s.dim == 192) latent_attention_h3_kernel<192, 128><<<grid, 256, latent_h3_smem_bytes<192>(), g_stream>>>(q, sm, s, d_tiles, kp, out);
-            else latent_attention_h3_kernel<160, 128><<<grid, 256, latent_h3_smem_bytes<160>(), g_stream>>>(q, sm, s, d_tiles, kp, out);
+#define TI_LAT_CASE(K, V, KT, X) latent_attention_h3_kernel<K, V, KT, X><<<grid, 256, latent_h3_smem_bytes<K, KT>(), g_stream>>>(q, sm, s, d_tiles, kp, out)
+            if (s.dim == s.vdim) {   // no rotated part: rows of up to 512 in fours, padded to 128 / 256 / 512
+                if (s.dim == 128) TI_LAT_CASE(128, 128, 64, true);
+                else if (s.dim < 128) TI_LAT_CASE(128, 128, 64, false);
+                else if (s.dim == 256) TI_LAT_CASE(256, 256, 64, true);
+                else if (s.dim < 256) TI_LAT_CASE(256, 256, 64, false);
+                else if (s.dim == 512) TI_LAT_CASE(512, 512, 32, true);
+                else TI_LAT_CASE(512, 512, 32, false);
+            } else if (s.dim == 320) TI_LAT_CASE(320, 256, 64, true);
+            else if (s.dim == 192) TI_LAT_CASE(192, 128, 64, true);
+            else TI_LAT_CASE(160, 128, 64, true);
+#undef TI_LAT_CASE
             LAUNCHED();
         } else if (h3_ok) {
             const dim3 grid(n_tiles128, s.heads);
@@ -1167,7 +1213,8 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         }
         if (n_rest > 0) {
             // single rows: key chunks in parallel (a row-at-a-time walk is one memory round trip a key) unless the rows alone fill the GPU
-            const int span = s.window > 0 ? std::min(s.window, max_pos + 1) : max_pos + 1;
+            int span = s.window > 0 ? std::min(s.window, max_pos + 1) : max_pos + 1;
+            if (s.chunk > 0) span = std::min(span, s.chunk);
             int splits = 1;
             if (span >= 32) splits = std::max(1, std::min({(span + 15) / 16, kAttnMaxSplits, (2 * g_num_sms) / std::max(1, n_rest * s.heads)}));
             if (splits > 1 && m.attn_part.p) {
@@ -1269,6 +1316,50 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         LAUNCHED();
         return 0;
     };
+    auto delta_scan = [&](const DeltaArgs& a) -> int {
+        const dim3 grid(E, a.heads, (a.dv + kDeltaCols - 1) / kDeltaCols);
+        if (a.dk <= 32) TRY(launch_dep(delta_scan_kernel<4, 8>, grid, dim3(128), 0, a, sm));
+        else if (a.dk <= 64) TRY(launch_dep(delta_scan_kernel<8, 8>, grid, dim3(128), 0, a, sm));
+        else if (a.dk <= 128) TRY(launch_dep(delta_scan_kernel<16, 8>, grid, dim3(128), 0, a, sm));
+        else if (a.dk <= 256) TRY(launch_dep(delta_scan_kernel<32, 8>, grid, dim3(128), 0, a, sm));
+        else TRY(launch_dep(delta_scan_kernel<64, 4>, grid, dim3(128), 0, a, sm));
+        LAUNCHED();
+        return 0;
+    };
+    // latent attention behind its front product (in m.proj): the heads' outputs go to rows of `out` (stride ldo)
+    auto latent = [&](LayerW& L, Run& R, float* out, int ldo) -> int {
+        const ti_seq_layer_desc& d = L.d;
+        const int H = d.heads, dr = d.rot_dims, rank = d.kv_rank, kd = rank + dr, nf = L.ld_front;
+        if (d.q_rank > 0) {   // q = Uq norm(Dq h): the norm rides in the second product's prologue when the rows are few
+            const int qr = d.q_rank, nq = H * (d.dim + dr);
+            if (few_rows(T, qr)) {
+                Fuse f;
+                f.norm_gain = L.dqnorm; f.eps = eps; f.gvec = 1;
+                TRY(gemm(m, m.proj.p + L.off_dq, nf, L.uq, m.proj.p + L.off_q, nf, T, nq, qr, EPI_NONE, 1.f, &f));
+            } else {
+                TRY(launch_dep(rmsnorm_kernel, dim3(T), dim3(nt), 0, (const float*)(m.proj.p + L.off_dq), nf, (const int*)nullptr, qr, L.dqnorm, 1, eps, m.lora.p));
+                LAUNCHED();
+                TRY(gemm(m, m.lora.p, qr, L.uq, m.proj.p + L.off_q, nf, T, nq, qr));
+            }
+        }
+        float* pool = R.kv_run >= 0 ? m.runs[R.kv_run].k_pool.p : R.k_pool.p;
+        LatentShape ls{};
+        ls.heads = H; ls.dim = d.dim; ls.rot = dr; ls.rank = rank; ls.ld = nf; ls.off_q = L.off_q; ls.off_dkv = L.off_dkv; ls.eps = eps;
+        ls.rot_half = d.rot_half;
+        TRY(launch_dep(latent_prepare_kernel, dim3(T), dim3(128), 0, (const float*)m.proj.p, sm, ls, (const float*)L.inv_freq.p, L.cnorm, pool, m.aux.p));
+        LAUNCHED();
+        // the key up-projection moves to the query: qabs[t][h][0 .. rank) = Uk_h^T q_h
+        TRY(gemm_heads(m, m.proj.p + L.off_q, nf, d.dim + dr, L.ukT.p, m.aux.p, H * kd, kd, H, T, rank, d.dim));
+        AttnShape s{};
+        s.heads = H; s.kv_heads = 1; s.dim = kd; s.vdim = rank; s.window = d.window; s.chunk = d.chunk; s.rot_dims = 0; s.qk_norm = 0;
+        s.scale = d.scale; s.eps = eps; s.ld = H * kd; s.v_ld = kd; s.sink = L.sink;
+        // (a gate of one number a head commutes with the value up-projection behind the weighted sum; a gate per coordinate rides in its epilogue)
+        const float* g = d.out_gate ? m.proj.p + L.off_g : nullptr;
+        s.out_gate = d.out_gate == TI_SEQ_GATE_HEAD ? 1 : 0; s.gate = s.out_gate ? g : nullptr; s.gate_ld = nf;
+        TRY(attention(s, m.aux.p, pool, pool, m.aux2.p));
+        // ... and the value up-projection behind the weighted sum: out[t][h] = Uv_h (sum_j p_j c_j)
+        return gemm_heads(m, m.aux2.p, H * rank, rank, L.uv, out, ldo, d.vdim, H, T, d.vdim, rank, d.out_gate == TI_SEQ_GATE_ELEMENT ? g : nullptr, nf);
+    };
     auto route_shape = [&](const ti_seq_layer_desc& d) {
         RouteShape r{};
         r.n_real = d.experts; r.n_id = d.identity; r.top = d.top; r.groups = d.groups; r.keep = d.groups_keep;
@@ -1316,13 +1407,17 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             in = m.h.p;
         }
         float* ffo = m.act.p + L.back_ff;   // the feed-forward's part of the back product's rows
-        const bool gated = F > 0 && d.ff_kind == TI_SEQ_FF_GLU, routed = F > 0 && d.ff_kind == TI_SEQ_FF_EXPERTS;
+        const bool gated = F > 0 && d.ff_kind == TI_SEQ_FF_GLU, routed = F > 0 && d.ff_kind == TI_SEQ_FF_EXPERTS, dense = F > 0 && d.ff_kind == TI_SEQ_FF_DENSE;
         const RouteShape rs = routed ? route_shape(d) : RouteShape{};
         const size_t rper = routed ? route_row_bytes(d) : 0;
         const bool sparse = routed && few && bf && d.experts > 0 && T * rper <= 40 * 1024;   // the router first, then only the chosen experts' rows
-        if (few && gated) {
+        if (dense) {   // the activation rides in the product's epilogue, its columns go straight to the back product's rows
+            Fuse f = few ? fn : Fuse{};
+            f.glu = GluCols{F, d.ff_act, L.off_up, 0.f, ffo, KB, 1};
+            TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, L.n_front, D, EPI_NONE, 1.f, &f));
+        } else if (few && gated) {
             Fuse f = fn;
-            f.glu = GluCols{F, d.ff_act, L.off_up, d.ff_limit, ffo, KB};
+            f.glu = GluCols{F, d.ff_act, L.off_up, d.ff_limit, ffo, KB, 0};
             TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, L.off_up + F, D, EPI_NONE, 1.f, &f));
         } else {
             TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, sparse ? L.off_up : L.n_front, D, EPI_NONE, 1.f, few ? &fn : nullptr));
@@ -1336,17 +1431,30 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             s.heads = d.heads; s.kv_heads = d.kv_heads; s.dim = d.dim; s.vdim = d.vdim; s.window = d.window; s.rot_dims = d.rot_dims; s.rot_half = d.rot_half;
             s.qk_norm = d.qk_norm == TI_SEQ_QK_NORM_HEAD ? 1 : 0; s.qgain = L.qgain; s.kgain = L.kgain; s.rot_amp = d.rot_amp > 0.f ? d.rot_amp : 1.f;
             s.scale = d.scale; s.eps = eps; s.ld = nf; s.sink = L.sink; s.softcap = d.softcap; s.v_norm = d.v_norm; s.bias = L.qkv_bias.p; s.temp = L.temp; s.pb = L.pb;
-            s.out_ld = KB; s.out_scale = has_ssm(d) ? d.left_scale : 1.f;
+            s.out_ld = KB; s.out_scale = has_ssm(d) ? d.left_scale : 1.f; s.chunk = d.chunk;
             if (few && has_ssm(d)) {   // with the state-space mixer's convolution in the same launch
                 TRY(launch_dep(attn_prepare_conv_kernel, dim3(T, 1 + (ssm_channels(d) + kPrepareFewThreads - 1) / kPrepareFewThreads), dim3(kPrepareFewThreads), 0, m.proj.p, sm, s,
-                               (const float*)L.inv_freq.p, R.k_pool.p, R.v_pool.p, ssm_u + inner, cf, ssm_channels(d), d.ssm_taps, L.ssm_conv, R.ssm_conv.p, m.aux2.p));
+                               (const float*)L.inv_freq.p, R.k_pool.p, R.v_pool.p, ssm_u + inner, cf, ssm_channels(d), d.ssm_taps, L.ssm_conv, R.mix_conv.p, m.aux2.p));
                 LAUNCHED();
-                TRY(conv_save(ssm_u + inner, nf, ssm_channels(d), d.ssm_taps, R.ssm_conv.p));
+                TRY(conv_save(ssm_u + inner, nf, ssm_channels(d), d.ssm_taps, R.mix_conv.p));
             } else {
                 TRY(launch_dep(attn_prepare_kernel, dim3(T), dim3(prepare_threads), 0, m.proj.p, sm, s, L.inv_freq.p, R.k_pool.p, R.v_pool.p));
                 LAUNCHED();
             }
             TRY(attention(s, m.proj.p, R.k_pool.p, R.v_pool.p, m.act.p));
+        } else if (d.mixer == TI_SEQ_MIXER_LATENT) {
+            TRY(latent(L, R, m.act.p, KB));
+        } else if (d.mixer == TI_SEQ_MIXER_DELTA) {
+            ConvForm df{};
+            df.ldx = nf; df.silu = 1;
+            const int ch = delta_channels(d);
+            TRY(conv(m.proj.p + L.off_q, df, ch, L.delta_conv.p, d.mix_taps, R.mix_conv.p, m.aux2.p));
+            DeltaArgs a{};
+            a.qkv = m.aux2.p; a.ld = ch; a.a = m.proj.p + L.off_a1; a.b = m.proj.p + L.off_b; a.ld_ab = nf; a.dt_bias = L.dt_bias; a.A_log = L.A_log;
+            a.state = R.state.p; a.out = m.act.p; a.ldo = KB; a.heads = d.heads; a.kv_heads = d.kv_heads; a.dk = d.dim; a.dv = d.vdim; a.qscale = 1.f / sqrtf((float)d.dim);
+            TRY(delta_scan(a));
+            TRY(launch_dep(head_rmsnorm_gate_kernel, dim3((T * d.heads + 7) / 8), dim3(256), 0, m.act.p, KB, (const float*)(m.proj.p + L.off_g), nf, 1, L.normw, 0, T, d.heads, d.vdim, eps));
+            LAUNCHED();
         } else if (d.mixer == TI_SEQ_MIXER_GLA) {
             const int H = d.heads, C = H * d.dim;
             TRY(gemm(m, m.proj.p + L.off_a1, nf, L.a2, m.aux.p, C, T, C, d.decay_rank));
@@ -1362,7 +1470,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         if (has_ssm(d)) {
             const int ch = ssm_channels(d);
             const float* u = ssm_u;
-            if (!few || d.mixer == TI_SEQ_MIXER_SSM) TRY(conv(u + inner, cf, ch, L.ssm_conv, d.ssm_taps, R.ssm_conv.p, m.aux2.p));
+            if (!few || d.mixer == TI_SEQ_MIXER_SSM) TRY(conv(u + inner, cf, ch, L.ssm_conv, d.ssm_taps, R.mix_conv.p, m.aux2.p));
             SsmArgs a{};
             a.xbc = m.aux2.p; a.ld = ch; a.dt = u + inner + ch; a.ld_dt = nf; a.dt_bias = L.dt_bias; a.A_log = L.A_log; a.state = R.ssm_state.p;
             a.out = m.act.p + L.back_ssm; a.ldo = KB; a.heads = d.ssm_heads; a.N = d.ssm_state; a.dv = d.ssm_vdim; a.groups = d.ssm_groups;
@@ -1444,7 +1552,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         if (attn) {
             AttnShape s{};
             s.heads = L.d.heads; s.kv_heads = L.d.kv_heads; s.dim = L.d.dim; s.vdim = L.d.vdim;
-            s.window = L.d.window; s.rot_dims = L.d.rot_dims; s.qk_norm = L.d.qk_norm == TI_SEQ_QK_NORM_HEAD ? 1 : 0; s.out_gate = L.d.out_gate;
+            s.window = L.d.window; s.chunk = L.d.chunk; s.rot_dims = L.d.rot_dims; s.qk_norm = L.d.qk_norm == TI_SEQ_QK_NORM_HEAD ? 1 : 0; s.out_gate = L.d.out_gate;
             s.scale = L.d.scale; s.eps = eps; s.ld = L.n_qkvg;
             if (fuse_rows) {
                 Fuse f;
@@ -1525,37 +1633,10 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             LAUNCHED();
             TRY(gemm(m, m.att.p, Cv, L.o, m.mo.p, D, T, D, Cv));
         } else {   // latent attention
-            const int H = L.d.heads, d = L.d.dim, dr = L.d.rot_dims, dv = L.d.vdim, rank = L.d.kv_rank, kd = rank + dr, nf = L.ld_front;
-            TRY(gemm(m, front_in, D, L.front, m.proj.p, nf, T, L.n_front, D, EPI_NONE, 1.f, front_fuse));
-            if (L.d.q_rank > 0) {   // q = Uq norm(Dq h): the norm rides in the second product's prologue when the rows are few
-                const int qr = L.d.q_rank, nq = H * (d + dr);
-                if (few_rows(T, qr)) {
-                    Fuse f;
-                    f.norm_gain = L.dqnorm; f.eps = eps; f.gvec = 1;
-                    TRY(gemm(m, m.proj.p + L.off_dq, nf, L.uq, m.proj.p + L.off_q, nf, T, nq, qr, EPI_NONE, 1.f, &f));
-                } else {
-                    TRY(launch_dep(rmsnorm_kernel, dim3(T), dim3(nt), 0, (const float*)(m.proj.p + L.off_dq), nf, (const int*)nullptr, qr, L.dqnorm, 1, eps, m.lora.p));
-                    LAUNCHED();
-                    TRY(gemm(m, m.lora.p, qr, L.uq, m.proj.p + L.off_q, nf, T, nq, qr));
-                }
-            }
-            float* pool = R.kv_run >= 0 ? m.runs[R.kv_run].k_pool.p : R.k_pool.p;
-            LatentShape ls{};
-            ls.heads = H; ls.dim = d; ls.rot = dr; ls.rank = rank; ls.ld = nf; ls.off_q = L.off_q; ls.off_dkv = L.off_dkv; ls.eps = eps;
-            ls.rot_half = L.d.rot_half;
-            TRY(launch_dep(latent_prepare_kernel, dim3(T), dim3(128), 0, (const float*)m.proj.p, sm, ls, (const float*)L.inv_freq.p, L.cnorm, pool, m.aux.p));
-            LAUNCHED();
-            // the key up-projection moves to the query: qabs[t][h][0 .. rank) = Uk_h^T q_h
-            TRY(gemm_heads(m, m.proj.p + L.off_q, nf, d + dr, L.ukT.p, m.aux.p, H * kd, kd, H, T, rank, d));
-            AttnShape s{};
-            s.heads = H; s.kv_heads = 1; s.dim = kd; s.vdim = rank; s.window = L.d.window; s.rot_dims = 0; s.qk_norm = 0;
-            s.scale = L.d.scale; s.eps = eps; s.ld = H * kd; s.v_ld = kd; s.sink = L.sink;
-            // (the gate is one number a head: it commutes with the value up-projection behind the weighted sum)
-            s.out_gate = L.d.out_gate; s.gate = L.d.out_gate ? m.proj.p + L.off_g : nullptr; s.gate_ld = nf;
-            TRY(attention(s, m.aux.p, pool, pool, m.aux2.p));
-            // ... and the value up-projection behind the weighted sum: att[t][h] = Uv_h (sum_j p_j c_j)
-            TRY(gemm_heads(m, m.aux2.p, H * rank, rank, L.uv, m.att.p, H * dv, dv, H, T, dv, rank));
-            TRY(gemm(m, m.att.p, H * dv, L.o, m.mo.p, D, T, D, H * dv));
+            const int Cv = L.d.heads * L.d.vdim;
+            TRY(gemm(m, front_in, D, L.front, m.proj.p, L.ld_front, T, L.n_front, D, EPI_NONE, 1.f, front_fuse));
+            TRY(latent(L, R, m.att.p, Cv));
+            TRY(gemm(m, m.att.p, Cv, L.o, m.mo.p, D, T, D, Cv));
         }
         if (L.d.ff > 0) {
             const bool fuse_ff = fuse_rows && L.d.ff_kind == TI_SEQ_FF_GLU;
@@ -1580,7 +1661,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             bool down_done = false;
             const int F = L.d.ff;
             if (L.d.ff_kind == TI_SEQ_FF_DENSE) {   // the activation rides in the up product's epilogue
-                const int epi = L.d.ff_act == TI_SEQ_ACT_XIELU ? EPI_XIELU : L.d.ff_act == TI_SEQ_ACT_SILU ? EPI_SILU : L.d.ff_act == TI_SEQ_ACT_GELU_TANH ? EPI_GELU_TANH : EPI_MAX0;
+                const int epi = L.d.ff_act == TI_SEQ_ACT_XIELU ? EPI_XIELU : L.d.ff_act == TI_SEQ_ACT_SILU ? EPI_SILU : L.d.ff_act == TI_SEQ_ACT_GELU_TANH ? EPI_GELU_TANH : L.d.ff_act == TI_SEQ_ACT_GELU ? EPI_GELU : EPI_MAX0;
                 TRY(gemm(m, ff_in, D, L.ffront, m.act.p, F, T, F, D, epi, L.act_a, nullptr, L.act_b));
             } else if (L.d.ff_kind == TI_SEQ_FF_GLU) {
                 if (fuse_ff) {   // norm -> [gate | up] -> act(gate) * up in one launch
@@ -1652,7 +1733,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
     }
     m.dbg_rows = T;
     if (n_out > 0) {
-        // logits: scaled, or capped through cap * tanh(. / cap)
+        // logits: scaled, or scaled and capped through cap * tanh(scale * . / cap)
         const int head_epi = m.d.logit_softcap > 0.f ? EPI_SOFTCAP : EPI_SCALE;
         const float head_alpha = m.d.logit_softcap > 0.f ? m.d.logit_softcap : m.d.logit_scale;
         if (few_rows(n_out, D)) {
@@ -1660,11 +1741,11 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             LAUNCHED();
             Fuse f;
             f.norm_gain = m.final_norm; f.eps = eps; f.gvec = m.gvec;
-            TRY(gemm(m, m.hn.p, D, m.head, m.logits.p, V, n_out, V, D, head_epi, head_alpha, &f));
+            TRY(gemm(m, m.hn.p, D, m.head, m.logits.p, V, n_out, V, D, head_epi, head_alpha, &f, m.d.logit_scale));
         } else {
             TRY(launch_dep(rmsnorm_kernel, dim3(n_out), dim3(nt), 0, (const float*)m.x.p, D, d_out, D, m.final_norm, m.gvec, eps, m.hn.p));
             LAUNCHED();
-            TRY(gemm(m, m.hn.p, D, m.head, m.logits.p, V, n_out, V, D, head_epi, head_alpha));
+            TRY(gemm(m, m.hn.p, D, m.head, m.logits.p, V, n_out, V, D, head_epi, head_alpha, nullptr, m.d.logit_scale));
         }
     }
     if (smp.on) {
@@ -1725,7 +1806,7 @@ int close_seq(Model& m, int32_t seq) {
     return 0;
 }
 
-// A layer whose sublayers share one norm: its front and back matrices (the order of the front's rows: first mixer, state space, router,
+// A layer whose sublayers share one norm: its front and back matrices (the order of the front's rows: first mixer, state space, [up], router,
 // shared expert's scale, [gate | up] or the experts' stacked input matrices; of the back's columns: first mixer, state space, feed-forward).
 int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
     const ti_seq_layer_desc& d = L.d;
@@ -1738,14 +1819,14 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
     std::vector<int*> at;            // where the offset of every front part goes (null: nowhere)
     std::vector<std::string> used;   // tensors that live on inside the two matrices
     const auto add = [&](const std::string& nm, int* off) { fr.push_back(T(nm)); at.push_back(off); used.push_back(nm); };
-    std::vector<std::unique_ptr<Tensor>> zeros;   // rows of zeros that let the part behind them start on a multiple of four columns
-    const auto align = [&]() -> int {
+    std::vector<std::unique_ptr<Tensor>> zeros;   // rows of zeros that let the part behind them start on a multiple of `to` columns
+    const auto align = [&](int to) -> int {
         int64_t rows = 0;
         for (const Tensor* t : fr) rows += t->shape[0];
-        if (rows % 4 == 0) return 0;
+        if (rows % to == 0) return 0;
         zeros.push_back(std::make_unique<Tensor>());
         Tensor& z = *zeros.back();
-        z.shape = {4 - rows % 4, (int64_t)m.d.width};
+        z.shape = {to - rows % to, (int64_t)m.d.width};
         TRY(z.data.alloc(z.count() * m.wsize));
         CK(cudaMemset(z.data.p, 0, z.data.n));
         fr.push_back(&z);
@@ -1755,7 +1836,18 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
     const auto add_back = [&](const std::string& nm) { bk.push_back(T(nm)); used.push_back(nm); };
     int width = 0;
     const std::string pl = p + mix_prefix(d, false), pr = p + mix_prefix(d, true);
-    if (d.mixer != TI_SEQ_MIXER_SSM) {
+    if (d.mixer == TI_SEQ_MIXER_LATENT) {
+        add(pl + (d.q_rank > 0 ? "dq" : "q"), d.q_rank > 0 ? &L.off_dq : &L.off_q);
+        add(pl + "dkv", &L.off_dkv);
+        if (d.out_gate) add(pl + "g", &L.off_g);
+        add_back(pl + "o");
+        width += d.heads * d.vdim;
+    } else if (d.mixer == TI_SEQ_MIXER_DELTA) {
+        add(pl + "q", &L.off_q); add(pl + "k", &L.off_k); add(pl + "v", &L.off_v);   // (side by side: one convolution runs over all three)
+        add(pl + "g", &L.off_g); add(pl + "b", &L.off_b); add(pl + "a", &L.off_a1);
+        add_back(pl + "o");
+        width += d.heads * d.vdim;
+    } else if (d.mixer != TI_SEQ_MIXER_SSM) {
         add(pl + "q", &L.off_q); add(pl + "k", &L.off_k); add(pl + "v", &L.off_v);
         if (d.mixer == TI_SEQ_MIXER_GLA) { add(pl + "g", &L.off_g); add(pl + "a1", &L.off_a1); }
         add_back(pl + "o");
@@ -1772,8 +1864,13 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
     if (d.ff > 0) {
         L.back_ff = width;
         if (d.ff_kind == TI_SEQ_FF_GLU) {
-            TRY(align());
+            TRY(align(4));
             add(p + "mlp.gate", &L.off_up); add(p + "mlp.up", nullptr);
+            add_back(p + "mlp.down");
+            L.ff_width = d.ff;
+        } else if (d.ff_kind == TI_SEQ_FF_DENSE) {
+            TRY(align(16));
+            add(p + "mlp.up", &L.off_up);
             add_back(p + "mlp.down");
             L.ff_width = d.ff;
         } else {
@@ -1784,7 +1881,7 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
                 else add(q + "up", off);
                 add_back(q + "down");
             };
-            TRY(align());
+            TRY(align(4));
             for (int e = 0; e < d.experts; ++e) expert(p + "mlp.e" + std::to_string(e) + ".", e == 0 ? &L.off_up : nullptr);
             if (d.shared_ff > 0) expert(p + "mlp.shared.", &L.off_sh);
             L.ff_width = d.experts * d.ff + d.shared_ff;
@@ -1800,6 +1897,10 @@ int build_shared_norm_layer(Model& m, LayerW& L, const std::string& p) {
         if (at[k]) *at[k] = off[k];
     L.front = L.front_buf.p;
     L.ld_front = (L.n_front + 3) / 4 * 4;   // (rows of the front product start on 16-byte boundaries)
+    if (d.mixer == TI_SEQ_MIXER_LATENT && d.q_rank > 0) {   // the queries come from a second product and sit behind the first one's columns
+        L.off_q = L.ld_front;
+        L.ld_front = (L.ld_front + d.heads * (d.dim + d.rot_dims) + 3) / 4 * 4;
+    }
     TRY(concat_cols(m, bk, L.back_buf, &L.n_back));
     if (L.n_back != width) return fail("internal: output matrices of %d columns, %d expected", L.n_back, width);
     L.back = L.back_buf.p;
@@ -1828,8 +1929,9 @@ int ti_seq_init(int device) {
     g_smem_optin = std::min<size_t>(p.sharedMemPerBlockOptin, 200 * 1024);
     if (!g_stream) CK(cudaStreamCreateWithFlags(&g_stream, cudaStreamNonBlocking));
     CK(cudaFuncSetAttribute(gemv_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
-    CK(cudaFuncSetAttribute(gemv_rows_mma_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
-    CK(cudaFuncSetAttribute(gemv_rows_mma_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
+    CK(cudaFuncSetAttribute(gemv_rows_mma_kernel<COLS_PAIR>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
+    CK(cudaFuncSetAttribute(gemv_rows_mma_kernel<COLS_SINGLE>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
+    CK(cudaFuncSetAttribute(gemv_rows_mma_kernel<COLS_PLAIN>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(wkv_front_rows_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(wkv_front_rows_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(gemv_rows_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
@@ -1852,9 +1954,17 @@ int ti_seq_init(int device) {
     CK(cudaFuncSetAttribute(wkv_scan_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(window_attention_tiled_kernel<8>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(linear_scan_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
-    CK(cudaFuncSetAttribute(latent_attention_h3_kernel<320, 256>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_h3_smem_bytes<320>()));
-    CK(cudaFuncSetAttribute(latent_attention_h3_kernel<192, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_h3_smem_bytes<192>()));
-    CK(cudaFuncSetAttribute(latent_attention_h3_kernel<160, 128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_h3_smem_bytes<160>()));
+#define TI_LAT_ATTR(K, V, KT, X) CK(cudaFuncSetAttribute(latent_attention_h3_kernel<K, V, KT, X>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)latent_h3_smem_bytes<K, KT>()))
+    TI_LAT_ATTR(320, 256, 64, true);
+    TI_LAT_ATTR(192, 128, 64, true);
+    TI_LAT_ATTR(160, 128, 64, true);
+    TI_LAT_ATTR(128, 128, 64, true);
+    TI_LAT_ATTR(128, 128, 64, false);
+    TI_LAT_ATTR(256, 256, 64, true);
+    TI_LAT_ATTR(256, 256, 64, false);
+    TI_LAT_ATTR(512, 512, 32, true);
+    TI_LAT_ATTR(512, 512, 32, false);
+#undef TI_LAT_ATTR
     CK(cudaFuncSetAttribute(mix_scores_tiles_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(mix_scores_tiles_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(mix_scores_rows_kernel<kAttnMaxPerLane>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
@@ -2127,6 +2237,14 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             note_k(L.d.decay_rank);
             m.max_aux = std::max(m.max_aux, L.d.heads * L.d.dim);
         } else if (L.d.mixer == TI_SEQ_MIXER_SSM) {   // (below)
+        } else if (L.d.mixer == TI_SEQ_MIXER_DELTA) {
+            const size_t nq = T(p + "mix.q.conv")->count(), nv = T(p + "mix.v.conv")->count();
+            TRY(L.delta_conv.alloc(2 * nq + nv));
+            CK(cudaMemcpy(L.delta_conv.p, F(p + "mix.q.conv"), nq * sizeof(float), cudaMemcpyDeviceToDevice));
+            CK(cudaMemcpy(L.delta_conv.p + nq, F(p + "mix.k.conv"), nq * sizeof(float), cudaMemcpyDeviceToDevice));
+            CK(cudaMemcpy(L.delta_conv.p + 2 * nq, F(p + "mix.v.conv"), nv * sizeof(float), cudaMemcpyDeviceToDevice));
+            L.dt_bias = F(p + "mix.dt_bias"); L.A_log = F(p + "mix.A_log"); L.normw = F(p + "mix.norm");
+            m.max_aux2 = std::max(m.max_aux2, delta_channels(L.d));
         } else if (L.d.mixer == TI_SEQ_MIXER_GLA || L.d.mixer == TI_SEQ_MIXER_HGRN2) {
             const bool gla = L.d.mixer == TI_SEQ_MIXER_GLA;
             const int C = L.d.heads * L.d.dim, Cv = L.d.heads * L.d.vdim;
@@ -2153,6 +2271,7 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             m.max_att = std::max(m.max_att, Cv);
         } else {   // latent attention
             const int H = L.d.heads, kd = L.d.kv_rank + L.d.rot_dims;
+            if (!shared) {
             std::vector<int> off;
             TRY(concat_rows(m, {T(p + (L.d.q_rank > 0 ? "mix.dq" : "mix.q")), L.d.kv_from < 0 ? T(p + "mix.dkv") : nullptr, L.d.res_gate ? T(p + "rg1") : nullptr,
                                 L.d.out_gate ? T(p + "mix.g") : nullptr}, L.front_buf, &L.n_front, &off));
@@ -2163,13 +2282,17 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
                 L.off_dq = off[0];
                 L.off_q = L.n_front;
                 L.ld_front = L.n_front + H * (L.d.dim + L.d.rot_dims);
+            }
+            rg1_fused = L.d.res_gate != 0;
+            for (const char* s : {"mix.q", "mix.dq", "mix.dkv", "rg1", "mix.g"}) release(p + s);
+            L.o = P(p + "mix.o");
+            }
+            if (L.d.q_rank > 0) {
                 L.uq = P(p + "mix.uq");
                 L.dqnorm = F(p + "mix.dq.norm");
                 note_k(L.d.q_rank);
                 m.max_rank = std::max(m.max_rank, L.d.q_rank);
             }
-            rg1_fused = L.d.res_gate != 0;
-            for (const char* s : {"mix.q", "mix.dq", "mix.dkv", "rg1", "mix.g"}) release(p + s);
             if (L.d.kv_from < 0) L.cnorm = F(p + "mix.dkv.norm");
             if (L.d.sink == TI_SEQ_SINK_LEARNED) L.sink = F(p + "mix.sink");
             TRY(L.ukT.alloc((size_t)H * L.d.dim * L.d.kv_rank * m.wsize));
@@ -2182,7 +2305,6 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             CK(cudaStreamSynchronize(g_stream));
             release(p + "mix.uk");
             L.uv = P(p + "mix.uv");
-            L.o = P(p + "mix.o");
             ti_seq_layer_desc rd = L.d;   // frequencies of the rotated part: every pair of it turns
             rd.rot_scaled = 0;
             const std::vector<float> f = rotary_frequencies(rd);
@@ -2191,7 +2313,7 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             note_k(L.d.dim);
             note_k(L.d.kv_rank);
             m.max_proj = std::max(m.max_proj, L.ld_front);
-            m.max_att = std::max(m.max_att, H * L.d.vdim);
+            if (!shared) m.max_att = std::max(m.max_att, H * L.d.vdim);
             m.max_aux = std::max(m.max_aux, H * kd);
             m.max_aux2 = std::max(m.max_aux2, H * L.d.kv_rank);
             m.max_heads_v = std::max(m.max_heads_v, H * (L.d.kv_rank + 2));
@@ -2322,11 +2444,15 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
             TRY(R.state.alloc((size_t)m.d.max_seqs * L.heads * L.dim * L.vdim));
             CK(cudaMemset(R.state.p, 0, R.state.n * sizeof(float)));
         }
+        if (L.mixer == TI_SEQ_MIXER_DELTA) {
+            TRY(R.mix_conv.alloc(std::max<size_t>(1, (size_t)m.d.max_seqs * (L.mix_taps - 1) * delta_channels(L))));
+            CK(cudaMemset(R.mix_conv.p, 0, R.mix_conv.n * sizeof(float)));
+        }
         if (has_ssm(L)) {
             TRY(R.ssm_state.alloc((size_t)m.d.max_seqs * L.ssm_heads * L.ssm_state * L.ssm_vdim));
             CK(cudaMemset(R.ssm_state.p, 0, R.ssm_state.n * sizeof(float)));
-            TRY(R.ssm_conv.alloc(std::max<size_t>(1, (size_t)m.d.max_seqs * (L.ssm_taps - 1) * ssm_channels(L))));
-            CK(cudaMemset(R.ssm_conv.p, 0, R.ssm_conv.n * sizeof(float)));
+            TRY(R.mix_conv.alloc(std::max<size_t>(1, (size_t)m.d.max_seqs * (L.ssm_taps - 1) * ssm_channels(L))));
+            CK(cudaMemset(R.mix_conv.p, 0, R.mix_conv.n * sizeof(float)));
         }
         if (L.conv_taps > 1) {
             TRY(R.conv_state.alloc((size_t)m.d.max_seqs * (L.conv_taps - 1) * D));
@@ -2545,9 +2671,12 @@ int ti_seq_model_bytes(ti_seq_model_t h, double* weight_bytes, double* kv_bytes_
             w += (2 * C * D + 2 * Cv * D) * ws;   // q, k or f, v, o
             if (L.mixer == TI_SEQ_MIXER_GLA) w += (Cv * D + (double)L.decay_rank * (D + C)) * ws;
             st += (double)L.heads * L.dim * L.vdim * 4;
+        } else if (L.mixer == TI_SEQ_MIXER_DELTA) {
+            w += (2.0 * L.kv_heads * L.dim + 3.0 * L.heads * L.vdim + 2.0 * L.heads) * D * ws;   // q, k, v, gate, o, beta, decay
+            st += ((double)L.heads * L.dim * L.vdim + (double)(L.mix_taps - 1) * delta_channels(L)) * 4;
         } else if (L.mixer != TI_SEQ_MIXER_SSM) {
             const double H = L.heads;
-            w += (H * (L.dim + L.vdim) * L.kv_rank + H * L.vdim * D + (L.out_gate ? H * D : 0.0)) * ws;
+            w += (H * (L.dim + L.vdim) * L.kv_rank + H * L.vdim * D + (L.out_gate == TI_SEQ_GATE_ELEMENT ? H * L.vdim * D : L.out_gate ? H * D : 0.0)) * ws;
             w += (L.q_rank > 0 ? (double)L.q_rank * (D + H * (L.dim + L.rot_dims)) : H * (L.dim + L.rot_dims) * D) * ws;
             if (L.kv_from < 0) {
                 w += (double)(L.kv_rank + L.rot_dims) * D * ws;

@@ -30,6 +30,7 @@ struct TcArgs {
     int ldc;
     int epi;
     float alpha, beta;
+    GluCols cols;   // cols.single with cols.ff > 0: columns cols.first .. N - 1 end as act(v) in cols.out instead of C
     int* err;   // set to 1 when a wait ran out
 };
 
@@ -132,6 +133,24 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
             if (row_ok) {
                 const int nbase = nb * kSgBN + c0;
+                if (g.cols.ff > 0 && nbase + 16 > g.cols.first) {   // activated columns (and the last plain ones beside them)
+                    float* orow = g.cols.out + (size_t)row * g.cols.ld - g.cols.first;
+                    if (nbase >= g.cols.first && nbase + 16 <= g.N && (reinterpret_cast<uintptr_t>(orow + nbase) & 15) == 0) {
+#pragma unroll
+                        for (int i = 0; i < 16; i += 4)
+                            *reinterpret_cast<float4*>(orow + nbase + i) = make_float4(ff_act(__uint_as_float(a[i]), g.cols.act), ff_act(__uint_as_float(a[i + 1]), g.cols.act),
+                                                                                       ff_act(__uint_as_float(a[i + 2]), g.cols.act), ff_act(__uint_as_float(a[i + 3]), g.cols.act));
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < 16; ++i) {
+                            const int n = nbase + i;
+                            if (n >= g.N) break;
+                            if (n >= g.cols.first) orow[n] = ff_act(__uint_as_float(a[i]), g.cols.act);
+                            else epi_put(g.C + (size_t)row * g.ldc + n, __uint_as_float(a[i]), g.epi, g.alpha, g.beta);
+                        }
+                    }
+                    continue;
+                }
                 float* crow = g.C + (size_t)row * g.ldc;
                 if ((g.ldc & 3) == 0 && nbase + 16 <= g.N && (reinterpret_cast<uintptr_t>(g.C) & 15) == 0) {
 #pragma unroll

@@ -26,13 +26,13 @@ namespace seq {
 // What a depth-wise convolution over the last `taps` inputs of a sequence adds up to: y = act(start + sum_j w[d][j] x[pos - (taps - 1) + j])
 struct ConvForm {
     int ldx;            // row stride of the inputs
-    int add_input;      // 1: start = the newest input itself (y = x + conv(x)); 0: start = bias[d]
-    const float* bias;  // [D]; read when add_input is 0
+    int add_input;      // 1: start = the newest input itself (y = x + conv(x)); 0: start = bias[d], or 0 without a bias
+    const float* bias;  // [D] or null; read when add_input is 0
     int silu;           // 1: act(v) = v sigmoid(v)
 };
 template <int V> __device__ __forceinline__ void conv_start(const ConvForm& f, int d, const float (&xv)[V], float (&acc)[V]) {
 #pragma unroll
-    for (int c = 0; c < V; ++c) acc[c] = f.add_input ? xv[c] : f.bias[d + c];
+    for (int c = 0; c < V; ++c) acc[c] = f.add_input ? xv[c] : f.bias ? f.bias[d + c] : 0.f;
 }
 template <int V> __device__ __forceinline__ void conv_finish(const ConvForm& f, float (&acc)[V]) {
     if (f.silu) {

@@ -155,36 +155,41 @@ __global__ void postnorm_residual_kernel(PostArgs a) {
 
 // ---- matrix products: C[M, N] = epi(A[M, K] . W[N, K]^T) ----------------------------------------------------------------
 enum {
-    EPI_NONE = 0, EPI_TANH = 1, EPI_SCALE = 2, EPI_SILU = 3, EPI_SOFTCAP = 4 /* alpha * tanh(v / alpha) */, EPI_GELU_TANH = 5,
-    EPI_XIELU = 6 /* alpha v^2 + v / 2 for v > 0, beta (exp(v) - 1 - v) + v / 2 otherwise */, EPI_MAX0 = 7,
+    EPI_NONE = 0, EPI_TANH = 1, EPI_SCALE = 2, EPI_SILU = 3, EPI_SOFTCAP = 4 /* alpha * tanh(beta v / alpha) */, EPI_GELU_TANH = 5,
+    EPI_XIELU = 6 /* alpha v^2 + v / 2 for v > 0, beta (exp(v) - 1 - v) + v / 2 otherwise */, EPI_MAX0 = 7, EPI_GELU = 9 /* the error-function form */,
     EPI_ADD = 8 /* C += v: the product ends in the residual sum (every element of C has one writer) */
 };
 __device__ __forceinline__ float xielu(float v, float a_pos, float a_neg) {
     return v > 0.f ? fmaf(a_pos * v, v, 0.5f * v) : fmaf(a_neg, expm1f(v) - v, 0.5f * v);
 }
+__device__ __forceinline__ float gelu_erf(float v) { return 0.5f * v * (1.f + erff(v * 0.7071067811865476f)); }
 __device__ __forceinline__ float epi_apply(float v, int epi, float alpha, float beta = 0.f) {
     if (epi == EPI_XIELU) return xielu(v, alpha, beta);
     if (epi == EPI_MAX0) return fmaxf(v, 0.f);
     if (epi == EPI_TANH) return tanhf(v);
     if (epi == EPI_SCALE) return v * alpha;
     if (epi == EPI_SILU) return v / (1.f + expf(-v));
-    if (epi == EPI_SOFTCAP) return alpha * tanhf(v / alpha);
+    if (epi == EPI_SOFTCAP) return alpha * tanhf(v * beta / alpha);
+    if (epi == EPI_GELU) return gelu_erf(v);
     if (epi == EPI_GELU_TANH) return 0.5f * v * (1.f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
     return v;
 }
 
+__device__ __forceinline__ float sigmoid_f32(float z) { return 1.f / (1.f + expf(-z)); }
 __device__ __forceinline__ void epi_put(float* c, float v, int epi, float alpha, float beta) {
     *c = epi == EPI_ADD ? *c + v : epi_apply(v, epi, alpha, beta);
 }
 
 // true fp32: 64 x 64 tile, 16-deep k-steps, 256 threads with 4 x 4 outputs each
-// (grid.z > 1: a batch of products, number z reads A + z * za, W + z * zw and writes C + z * zc -- one small matrix per head)
+// (grid.z > 1: a batch of products, number z reads A + z * za, W + z * zw and writes C + z * zc -- one small matrix per head;
+// gate: the result is multiplied by sigmoid(gate[row * ldg + z * zc + column]), the columns of all products side by side)
 __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* A, int lda, const float* W, float* C, int ldc, int M, int N, int K,
-                                                        int epi, float alpha, float beta, size_t za, size_t zw, size_t zc) {
+                                                        int epi, float alpha, float beta, size_t za, size_t zw, size_t zc, const float* gate, int ldg) {
     __shared__ float As[16][64 + 4], Ws[16][64 + 4];
     A += blockIdx.z * za;
     W += blockIdx.z * zw;
     C += blockIdx.z * zc;
+    if (gate) gate += blockIdx.z * zc;
     const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
     const int m0 = blockIdx.y * 64, n0 = blockIdx.x * 64;
     float acc[4][4] = {};
@@ -215,7 +220,7 @@ __global__ void __launch_bounds__(256) gemm_f32_kernel(const float* A, int lda, 
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int gm = m0 + ty * 4 + i, gn = n0 + tx * 4 + j;
-            if (gm < M && gn < N) epi_put(C + (size_t)gm * ldc + gn, acc[i][j], epi, alpha, beta);
+            if (gm < M && gn < N) epi_put(C + (size_t)gm * ldc + gn, gate ? acc[i][j] * sigmoid_f32(gate[(size_t)gm * ldg + gn]) : acc[i][j], epi, alpha, beta);
         }
 }
 
@@ -228,12 +233,13 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], const uint32_t (&a
 }
 // (grid.z > 1: a batch of products, as in gemm_f32_kernel)
 __global__ void __launch_bounds__(128) gemm_bf16_kernel(const float* A, int lda, const __nv_bfloat16* W, float* C, int ldc, int M, int N,
-                                                         int K, int epi, float alpha, float beta, size_t za, size_t zw, size_t zc) {
+                                                         int K, int epi, float alpha, float beta, size_t za, size_t zw, size_t zc, const float* gate, int ldg) {
     constexpr int BM = 64, BN = 64, BK = 32, LD = BK + 8;
     __shared__ __align__(16) __nv_bfloat16 As[BM * LD], Ws[BN * LD];
     A += blockIdx.z * za;
     W += blockIdx.z * zw;
     C += blockIdx.z * zc;
+    if (gate) gate += blockIdx.z * zc;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t4 = lane & 3;
     const int wm = (warp >> 1) * 32, wn = (warp & 1) * 32;
     const int m0 = blockIdx.y * BM, n0 = blockIdx.x * BN;
@@ -301,7 +307,7 @@ __global__ void __launch_bounds__(128) gemm_bf16_kernel(const float* A, int lda,
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
                 const int gm = m0 + wm + i * 16 + g + (e >> 1) * 8, gn = n0 + wn + j * 8 + 2 * t4 + (e & 1);
-                if (gm < M && gn < N) epi_put(C + (size_t)gm * ldc + gn, acc[i][j][e], epi, alpha, beta);
+                if (gm < M && gn < N) epi_put(C + (size_t)gm * ldc + gn, gate ? acc[i][j][e] * sigmoid_f32(gate[(size_t)gm * ldg + gn]) : acc[i][j][e], epi, alpha, beta);
             }
 }
 
@@ -312,13 +318,16 @@ __global__ void __launch_bounds__(128) gemm_bf16_kernel(const float* A, int lda,
 constexpr int kRowGemvMaxRows = 8;
 constexpr int kRowGemvThreads = 256;
 __device__ __forceinline__ float glu_pair(float g, float u, int act, float limit);
+__device__ __forceinline__ float ff_act(float z, int act);
 // Columns [0, first) of the product are plain and go to C; columns first .. N - 1 are gates whose partner column lies ff behind:
-// out[r * ld + n - first] = act(gate) * up.  ff = 0: every column is plain.
+// out[r * ld + n - first] = act(gate) * up.  ff = 0: every column is plain.  single = 1: no partners, columns first .. N - 1 end as
+// out[r * ld + n - first] = act(column) (a feed-forward without a gate).
 struct GluCols {
     int ff, act, first;
     float limit;
     float* out;
     int ld;
+    int single;
 };
 // eight consecutive weights as they lie in memory (kept packed while the loads are in flight) and as fp32
 template <typename WT> struct Raw8;
@@ -394,7 +403,7 @@ __global__ void __launch_bounds__(kRowGemvThreads, 2) gemv_rows_kernel(const flo
         if (n < N) {
             const char* w = reinterpret_cast<const char*>(W + (size_t)n * K);
             for (size_t o = (size_t)lane * 128; o < row_bytes; o += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
-            if (glu.ff > 0 && n >= glu.first) {
+            if (glu.ff > 0 && !glu.single && n >= glu.first) {
                 const char* w2 = reinterpret_cast<const char*>(W + (size_t)(n + glu.ff) * K);
                 for (size_t o = (size_t)lane * 128; o < row_bytes; o += 32 * 128) asm volatile("prefetch.global.L2 [%0];" ::"l"(w2 + o));
             }
@@ -442,12 +451,12 @@ __global__ void __launch_bounds__(kRowGemvThreads, 2) gemv_rows_kernel(const flo
     for (int n = blockIdx.x * nw + warp; n < N; n += gridDim.x * nw) {
         gemv_row_dot<WT>(W + (size_t)n * K, xs, M, K, vec, lane, acc);
         const bool gated = glu.ff > 0 && n >= glu.first;
-        if (gated) gemv_row_dot<WT>(W + (size_t)(n + glu.ff) * K, xs, M, K, vec, lane, acc2);
+        if (gated && !glu.single) gemv_row_dot<WT>(W + (size_t)(n + glu.ff) * K, xs, M, K, vec, lane, acc2);
         if (lane == 0) {
 #pragma unroll
             for (int r = 0; r < kRowGemvMaxRows; ++r)
                 if (r < M) {
-                    if (gated) glu.out[(size_t)r * glu.ld + n - glu.first] = glu_pair(acc[r], acc2[r], glu.act, glu.limit);
+                    if (gated) glu.out[(size_t)r * glu.ld + n - glu.first] = glu.single ? ff_act(acc[r], glu.act) : glu_pair(acc[r], acc2[r], glu.act, glu.limit);
                     else epi_put(C + (size_t)r * ldc + n, acc[r], epi, alpha, beta);
                 }
         }
@@ -455,10 +464,11 @@ __global__ void __launch_bounds__(kRowGemvThreads, 2) gemv_rows_kernel(const flo
 }
 
 // Few rows, one small matrix per head: C[r][h * c_stride + n] = sum_k A[r][h * a_stride + k] * W[h][n][k] (W: [heads][N][K]).
-// grid (column groups, heads); the head's slice of the rows sits in shared memory, one warp per output column.
+// grid (column groups, heads); the head's slice of the rows sits in shared memory, one warp per output column.  gate: the result is
+// multiplied by sigmoid(gate[r * ldg + h * c_stride + n]).
 template <typename WT>
 __global__ void __launch_bounds__(kRowGemvThreads) gemv_heads_rows_kernel(const float* A, int lda, int a_stride, const WT* W, float* C, int ldc, int c_stride, int M, int N,
-                                                                           int K) {
+                                                                           int K, const float* gate, int ldg) {
     extern __shared__ __align__(16) float xs[];   // [M][K]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5, h = blockIdx.y;
     pdl_launch_dependents();
@@ -473,7 +483,7 @@ __global__ void __launch_bounds__(kRowGemvThreads) gemv_heads_rows_kernel(const 
         if (lane == 0) {
 #pragma unroll
             for (int r = 0; r < kRowGemvMaxRows; ++r)
-                if (r < M) C[(size_t)r * ldc + (size_t)h * c_stride + n] = acc[r];
+                if (r < M) C[(size_t)r * ldc + (size_t)h * c_stride + n] = gate ? acc[r] * sigmoid_f32(gate[(size_t)r * ldg + (size_t)h * c_stride + n]) : acc[r];
         }
     }
 }
@@ -510,10 +520,12 @@ __device__ __forceinline__ void mma_bf16_16816(float (&c)[4], uint32_t a0, uint3
                  : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
                  : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
-template <bool GLU>
+enum { COLS_PLAIN = 0, COLS_PAIR = 1, COLS_SINGLE = 2 };   // GluCols: none, gates with a partner, activation columns
+template <int COLS>
 __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int lda, const __nv_bfloat16* W, float* C, int ldc, int M, int N, int K, int epi,
                                                            float alpha, float beta, const float* norm_gain, float eps, GluCols glu, int gvec, ExpertSkip nskip,
                                                            ExpertSkip kskip) {
+    constexpr bool GLU = COLS == COLS_PAIR, SPLIT = COLS != COLS_PLAIN;
     extern __shared__ __align__(16) unsigned char smraw[];
     const int Kp = K + 32;
     __nv_bfloat16* xs = reinterpret_cast<__nv_bfloat16*>(smraw);                       // [M][Kp]
@@ -526,16 +538,16 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
     __shared__ int ucount;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
     const bool skip = kskip.used && !norm_gain && kskip.count <= kSkipMaxExperts;   // (a norm in front needs the whole row)
-    const bool nskips = !GLU && nskip.used && nskip.count <= kSkipMaxExperts;
+    const bool nskips = !SPLIT && nskip.used && nskip.count <= kSkipMaxExperts;
     const int per_expert = nskip.group / kMmaCols;
     const bool dealt = nskips && nskip.first == 0 && nskip.group % kMmaCols == 0;   // every expert's columns are whole tiles
     const int NC = K / 32, c_begin = warp * NC / 8, c_end = (warp + 1) * NC / 8;   // this warp's 32-k chunks
-    // column tiles: the plain columns in sixteens, then (GLU) the gated ones
-    const int plain_cols = GLU ? glu.first : N, plain_tiles = (plain_cols + kMmaCols - 1) / kMmaCols;
-    const int tiles = plain_tiles + (GLU ? (N - plain_cols + kMmaCols - 1) / kMmaCols : 0);
+    // column tiles: the plain columns in sixteens, then the gated / activated ones
+    const int plain_cols = SPLIT ? glu.first : N, plain_tiles = (plain_cols + kMmaCols - 1) / kMmaCols;
+    const int tiles = plain_tiles + (SPLIT ? (N - plain_cols + kMmaCols - 1) / kMmaCols : 0);
     pdl_launch_dependents();
     {   // ask L2 for this warp's slice of the block's first 16 (32 with the gate's partner) weight rows
-        const bool gated = GLU && (int)blockIdx.x >= plain_tiles;
+        const bool gated = SPLIT && (int)blockIdx.x >= plain_tiles;
         const int n = gated ? min(plain_cols + ((int)blockIdx.x - plain_tiles) * kMmaCols + (lane & 15), N - 1) : min((int)blockIdx.x * kMmaCols + (lane & 15), plain_cols - 1);
         const char* w = reinterpret_cast<const char*>(W + (size_t)n * K + (size_t)c_begin * 32);
         // (what the step's rows chose is not known yet: nothing of the experts is asked for)
@@ -544,7 +556,7 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
         const size_t bytes = p_end > c_begin && !expert_tile ? (size_t)(p_end - c_begin) * 64 : 0;
         for (size_t o = (size_t)(lane >> 4) * 128; o < bytes; o += 256) {
             asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o));
-            if (gated) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o + (size_t)glu.ff * K * 2));
+            if (GLU && gated) asm volatile("prefetch.global.L2 [%0];" ::"l"(w + o + (size_t)glu.ff * K * 2));
         }
     }
     pdl_wait_prior_grid();
@@ -656,7 +668,7 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
     const int c0 = skip ? warp * NA / 8 : c_begin, c1 = skip ? (warp + 1) * NA / 8 : c_end;
     for (int turn = blockIdx.x; turn < turns; turn += gridDim.x) {
         const int tile = !dealt ? turn : turn < used_tiles ? (int)ulist[turn / per_expert] * per_expert + turn % per_expert : nskip.count * per_expert + turn - used_tiles;
-        const bool gated = GLU && tile >= plain_tiles;
+        const bool gated = SPLIT && tile >= plain_tiles;
         const int n0 = gated ? plain_cols + (tile - plain_tiles) * kMmaCols : tile * kMmaCols, end = gated ? N : plain_cols;
         if (nskips && !dealt && !expert_range_used(nskip, ubits, n0, min(n0 + kMmaCols, end) - 1)) continue;   // (uniform over the block)
         float acc[4] = {0.f, 0.f, 0.f, 0.f}, acc2[4] = {0.f, 0.f, 0.f, 0.f};
@@ -673,7 +685,7 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
                     const int k = (skip ? (int)klist[cc] : cc) * 32;
                     ra[q] = *reinterpret_cast<const uint4*>(w0 + k);
                     rb[q] = *reinterpret_cast<const uint4*>(w1 + k);
-                    if (gated) {
+                    if (GLU && gated) {
                         ua[q] = *reinterpret_cast<const uint4*>(w0 + up + k);
                         ub[q] = *reinterpret_cast<const uint4*>(w1 + up + k);
                     }
@@ -686,7 +698,7 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
                     if (g < M) x = *reinterpret_cast<const uint4*>(xr + (c + q) * 32);
                     mma_bf16_16816(acc, ra[q].x, rb[q].x, ra[q].y, rb[q].y, x.x, x.y);
                     mma_bf16_16816(acc, ra[q].z, rb[q].z, ra[q].w, rb[q].w, x.z, x.w);
-                    if (gated) {
+                    if (GLU && gated) {
                         mma_bf16_16816(acc2, ua[q].x, ub[q].x, ua[q].y, ub[q].y, x.x, x.y);
                         mma_bf16_16816(acc2, ua[q].z, ub[q].z, ua[q].w, ub[q].w, x.z, x.w);
                     }
@@ -708,7 +720,7 @@ __global__ void __launch_bounds__(256) gemv_rows_mma_kernel(const float* A, int 
                 if (GLU) v2 += red[(w * 2 + 1) * 128 + src];
             }
             if (r < M && n0 + j < end) {
-                if (gated) glu.out[(size_t)r * glu.ld + n0 + j - plain_cols] = glu_pair(v, v2, glu.act, glu.limit);
+                if (gated) glu.out[(size_t)r * glu.ld + n0 + j - plain_cols] = GLU ? glu_pair(v, v2, glu.act, glu.limit) : ff_act(v, glu.act);
                 else epi_put(C + (size_t)r * ldc + n0 + j, v, epi, alpha, beta);
             }
         }
@@ -814,7 +826,14 @@ struct AttnShape {
     const float* pb;                  // [heads] or null: no softmax, a visible key's weight is sigmoid(score + pb[h])
     int out_ld = 0;                   // row stride of the output; 0: heads * vdim
     float out_scale = 1.f;            // factor on the output
+    int chunk = 0;                    // > 0: a row sees no key in front of its own chunk of positions (pos / chunk * chunk)
 };
+// the first key position a row at `pos` sees (never later for an earlier row)
+__device__ __forceinline__ int attn_first_key(const AttnShape& s, int pos) {
+    int lo = s.window > 0 ? max(pos - s.window + 1, 0) : 0;
+    if (s.chunk > 0) lo = max(lo, pos / s.chunk * s.chunk);
+    return lo;
+}
 __device__ __forceinline__ size_t attn_out_stride(const AttnShape& s) { return s.out_ld ? (size_t)s.out_ld : (size_t)s.heads * s.vdim; }
 // score of a (query, key) pair from their dot product, and a visible key's weight when there is no softmax
 __device__ __forceinline__ float attn_score(const AttnShape& s, float dot) {
@@ -947,7 +966,7 @@ __global__ void __launch_bounds__(kAttnWarps * 32) window_attention_kernel(const
         qr[i] = d < s.dim ? q[d] : 0.f;
         o[i] = 0.f;
     }
-    const int lo = (s.window > 0 && pos - s.window + 1 > 0) ? pos - s.window + 1 : 0;
+    const int lo = attn_first_key(s, pos);
     float mx = s.pb ? 0.f : -INFINITY, l = 0.f;   // (weights without a softmax: the running maximum stays 0)
     const float pb = s.pb ? s.pb[h] : 0.f;
     const size_t kstride = (size_t)s.kv_heads * s.dim, vstride = attn_vstride(s);
@@ -1027,7 +1046,7 @@ __global__ void __launch_bounds__(256) window_attention_tiled_kernel(const float
         const int r = i / d, k = i % d;
         Qs[r * ldq + k] = r < n ? qkvg[(size_t)(row0 + r) * s.ld + (size_t)h * d + k] : 0.f;
     }
-    const int lo = (s.window > 0 && p0 - s.window + 1 > 0) ? p0 - s.window + 1 : 0, hi = p0 + n - 1;
+    const int lo = attn_first_key(s, p0), hi = p0 + n - 1;
     float mrow[4], lrow[4], acc[4][DV4 * 4];
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
@@ -1072,13 +1091,13 @@ __global__ void __launch_bounds__(256) window_attention_tiled_kernel(const float
         }
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
-            const int r = ty + 16 * i, pos = p0 + r;
+            const int r = ty + 16 * i, pos = p0 + r, row_lo = attn_first_key(s, pos);
             bool ok[4];
             float tmax = -INFINITY;
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 const int key = pg * kPageTokens + tx + 16 * j;
-                ok[j] = r < n && key <= pos && (s.window <= 0 || key > pos - s.window);
+                ok[j] = r < n && key <= pos && key >= row_lo;
                 sc[i][j] = ok[j] ? attn_score(s, sc[i][j]) : -INFINITY;
                 tmax = fmaxf(tmax, sc[i][j]);
             }
@@ -1154,10 +1173,11 @@ inline size_t attn_tiled_smem_bytes(int d, int dv, bool v_in_k = false) {
 }
 
 // ---- gated feed-forward: act(gate) * up over the fused projection output [gate | up] ------------------------------------
-enum { ACT_RELU = 0, ACT_SILU = 1, ACT_GELU_TANH = 2, ACT_CLAMPED_SWISH = 4 };
+enum { ACT_RELU = 0, ACT_SILU = 1, ACT_GELU_TANH = 2, ACT_CLAMPED_SWISH = 4, ACT_GELU = 5 };
 __device__ __forceinline__ float ff_act(float z, int act) {
     if (act == 0 /*ACT_RELU*/) return fmaxf(z, 0.f);
     if (act == 1 /*ACT_SILU*/) return z / (1.f + expf(-z));
+    if (act == ACT_GELU) return gelu_erf(z);
     return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 // the gated feed-forward's inner value.  CLAMPED_SWISH: g = min(gate, limit), u = up cut to [-limit, limit], g sigmoid(1.702 g) (u + 1)
@@ -1185,6 +1205,26 @@ __global__ void glu_kernel(const float* gu, int ld, int ff, int act, float limit
             *reinterpret_cast<float4*>(o) = make_float4(glu_pair(a.x, b.x, act, limit), glu_pair(a.y, b.y, act, limit), glu_pair(a.z, b.z, act, limit), glu_pair(a.w, b.w, act, limit));
         } else {
             *o = glu_pair(*g, *u, act, limit);
+        }
+    }
+}
+
+// act of every element of rows [T][ff] (row stride ld) -> y (row stride ldy); V as above
+template <int V>
+__global__ void act_kernel(const float* u, int ld, int ff, int act, float* y, int ldy, int T) {
+    pdl_launch_dependents();
+    pdl_wait_prior_grid();
+    const int per = ff / V;
+    const size_t n = (size_t)T * per;
+    for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t t = i / per, c = (i % per) * V;
+        const float* g = u + t * ld + c;
+        float* o = y + t * ldy + c;
+        if constexpr (V == 4) {
+            const float4 a = *reinterpret_cast<const float4*>(g);
+            *reinterpret_cast<float4*>(o) = make_float4(ff_act(a.x, act), ff_act(a.y, act), ff_act(a.z, act), ff_act(a.w, act));
+        } else {
+            *o = ff_act(*g, act);
         }
     }
 }

@@ -7,7 +7,9 @@
 //     out_h(i)      = sum_j p_h(i, j) Uv_h c_j                = Uv_h (sum_j p_h(i, j) c_j)
 // so the attention itself is one key/value head of size rank + rot (values = the first rank coordinates of the key row) shared
 // by all query heads, and runs on the paged attention kernels of seq_kernels.cuh / seq_attn_tc.cuh (value pool = key pool; a
-// sliding window, a sink term and a per-head output gate -- one number a head, so it commutes with Uv -- are the layer's choice).  This file holds what is special: the cache append and the query's rotated part.
+// sliding window, chunks, a sink term and an output gate are the layer's choice: a gate of one number a head commutes with Uv and is
+// applied to the weighted sum, a gate per coordinate in the epilogue of the product with Uv).  rot may be 0: no rotated part.  This file
+// holds what is special: the cache append and the query's rotated part.
 #pragma once
 #include "seq_attn_tc.cuh"
 #include "seq_kernels.cuh"
@@ -80,19 +82,22 @@ __global__ void transpose_heads_kernel(const WT* uk, int heads, int dim, int ran
 // coordinates of its DK-wide key rows -- so the key tile in shared memory is also the value tile and nothing is loaded twice.
 // A block owns up to 64 consecutive rows of one sequence and one query head; its 8 warps are 4 row groups x 2 halves of the
 // value columns: both warps of a row group compute the 16 x 64 scores of a key tile (the softmax needs whole rows), each
-// accumulates its half of the DV output columns -- a DV-wide output tile of 16 rows does not fit one warp's registers.
+// accumulates its half of the DV output columns -- a DV-wide output tile of 16 rows does not fit one warp's registers.  KT keys a
+// tile (64 = a page; 32 where two halves of 64 wide rows would not fit shared memory).  SIZED = false (DK = DV): the layer's row is
+// s.dim <= DK wide (in fours), padded with zeros in shared memory.
 // tiles[2 i] = first row, tiles[2 i + 1] = row count; q = absorbed queries [T][heads][DK]; pool = [pages * 64][DK].
 constexpr int kLatQ = 64;
-template <int DK> constexpr size_t latent_h3_smem_bytes() { return ((size_t)2 * kLatQ + 2 * kTcKT) * (DK + 8) * sizeof(__half); }
-template <int DK, int DV>
+template <int DK, int KT = kTcKT> constexpr size_t latent_h3_smem_bytes() { return ((size_t)2 * kLatQ + 2 * KT) * (DK + 8) * sizeof(__half); }
+template <int DK, int DV, int KT, bool SIZED>
 __global__ void __launch_bounds__(256, 1) latent_attention_h3_kernel(const float* q, StepMeta m, AttnShape s, const int* tiles, const float* pool, float* out) {
     constexpr int LD = DK + 8, KS = DK / 16, NTH = DV / 16;   // NTH: 8-column output tiles a warp owns = (DV / 2) / 8
-    static_assert(DK % 16 == 0 && DV % 32 == 0 && DV <= DK, "tile sizes");
+    static_assert(DK % 16 == 0 && DV % 32 == 0 && DV <= DK && kPageTokens % KT == 0 && KT % 16 == 0 && (SIZED || DK == DV), "tile sizes");
+    const int d = SIZED ? DK : s.dim, dv = SIZED ? DV : s.vdim;
     extern __shared__ __align__(16) __half lat_smem[];
     __half* Qh = lat_smem;                 // [64][LD]
     __half* Ql = Qh + kLatQ * LD;
     __half* Kh = Ql + kLatQ * LD;          // [64][LD]: keys, and in their leading DV columns the values
-    __half* Kl = Kh + kTcKT * LD;
+    __half* Kl = Kh + KT * LD;
     const int row0 = tiles[2 * blockIdx.x], M = tiles[2 * blockIdx.x + 1], h = blockIdx.y;
     const int pos0 = m.row_pos[row0];
     const int* table = m.page_table + (size_t)m.ent_slot[m.row_ent[row0]] * m.table_stride;
@@ -108,8 +113,8 @@ __global__ void __launch_bounds__(256, 1) latent_attention_h3_kernel(const float
     for (int i = tid; i < kLatQ * (DK / 4); i += 256) {
         const int qi = i / (DK / 4), d4 = (i % (DK / 4)) * 4;
         float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (qi < M) {
-            const float* src = q + (size_t)(row0 + qi) * s.ld + (size_t)h * DK + d4;
+        if (qi < M && d4 < d) {
+            const float* src = q + (size_t)(row0 + qi) * s.ld + (size_t)h * d + d4;
             v = make_float4(src[0], src[1], src[2], src[3]);
         }
         store_split4(v, Qh + qi * LD + d4, Ql + qi * LD + d4);
@@ -119,35 +124,35 @@ __global__ void __launch_bounds__(256, 1) latent_attention_h3_kernel(const float
     for (int n = 0; n < NTH; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
     float m0 = -INFINITY, m1 = -INFINITY, l0 = 0.f, l1 = 0.f;
     const int last_pos = pos0 + M - 1;
-    const int lo = (s.window > 0 && pos0 - s.window + 1 > 0) ? pos0 - s.window + 1 : 0;   // first key any row of the tile sees
+    const int lo = attn_first_key(s, pos0);   // first key any row of the tile sees
     const int warp_first = pos0 + 16 * rg, warp_last = pos0 + min(16 * rg + 15, M - 1);
-    const int warp_lo = (s.window > 0 && warp_first - s.window + 1 > 0) ? warp_first - s.window + 1 : 0;
+    const int warp_lo = attn_first_key(s, warp_first), lo0 = attn_first_key(s, pos0 + r0), lo1 = attn_first_key(s, pos0 + r1);
     const uint32_t* qh_row = reinterpret_cast<const uint32_t*>(Qh + (16 * rg + g) * LD) + t;
     const uint32_t* ql_row = reinterpret_cast<const uint32_t*>(Ql + (16 * rg + g) * LD) + t;
     const int lm = lane >> 3, lr = lane & 7;
     const uint32_t k_ld = (uint32_t)(((lr + 8 * (lm >> 1)) * LD + 8 * (lm & 1)) * 2);
     const uint32_t v_ld = (uint32_t)(((lr + 8 * (lm & 1)) * LD + 8 * (lm >> 1)) * 2);
     const uint32_t kh_s = smem_u32(Kh), kl_s = smem_u32(Kl);
-    for (int t0 = lo / kPageTokens * kPageTokens; t0 <= last_pos; t0 += kTcKT) {   // a key tile = a page; pages below the window are not visited
+    for (int t0 = lo / KT * KT; t0 <= last_pos; t0 += KT) {   // a key tile lies in one page; tiles below the window are not visited
         __syncthreads();
-        const size_t tok0 = (size_t)table[t0 / kPageTokens] * kPageTokens;
-        for (int i = tid; i < kTcKT * (DK / 4); i += 256) {
+        const size_t tok0 = (size_t)table[t0 / kPageTokens] * kPageTokens + t0 % kPageTokens;
+        for (int i = tid; i < KT * (DK / 4); i += 256) {
             const int kk = i / (DK / 4), d4 = (i % (DK / 4)) * 4;
             float4 kv = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (t0 + kk >= lo && t0 + kk <= last_pos) kv = *reinterpret_cast<const float4*>(pool + (tok0 + kk) * (size_t)DK + d4);
+            if (t0 + kk >= lo && t0 + kk <= last_pos && d4 < d) kv = *reinterpret_cast<const float4*>(pool + (tok0 + kk) * (size_t)d + d4);
             store_split4(kv, Kh + kk * LD + d4, Kl + kk * LD + d4);
         }
         __syncthreads();
-        if (t0 > warp_last || t0 + kTcKT - 1 < warp_lo || 16 * rg >= M) continue;   // nothing of this page is visible to the warp's rows
-        float sc[kTcKT / 8][4];
+        if (t0 > warp_last || t0 + KT - 1 < warp_lo || 16 * rg >= M) continue;   // nothing of this page is visible to the warp's rows
+        float sc[KT / 8][4];
 #pragma unroll
-        for (int j = 0; j < kTcKT / 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
+        for (int j = 0; j < KT / 8; ++j) sc[j][0] = sc[j][1] = sc[j][2] = sc[j][3] = 0.f;
 #pragma unroll 4
         for (int ks = 0; ks < KS; ++ks) {
             const uint32_t ah[4] = {qh_row[8 * ks], qh_row[8 * ks + 4 * LD], qh_row[8 * ks + 4], qh_row[8 * ks + 4 * LD + 4]};
             const uint32_t al[4] = {ql_row[8 * ks], ql_row[8 * ks + 4 * LD], ql_row[8 * ks + 4], ql_row[8 * ks + 4 * LD + 4]};
 #pragma unroll
-            for (int jp = 0; jp < kTcKT / 16; ++jp) {
+            for (int jp = 0; jp < KT / 16; ++jp) {
                 uint32_t bh[4], bl[4];
                 const uint32_t off = (uint32_t)((16 * jp * LD + 16 * ks) * 2) + k_ld;
                 ldsm_x4(bh, kh_s + off);
@@ -161,15 +166,14 @@ __global__ void __launch_bounds__(256, 1) latent_attention_h3_kernel(const float
             }
         }
         const int qp0 = pos0 + r0, qp1 = pos0 + r1;
-        const int w = s.window > 0 ? s.window : 0x3FFFFFFF;
         float mx0 = -INFINITY, mx1 = -INFINITY;
 #pragma unroll
-        for (int j = 0; j < kTcKT / 8; ++j) {
+        for (int j = 0; j < KT / 8; ++j) {
             const int key = t0 + 8 * j + 2 * t;
-            sc[j][0] = (key <= qp0 && key > qp0 - w && r0 < M) ? sc[j][0] * s.scale : -INFINITY;
-            sc[j][1] = (key + 1 <= qp0 && key + 1 > qp0 - w && r0 < M) ? sc[j][1] * s.scale : -INFINITY;
-            sc[j][2] = (key <= qp1 && key > qp1 - w && r1 < M) ? sc[j][2] * s.scale : -INFINITY;
-            sc[j][3] = (key + 1 <= qp1 && key + 1 > qp1 - w && r1 < M) ? sc[j][3] * s.scale : -INFINITY;
+            sc[j][0] = (key <= qp0 && key >= lo0 && r0 < M) ? sc[j][0] * s.scale : -INFINITY;
+            sc[j][1] = (key + 1 <= qp0 && key + 1 >= lo0 && r0 < M) ? sc[j][1] * s.scale : -INFINITY;
+            sc[j][2] = (key <= qp1 && key >= lo1 && r1 < M) ? sc[j][2] * s.scale : -INFINITY;
+            sc[j][3] = (key + 1 <= qp1 && key + 1 >= lo1 && r1 < M) ? sc[j][3] * s.scale : -INFINITY;
             mx0 = fmaxf(mx0, fmaxf(sc[j][0], sc[j][1]));
             mx1 = fmaxf(mx1, fmaxf(sc[j][2], sc[j][3]));
         }
@@ -178,7 +182,7 @@ __global__ void __launch_bounds__(256, 1) latent_attention_h3_kernel(const float
         const float mn0 = fmaxf(m0, mx0), mn1 = fmaxf(m1, mx1);
         float rs0 = 0.f, rs1 = 0.f;
 #pragma unroll
-        for (int j = 0; j < kTcKT / 8; ++j) {
+        for (int j = 0; j < KT / 8; ++j) {
             sc[j][0] = mn0 == -INFINITY ? 0.f : expf(sc[j][0] - mn0);
             sc[j][1] = mn0 == -INFINITY ? 0.f : expf(sc[j][1] - mn0);
             sc[j][2] = mn1 == -INFINITY ? 0.f : expf(sc[j][2] - mn1);
@@ -196,7 +200,7 @@ __global__ void __launch_bounds__(256, 1) latent_attention_h3_kernel(const float
 #pragma unroll
         for (int n = 0; n < NTH; ++n) { o[n][0] *= c0; o[n][1] *= c0; o[n][2] *= c1; o[n][3] *= c1; }
 #pragma unroll
-        for (int jp = 0; jp < kTcKT / 16; ++jp) {
+        for (int jp = 0; jp < KT / 16; ++jp) {
             uint32_t ph[4], pl[4];
 #pragma unroll
             for (int i = 0; i < 4; ++i) {
@@ -224,10 +228,12 @@ __global__ void __launch_bounds__(256, 1) latent_attention_h3_kernel(const float
     }
     const float i0 = r0 < M ? attn_finish_factor(s, h, m0, l0) * attn_gate(s, q, row0 + r0, h) : 0.f;
     const float i1 = r1 < M ? attn_finish_factor(s, h, m1, l1) * attn_gate(s, q, row0 + r1, h) : 0.f;
-    const size_t opitch = (size_t)s.heads * DV;
+    const size_t opitch = attn_out_stride(s);
 #pragma unroll
     for (int n = 0; n < NTH; ++n) {
-        const size_t col = (size_t)h * DV + vh * (DV / 2) + 8 * n + 2 * t;
+        const int c = vh * (DV / 2) + 8 * n + 2 * t;
+        if (!SIZED && c >= dv) continue;   // (dv in fours)
+        const size_t col = (size_t)h * dv + c;
         if (r0 < M) *reinterpret_cast<float2*>(out + (size_t)(row0 + r0) * opitch + col) = make_float2(o[n][0] * i0, o[n][1] * i0);
         if (r1 < M) *reinterpret_cast<float2*>(out + (size_t)(row0 + r1) * opitch + col) = make_float2(o[n][2] * i1, o[n][3] * i1);
     }

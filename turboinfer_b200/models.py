@@ -24,6 +24,10 @@ reads folder/config.json and folder/model.safetensors.  Registered architectures
                   turn-dependent frequencies side by side with a state-space recurrence, causal attention with sigmoid weights, capped
                   scores and normed queries / keys, gated linear attention; a clamped gated feed-forward or squared-relu experts chosen by
                   sigmoid scores inside the best groups; layers that use an earlier layer's tensors; on the layered sequence engine too.
+  * "Nubipel"  -- layers with one norm for both sublayers, too: grouped attention inside chunks of positions (no rotation, normed queries and
+                  keys, a softmax sink), latent attention without positions (low-rank queries, a sigmoid gate per output coordinate), the
+                  gated delta rule (a recurrence that writes what its state does not yet answer), a dense gelu feed-forward; logits
+                  tied to the embedding table, scaled and capped; on the layered sequence engine too.
   * "llama"    -- the quantized Llama-style decoder of the persistent decode kernel (turboinfer_b200.capi.Model); built from
                   {"hidden", "layers", "heads", "inter", "vocab"} and fp32 tensors under the reference's names.
 """
@@ -406,6 +410,53 @@ def _load_sebudra(cfg: dict, weights: dict, dtype: str, max_tokens: int, max_seq
     mode = {"bfloat16": _seq.BF16, "float32": _seq.F32}[dtype]
     shapes = {k: tuple(getattr(v, "shape", ())) for k, v in weights.items()}
     desc, layers = sebudra_descs(cfg, mode, max_tokens, max_seqs, shapes)
+    return _seq.SeqModel(desc, layers).load(weights)
+
+
+def nubipel_descs(cfg: dict, mode: int, max_tokens: int, max_seqs: int):
+    """config.json of a Nubipel model -> (ModelDesc, [LayerDesc]).  Every size and constant comes from the configuration."""
+    layers: List[_seq.LayerDesc] = []
+    for i, L in enumerate(_req(cfg, "layers", "the model")):
+        where = f"layer {i}"
+        kind = _req(L, "type", where)
+        mx = _req(L, "mixer", where)
+        d = _seq.LayerDesc()
+        d.heads, d.dim, d.vdim = int(_req(mx, "heads", where)), int(_req(mx, "dim", where)), int(_req(mx, "vdim", where))
+        if kind == "attention":
+            d.mixer, d.qk_norm, d.sink = _seq.MIXER_ATTENTION, _seq.QK_NORM_HEAD_GAIN, _seq.SINK_LEARNED
+            d.kv_heads, d.scale = int(_req(mx, "kv_heads", where)), float(_req(mx, "scale", where))
+            mask = mx.get("mask")
+            d.chunk = int(_req(mask, "size", where + " mask")) if mask else 0
+            if mask and d.chunk < 1:
+                raise ValueError(f"{where}: mask.size {d.chunk}")
+        elif kind == "latent_attention":
+            d.mixer, d.kv_heads, d.out_gate = _seq.MIXER_LATENT, d.heads, _seq.GATE_ELEMENT
+            d.kv_rank, d.q_rank, d.scale = int(_req(mx, "kv_rank", where)), int(_req(mx, "q_rank", where)), float(_req(mx, "scale", where))
+        elif kind == "delta":
+            d.mixer, d.kv_heads, d.mix_taps = _seq.MIXER_DELTA, int(_req(mx, "kv_heads", where)), int(_req(mx, "conv", where))
+        else:
+            raise ValueError(f"{where}: unknown mixer type '{kind}'")
+        mlp = L.get("mlp")
+        if mlp:
+            if _req(mlp, "kind", where + " mlp") != "dense":
+                raise ValueError(f"{where}: unknown feed-forward kind '{mlp.get('kind')}'")
+            d.ff_kind, d.ff_act, d.ff = _seq.FF_DENSE, _seq.ACT_GELU, int(_req(mlp, "ff", where + " mlp"))
+        layers.append(d)
+    m = _seq.ModelDesc()
+    m.vocab, m.width, m.n_layers = int(_req(cfg, "vocab", "the model")), int(_req(cfg, "width", "the model")), len(layers)
+    m.norm_eps = float(_req(_req(cfg, "norm", "the model"), "eps", "norm"))
+    m.norm_kind, m.norm_place = _seq.NORM_VECTOR, _seq.NORMS_SHARED
+    m.embed_scale = float(_req(_req(cfg, "embedding", "the model"), "scale", "embedding"))
+    m.logit_scale, m.logit_softcap = float(_req(cfg, "logit_scale", "the model")), float(_req(cfg, "logit_softcap", "the model"))
+    m.tied_head = 1
+    m.mode, m.max_tokens, m.max_seqs = mode, int(max_tokens), int(max_seqs)
+    return m, layers
+
+
+@register("Nubipel")
+def _load_nubipel(cfg: dict, weights: dict, dtype: str, max_tokens: int, max_seqs: int):
+    mode = {"bfloat16": _seq.BF16, "float32": _seq.F32}[dtype]
+    desc, layers = nubipel_descs(cfg, mode, max_tokens, max_seqs)
     return _seq.SeqModel(desc, layers).load(weights)
 
 

@@ -11,8 +11,8 @@ import numpy as np
 
 HERE = os.path.dirname(os.path.abspath(__file__))
 BF16, F32 = 0, 1
-MIXER_ATTENTION, MIXER_WKV, MIXER_GLA, MIXER_HGRN2, MIXER_LATENT, MIXER_SSM = 0, 1, 2, 3, 4, 5
-ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_XIELU, ACT_CLAMPED_SWISH = 0, 1, 2, 3, 4
+MIXER_ATTENTION, MIXER_WKV, MIXER_GLA, MIXER_HGRN2, MIXER_LATENT, MIXER_SSM, MIXER_DELTA = 0, 1, 2, 3, 4, 5, 6
+ACT_RELU, ACT_SILU, ACT_GELU_TANH, ACT_XIELU, ACT_CLAMPED_SWISH, ACT_GELU = 0, 1, 2, 3, 4, 5
 FF_GLU, FF_POLYNORM, FF_EXPERTS, FF_DENSE = 0, 1, 2, 3
 NORM_SCALAR, NORM_ONE_PLUS, NORM_VECTOR = 0, 1, 2
 SINK_NONE, SINK_LEARNED, SINK_ZERO = 0, 1, 2
@@ -20,6 +20,7 @@ ROUTE_SOFTMAX_ALL, ROUTE_TOP_LOGITS, ROUTE_SIGMOID = 0, 1, 2
 QK_NORM_NONE, QK_NORM_HEAD, QK_NORM_WHOLE, QK_NORM_HEAD_GAIN = 0, 1, 2, 3
 NORMS_AROUND, NORMS_BEHIND, NORMS_FRONT, NORMS_SHARED = 0, 1, 2, 3
 WEIGHTS_SOFTMAX, WEIGHTS_SIGMOID = 0, 1
+GATE_NONE, GATE_HEAD, GATE_ELEMENT = 0, 1, 2
 BIAS_NONE, BIAS_QKVO, BIAS_QKV = 0, 1, 2
 EXPERT_GATED, EXPERT_RELU2 = 0, 1
 ROT_BY_WAVELENGTH, ROT_BY_TURNS = 1, 2
@@ -43,7 +44,7 @@ class LayerDesc(C.Structure):
                 ("head_temp", C.c_int32), ("q_rank", C.c_int32), ("weights_kind", C.c_int32), ("rot_amp", C.c_float),
                 ("ssm_heads", C.c_int32), ("ssm_vdim", C.c_int32), ("ssm_state", C.c_int32), ("ssm_groups", C.c_int32), ("ssm_taps", C.c_int32),
                 ("ssm_parts", C.c_int32), ("left_scale", C.c_float), ("right_scale", C.c_float), ("ff_limit", C.c_float),
-                ("expert_form", C.c_int32), ("route_scale", C.c_float), ("weights_of", C.c_int32)]
+                ("expert_form", C.c_int32), ("route_scale", C.c_float), ("weights_of", C.c_int32), ("chunk", C.c_int32), ("mix_taps", C.c_int32)]
 
     def __init__(self, *a, **kw):
         super().__init__(*a, **kw)
