@@ -111,6 +111,23 @@ def sebudra_config_for(size: str) -> dict:
     return {"architecture": "Sebudra", "embedding": {"scale": math.sqrt(D)}, "layers": order, "norm": {"eps": 1e-6}, "vocab": z["vocab"], "width": D}
 
 
+def nubipel_config_for(size: str) -> dict:
+    """Seven layers in the order latent attention, delta, attention, latent attention, delta, attention, latent attention, each with a
+    dense gelu feed-forward of the size's inner width.  Latent attention: the size's heads of 128 over all earlier tokens, a cached row of
+    256, queries through a vector of 3/8 of the width; delta: the size's heads of 128 x 128 with half as many query / key heads, four
+    taps; attention: the size's heads inside chunks of the size's window."""
+    z = SIZES[size]
+    D, H, d = z["width"], z["heads"], z["dim"]
+    mlp = {"kind": "dense", "ff": z["ff"]}
+    lat = {"type": "latent_attention", "mlp": mlp,
+           "mixer": {"heads": H, "dim": d, "vdim": d, "kv_rank": 256, "q_rank": 3 * D // 8, "scale": 1.0 / math.sqrt(d)}}
+    delta = {"type": "delta", "mlp": mlp, "mixer": {"heads": H, "kv_heads": H // 2, "dim": d, "vdim": d, "conv": 4}}
+    att = {"type": "attention", "mlp": mlp,
+           "mixer": {"heads": H, "kv_heads": z["kv_heads"], "dim": d, "vdim": d, "mask": {"size": z["window"]}, "scale": 1.0 / math.sqrt(d)}}
+    return {"architecture": "Nubipel", "embedding": {"scale": math.sqrt(D)}, "layers": [lat, delta, att, lat, delta, att, lat], "norm": {"eps": 1e-6},
+            "logit_scale": 0.5, "logit_softcap": 30.0, "vocab": z["vocab"], "width": D}
+
+
 def build_synthetic(cfg: dict, rank: int, dtype: str, max_tokens: int, max_seqs: int) -> seq.SeqModel:
     mode = {"bfloat16": seq.BF16, "float32": seq.F32}[dtype]
     if cfg["architecture"] == "Gulazen":
@@ -124,6 +141,8 @@ def build_synthetic(cfg: dict, rank: int, dtype: str, max_tokens: int, max_seqs:
     elif cfg["architecture"] == "Sebudra":
         shapes = {f"l{i}.mix.a1": (rank, cfg["width"]) for i, L in enumerate(cfg["layers"]) if L["type"] == "gla"}
         desc, layers = models.sebudra_descs(cfg, mode, max_tokens, max_seqs, shapes)
+    elif cfg["architecture"] == "Nubipel":
+        desc, layers = models.nubipel_descs(cfg, mode, max_tokens, max_seqs)
     else:
         shapes = {f"l{i}.mix.w1": (rank, cfg["width"]) for i, L in enumerate(cfg["layers"]) if L["type"] == "wkv"}
         desc, layers = models.binusun_descs(cfg, mode, max_tokens, max_seqs, shapes)
@@ -140,6 +159,10 @@ def build_synthetic(cfg: dict, rank: int, dtype: str, max_tokens: int, max_seqs:
             amp, off = 0.25, 1.0   # plain gains around one
         elif cfg["architecture"] == "Sebudra" and leaf in ("dt_bias", "A_log", "pb", "correction", "b"):
             amp, off = 0.5, {"dt_bias": -3.0, "pb": -4.0}.get(leaf, 0.0)
+        elif cfg["architecture"] == "Nubipel" and leaf in ("norm1", "norm"):
+            amp, off = 0.25, 1.0   # plain gains around one
+        elif cfg["architecture"] == "Nubipel" and leaf in ("dt_bias", "A_log"):
+            amp, off = 0.5, -3.0 if leaf == "dt_bias" else 0.0
         elif leaf in ("in", "out") and ".hc" in name:
             amp, off = 0.2, 0.6
         elif leaf == "mix" and ".hc" in name:
@@ -182,7 +205,7 @@ def prompt(n: int, vocab: int, offset: int = 0):
 
 def measure_seq(size: str, dtype: str, n_prompt: int, n_new: int, batch: int, steps: int, warmup: int, design: str = "Binusun") -> dict:
     cfg = {"Tudasun": tudasun_config_for, "Gulazen": gulazen_config_for, "BinusunAttention": binusun_attention_config_for,
-           "Zopipel": zopipel_config_for, "Sebudra": sebudra_config_for}.get(design, config_for)(size)
+           "Zopipel": zopipel_config_for, "Sebudra": sebudra_config_for, "Nubipel": nubipel_config_for}.get(design, config_for)(size)
     m = build_synthetic(cfg, SIZES[size]["rank"], dtype, max_tokens=(n_prompt + n_new + 64) * max(batch, 1) + 64, max_seqs=max(batch, 1))
     V = cfg["vocab"]
     launches0 = seq.launch_count()
@@ -283,6 +306,17 @@ def compare_sebudra(size: str, steps: int, warmup: int, n_prompt: int = 2048, n_
     out = {"size": size, "shape": SIZES[size], "prompt_tokens": n_prompt, "decode_steps": n_new}
     for design in ("Sebudra", "Tudasun", "BinusunAttention"):
         key = {"BinusunAttention": "binusun_attention"}.get(design, design.lower()) + "_bf16"
+        out[key] = measure_seq(size, "bfloat16", n_prompt, n_new, 1, steps, warmup, design)
+        out[key + "_batch4"] = {k: v for k, v in measure_seq(size, "bfloat16", 256, n_new, 4, 1, 1, design).items() if k.startswith("decode") or k == "batch"}
+    return out
+
+
+def compare_nubipel(size: str, steps: int, warmup: int, n_prompt: int = 2048, n_new: int = 64) -> dict:
+    """Nubipel next to the library's closest models on the same engine (bf16 weights all): Sebudra (one norm for both sublayers, softmax attention
+    and recurrences) and Tudasun (latent attention and recurrences)."""
+    out = {"size": size, "shape": SIZES[size], "prompt_tokens": n_prompt, "decode_steps": n_new}
+    for design in ("Nubipel", "Sebudra", "Tudasun"):
+        key = design.lower() + "_bf16"
         out[key] = measure_seq(size, "bfloat16", n_prompt, n_new, 1, steps, warmup, design)
         out[key + "_batch4"] = {k: v for k, v in measure_seq(size, "bfloat16", 256, n_new, 4, 1, 1, design).items() if k.startswith("decode") or k == "batch"}
     return out

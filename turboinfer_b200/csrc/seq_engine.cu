@@ -2272,20 +2272,20 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
         } else {   // latent attention
             const int H = L.d.heads, kd = L.d.kv_rank + L.d.rot_dims;
             if (!shared) {
-            std::vector<int> off;
-            TRY(concat_rows(m, {T(p + (L.d.q_rank > 0 ? "mix.dq" : "mix.q")), L.d.kv_from < 0 ? T(p + "mix.dkv") : nullptr, L.d.res_gate ? T(p + "rg1") : nullptr,
-                                L.d.out_gate ? T(p + "mix.g") : nullptr}, L.front_buf, &L.n_front, &off));
-            L.front = L.front_buf.p;
-            L.off_q = off[0]; L.off_dkv = off[1]; L.off_rg1 = off[2]; L.off_g = off[3];
-            L.ld_front = L.n_front;
-            if (L.d.q_rank > 0) {   // the queries come from a second product and sit behind the first one's columns
-                L.off_dq = off[0];
-                L.off_q = L.n_front;
-                L.ld_front = L.n_front + H * (L.d.dim + L.d.rot_dims);
-            }
-            rg1_fused = L.d.res_gate != 0;
-            for (const char* s : {"mix.q", "mix.dq", "mix.dkv", "rg1", "mix.g"}) release(p + s);
-            L.o = P(p + "mix.o");
+                std::vector<int> off;
+                TRY(concat_rows(m, {T(p + (L.d.q_rank > 0 ? "mix.dq" : "mix.q")), L.d.kv_from < 0 ? T(p + "mix.dkv") : nullptr, L.d.res_gate ? T(p + "rg1") : nullptr,
+                                    L.d.out_gate ? T(p + "mix.g") : nullptr}, L.front_buf, &L.n_front, &off));
+                L.front = L.front_buf.p;
+                L.off_q = off[0]; L.off_dkv = off[1]; L.off_rg1 = off[2]; L.off_g = off[3];
+                L.ld_front = L.n_front;
+                if (L.d.q_rank > 0) {   // the queries come from a second product and sit behind the first one's columns
+                    L.off_dq = off[0];
+                    L.off_q = L.n_front;
+                    L.ld_front = L.n_front + H * (L.d.dim + L.d.rot_dims);
+                }
+                rg1_fused = L.d.res_gate != 0;
+                for (const char* s : {"mix.q", "mix.dq", "mix.dkv", "rg1", "mix.g"}) release(p + s);
+                L.o = P(p + "mix.o");
             }
             if (L.d.q_rank > 0) {
                 L.uq = P(p + "mix.uq");
