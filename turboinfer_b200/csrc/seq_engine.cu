@@ -268,6 +268,7 @@ struct Model {
     DevBuf<__nv_bfloat16> abf;   // bf16 copy of a product's activations for the tcgen05 path: [rows][max_k]
     DevBuf<int> attn_arrived;    // split-key attention: finished splits of a (row, head), zero between launches
     DevBuf<float> attn_part;     // split-key attention partials: [rows][heads][splits][vdim + 2]
+    DevBuf<float> delta_buf;     // delta rule in chunks: Wk, Wv, A and three factors a row, per head
     DevBuf<float> mix_S, mix_den; // head-mixing attention: scores / weights [rows of a batch][heads][keys], 1 / denominators [rows][heads]
     bool any_mixed = false;
     int max_heads_v = 0;         // max over attention layers of heads * (vdim + 2)
@@ -1316,7 +1317,24 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         LAUNCHED();
         return 0;
     };
-    auto delta_scan = [&](const DeltaArgs& a) -> int {
+    auto delta_scan = [&](DeltaArgs a) -> int {
+        // portions of kAttnTiledMinRows rows and more in chunks (their tiles are the attention's), the other entries token by token
+        if (n_tiles > 0 && a.dk % 4 == 0 && a.dk <= kDeltaChunkMaxKey && a.ld % 4 == 0) {
+            const size_t rows = (size_t)T * a.heads;
+            TRY(m.delta_buf.ensure(rows * (size_t)(a.dk + (a.dv + 3) / 4 * 4 + kDeltaChunk + 3)));
+            DeltaChunkArgs c{};
+            c.d = a; c.tiles = d_tiles; c.min_rows = kAttnTiledMinRows;
+            c.wk = m.delta_buf.p; c.am = c.wk + rows * a.dk; c.wv = c.am + rows * kDeltaChunk; c.sq = c.wv + rows * ((a.dv + 3) / 4 * 4); c.sk = c.sq + rows; c.eg = c.sk + rows;
+            const dim3 pg(n_tiles, a.heads), sg(E, a.heads, (a.dv + kDeltaCols - 1) / kDeltaCols);
+            if (a.dk <= 64) TRY(launch_dep(delta_chunk_prepare_kernel<64>, pg, dim3(256), delta_prepare_smem_bytes<64>(), c, sm));
+            else TRY(launch_dep(delta_chunk_prepare_kernel<128>, pg, dim3(256), delta_prepare_smem_bytes<128>(), c, sm));
+            LAUNCHED();
+            if (a.dk <= 64) TRY(launch_dep(delta_chunk_scan_kernel<64>, sg, dim3(256), delta_chunk_smem_bytes<64>(), c, sm));
+            else TRY(launch_dep(delta_chunk_scan_kernel<128>, sg, dim3(256), delta_chunk_smem_bytes<128>(), c, sm));
+            LAUNCHED();
+            if (n_small == 0) return 0;
+            a.max_rows = kAttnTiledMinRows - 1;
+        }
         const dim3 grid(E, a.heads, (a.dv + kDeltaCols - 1) / kDeltaCols);
         if (a.dk <= 32) TRY(launch_dep(delta_scan_kernel<4, 8>, grid, dim3(128), 0, a, sm));
         else if (a.dk <= 64) TRY(launch_dep(delta_scan_kernel<8, 8>, grid, dim3(128), 0, a, sm));
@@ -1965,6 +1983,10 @@ int ti_seq_init(int device) {
     TI_LAT_ATTR(512, 512, 32, true);
     TI_LAT_ATTR(512, 512, 32, false);
 #undef TI_LAT_ATTR
+    CK(cudaFuncSetAttribute(delta_chunk_prepare_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)delta_prepare_smem_bytes<64>()));
+    CK(cudaFuncSetAttribute(delta_chunk_prepare_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)delta_prepare_smem_bytes<128>()));
+    CK(cudaFuncSetAttribute(delta_chunk_scan_kernel<64>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)delta_chunk_smem_bytes<64>()));
+    CK(cudaFuncSetAttribute(delta_chunk_scan_kernel<128>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)delta_chunk_smem_bytes<128>()));
     CK(cudaFuncSetAttribute(mix_scores_tiles_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(mix_scores_tiles_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
     CK(cudaFuncSetAttribute(mix_scores_rows_kernel<kAttnMaxPerLane>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)g_smem_optin));
