@@ -207,6 +207,12 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
 #pragma unroll
     for (int n = 0; n < NT; ++n) {
         const int c = 8 * n + 2 * t;
+        if (s.egate && c < dv) {
+            const float* eg = s.egate + (size_t)(row0 + r0) * s.egate_ld + (size_t)h * dv + c;
+            if (r0 < M) { o[n][0] *= sigmoid_f32(eg[0]); o[n][1] *= sigmoid_f32(eg[1]); }
+            eg += (size_t)8 * s.egate_ld;
+            if (r1 < M) { o[n][2] *= sigmoid_f32(eg[0]); o[n][3] *= sigmoid_f32(eg[1]); }
+        }
         if (pair) {
             if (r0 < M) *reinterpret_cast<float2*>(o0 + c) = make_float2(o[n][0] * i0, o[n][1] * i0);
             if (r1 < M) *reinterpret_cast<float2*>(o1 + c) = make_float2(o[n][2] * i1, o[n][3] * i1);

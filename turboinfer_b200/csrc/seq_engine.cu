@@ -209,6 +209,7 @@ struct LayerW {
     DevBuf<float> qkv_bias, sink_zero;         // biases of the fused [q | k | v] product side by side; zeros [heads]
     const float *o_bias = nullptr, *temp = nullptr, *canon2 = nullptr, *dqnorm = nullptr;
     const void* uq = nullptr;
+    const void* uk = nullptr;                  // latent attention: the key up-projection itself, where prompt portions may expand their keys
     int off_dq = -1, ld_front = 0;             // ld_front: row stride of the fused front product's output (>= n_front: room for q behind it)
     const float *hc_in[2] = {nullptr, nullptr}, *hc_out[2] = {nullptr, nullptr}, *hc_mix[2] = {nullptr, nullptr};
     // norms in front of both sublayers at once: `front` is [mixer parts | second mixer's in | feed-forward front], `back` the output
@@ -271,6 +272,10 @@ struct Model {
     DevBuf<float> delta_buf;     // delta rule in chunks: Wk, Wv, A and three factors a row, per head
     DevBuf<float> mix_S, mix_den; // head-mixing attention: scores / weights [rows of a batch][heads][keys], 1 / denominators [rows][heads]
     bool any_mixed = false;
+    bool any_expand = false;     // latent attention of prompt portions on expanded keys and values
+    DevBuf<float> kx, vx;        // ... of all cached tokens of the step's portions, page after page: [rows][heads * dim], [rows][heads * vdim]
+    DevBuf<__nv_bfloat16> cx;    // ... and the rows they come from: [rows][rank]
+    DevBuf<__nv_bfloat16> act16; // rows of the back product as bf16 (one norm for both sublayers, dense feed-forward)
     int max_heads_v = 0;         // max over attention layers of heads * (vdim + 2)
     DevBuf<int> err;             // device flag: a bounded wait in a kernel ran out
     int max_k = 0;
@@ -670,7 +675,7 @@ __global__ void add_one_kernel(float* w, size_t n) {
 // ---- tensor maps for the tcgen05 path: a bf16 matrix [rows][cols], cols contiguous, boxes of 64 x 128 with the 128-byte swizzle ----
 typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t, void*, const cuuint64_t*, const cuuint64_t*, const cuuint32_t*,
                                   const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle, CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-int make_tmap_bf16(CUtensorMap* map, const void* base, uint64_t cols, uint64_t rows) {
+int make_tmap_bf16(CUtensorMap* map, const void* base, uint64_t cols, uint64_t rows, uint64_t pitch) {   // pitch: elements between rows
     static EncodeTiledFn fn = nullptr;
     if (!fn) {
         void* p = nullptr;
@@ -680,7 +685,7 @@ int make_tmap_bf16(CUtensorMap* map, const void* base, uint64_t cols, uint64_t r
         fn = reinterpret_cast<EncodeTiledFn>(p);
     }
     const cuuint64_t dims[2] = {cols, rows};
-    const cuuint64_t strides[1] = {cols * 2};
+    const cuuint64_t strides[1] = {pitch * 2};
     const cuuint32_t box[2] = {(cuuint32_t)kSgBK, (cuuint32_t)kSgBM};
     const cuuint32_t estr[2] = {1, 1};
     const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, estr, CU_TENSOR_MAP_INTERLEAVE_NONE,
@@ -721,6 +726,22 @@ struct Fuse {
 };
 bool few_rows(int M, int K) { return M <= kRowGemvMaxRows && (size_t)M * K * sizeof(float) <= g_smem_optin; }
 
+// prompt-sized products in bf16 mode run on tcgen05 (TMA wants 16-byte row pitches and bases)
+bool tc_ok(const Model& m, const void* W, int M, int N, int K) {
+    return m.d.mode == TI_SEQ_BF16 && g_use_tc && M > 32 && N >= 64 && K >= 64 && K % 8 == 0 && (reinterpret_cast<uintptr_t>(W) & 15) == 0;
+}
+int gemm_tc(Model& m, const __nv_bfloat16* A, int lda, const void* W, float* C, int ldc, int M, int N, int K, int epi = EPI_NONE, float alpha = 1.f, float beta = 0.f,
+            const GluCols* cols = nullptr) {
+    CUtensorMap ma, mw;
+    TRY(make_tmap_bf16(&ma, A, (uint64_t)K, (uint64_t)M, (uint64_t)lda));
+    TRY(make_tmap_bf16(&mw, W, (uint64_t)K, (uint64_t)N, (uint64_t)K));
+    TcArgs g{};
+    g.M = M; g.N = N; g.K = K; g.C = C; g.ldc = ldc; g.epi = epi; g.alpha = alpha; g.beta = beta; g.err = m.err.p;
+    if (cols) g.cols = *cols;
+    gemm_bf16_tc_kernel<<<dim3((N + kSgBN - 1) / kSgBN, (M + kSgBM - 1) / kSgBM), kSgThreads, kSgSmemBytes, g_stream>>>(ma, mw, g);
+    LAUNCHED();
+    return 0;
+}
 int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, int M, int N, int K, int epi = EPI_NONE, float alpha = 1.f,
          const Fuse* fuse = nullptr, float beta = 0.f) {
     if (M <= 0 || N <= 0) return 0;
@@ -791,20 +812,10 @@ int gemm(Model& m, const float* A, int lda, const void* W, float* C, int ldc, in
         return 0;
     }
     if (!plain && (!single || fuse->norm_gain)) return fail("internal: a fused product was asked for on the many-row path");
-    // prompt-sized products in bf16 mode: tcgen05 (TMA wants 16-byte row pitches and bases)
-    if (m.d.mode == TI_SEQ_BF16 && g_use_tc && M > 32 && N >= 64 && K >= 64 && K % 8 == 0 && (reinterpret_cast<uintptr_t>(W) & 15) == 0 && m.abf.p &&
-        (size_t)M * K <= m.abf.n) {
-        rows_to_bf16_kernel<<<grid_for((size_t)M * K / 4), 256, 0, g_stream>>>(A, lda, M, K, m.abf.p);
+    if (tc_ok(m, W, M, N, K) && m.abf.p && (size_t)M * K <= m.abf.n) {
+        rows_to_bf16_kernel<<<grid_for((size_t)M * K / 4), 256, 0, g_stream>>>(A, lda, M, K, m.abf.p, K);
         LAUNCHED();
-        CUtensorMap ma, mw;
-        TRY(make_tmap_bf16(&ma, m.abf.p, (uint64_t)K, (uint64_t)M));
-        TRY(make_tmap_bf16(&mw, W, (uint64_t)K, (uint64_t)N));
-        TcArgs g{};
-        g.M = M; g.N = N; g.K = K; g.C = C; g.ldc = ldc; g.epi = epi; g.alpha = alpha; g.beta = beta; g.err = m.err.p;
-        if (single) g.cols = fuse->glu;
-        gemm_bf16_tc_kernel<<<dim3((N + kSgBN - 1) / kSgBN, (M + kSgBM - 1) / kSgBM), kSgThreads, kSgSmemBytes, g_stream>>>(ma, mw, g);
-        LAUNCHED();
-        return 0;
+        return gemm_tc(m, m.abf.p, K, W, C, ldc, M, N, K, epi, alpha, beta, single ? &fuse->glu : nullptr);
     }
     dim3 grid((N + 63) / 64, (M + 63) / 64);
     if (m.d.mode == TI_SEQ_BF16) gemm_bf16_kernel<<<grid, 128, 0, g_stream>>>(A, lda, (const __nv_bfloat16*)W, C, ldc, M, N, K, epi, alpha, beta, 0, 0, 0, nullptr, 0);
@@ -871,6 +882,7 @@ int ensure_scratch(Model& m, int rows, int want) {
         if (m.any_rgbuf) TRY(m.rgbuf.alloc(R * D));
         if (m.dbg) TRY(m.dbg_buf.alloc(m.runs.size() * R * D));
         if (m.d.mode == TI_SEQ_BF16 && g_use_tc) TRY(m.abf.alloc(R * (size_t)m.max_k));
+        if (m.d.mode == TI_SEQ_BF16 && g_use_tc && m.d.norm_place == TI_SEQ_NORMS_SHARED) TRY(m.act16.alloc(R * (size_t)m.max_ff));
         if (m.max_heads_v) {
             TRY(m.attn_part.alloc(R * (size_t)m.max_heads_v * kAttnMaxSplits));
             TRY(m.attn_arrived.alloc(R * (size_t)m.max_heads_v));
@@ -999,8 +1011,29 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         }
     }
     const int n_mtiles = (int)mtiles.size() / 2;
+    // latent attention on expanded keys and values: the portions' pages one after another, and the rows of the other entries in runs
+    std::vector<int> xpages, xfirst(E, -1), small_runs;
+    double xpairs = 0;
+    if (m.any_expand && n_tiles > 0) {
+        int r0 = 0;
+        for (int e = 0; e < E; ++e) {
+            const SeqState& s = m.seqs[seqs[e]];
+            if (counts[e] >= kAttnTiledMinRows) {
+                xfirst[e] = (int)xpages.size();
+                xpages.insert(xpages.end(), s.pages.begin(), s.pages.begin() + (s.len + counts[e] + kPageTokens - 1) / kPageTokens);
+                xpairs += (double)counts[e] * (s.len + 0.5 * (counts[e] + 1));
+            } else if (!small_runs.empty() && small_runs[small_runs.size() - 2] + small_runs.back() == r0) {
+                small_runs.back() += counts[e];
+            } else {
+                small_runs.push_back(r0);
+                small_runs.push_back(counts[e]);
+            }
+            r0 += counts[e];
+        }
+    }
+    const size_t n_xtable = xpages.empty() ? 0 : (size_t)m.seqs.size() * stride;
     const size_t n_meta = (size_t)3 * T + (size_t)(E + 1) + 2 * (size_t)E + (size_t)std::max(n_out, 1) + (size_t)m.seqs.size() * stride +
-                          (size_t)3 * T + 4 + mtiles.size() + row_tile.size();
+                          (size_t)3 * T + 4 + mtiles.size() + row_tile.size() + xpages.size() + n_xtable;
     if (n_meta > m.meta_host_cap) {
         if (m.meta_host) cudaFreeHost(m.meta_host);
         m.meta_host = nullptr;
@@ -1042,6 +1075,14 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
     std::copy(mtiles.begin(), mtiles.end(), h_mtiles);
     int* h_row_tile = h_mtiles + mtiles.size();
     std::copy(row_tile.begin(), row_tile.end(), h_row_tile);
+    int* h_xpages = h_row_tile + row_tile.size();
+    std::copy(xpages.begin(), xpages.end(), h_xpages);
+    int* h_xtable = h_xpages + xpages.size();   // the page table of the expanded rows
+    if (n_xtable) {
+        std::fill(h_xtable, h_xtable + n_xtable, 0);
+        for (int e = 0; e < E; ++e)
+            for (int p = 0; xfirst[e] >= 0 && p < (int)m.seqs[seqs[e]].pages.size(); ++p) h_xtable[(size_t)seqs[e] * stride + p] = xfirst[e] + p;
+    }
     // the previous step's copy out of this pinned buffer has completed: every step ends with a stream synchronisation
     CK(cudaMemcpyAsync(m.meta.p, hp, n_meta * sizeof(int), cudaMemcpyHostToDevice, g_stream));
     StepMeta sm{};
@@ -1058,6 +1099,8 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
     const int* d_tiles128 = d_small + small_rows.size();
     const int* d_mtiles = d_tiles128 + tiles128.size();
     const int* d_row_tile = d_mtiles + mtiles.size();
+    const int* d_xpages = d_row_tile + row_tile.size();
+    const int* d_xtable = d_xpages + xpages.size();
     sm.table_stride = stride;
     sm.T = T;
     sm.E = E;
@@ -1165,20 +1208,36 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
     };
     if (front) TRY(hyper(0, -1));
     // paged softmax attention of all rows of the step (prompt portions in tiles, the other rows one by one or split over their keys)
-    auto attention = [&](const AttnShape& s, const float* q, const float* kp, const float* vp, float* out) -> int {
+    auto h3_size = [](const AttnShape& s) { return s.dim <= 128 && s.vdim <= 128 && s.dim % 4 == 0 && s.vdim % 4 == 0 && s.v_ld == 0; };
+    auto h3_attention = [&](const StepMeta& sm, const AttnShape& s, const float* q, const float* kp, const float* vp, float* out) -> int {   // the portions' tiles
+        const dim3 grid(n_tiles128, s.heads);
+        const int dk = s.dim <= 64 ? 64 : 128, dv = s.vdim <= 64 ? 64 : 128;
+        const bool sized = dk == s.dim && dv == s.vdim;
+#define TI_H3_CASE(K, V, X) window_attention_h3_kernel<K, V, X><<<grid, kTcThreads, window_h3_smem_bytes<K, V>(), g_stream>>>(q, sm, s, d_tiles128, kp, vp, out)
+        if (dk == 64 && dv == 64) { if (sized) TI_H3_CASE(64, 64, true); else TI_H3_CASE(64, 64, false); }
+        else if (dk == 128 && dv == 128) { if (sized) TI_H3_CASE(128, 128, true); else TI_H3_CASE(128, 128, false); }
+        else if (dk == 64) TI_H3_CASE(64, 128, false);
+        else TI_H3_CASE(128, 64, false);
+#undef TI_H3_CASE
+        LAUNCHED();
+        return 0;
+    };
+    auto attention = [&](const AttnShape& s, const float* q, const float* kp, const float* vp, float* out, bool only_small = false) -> int {   // (only_small: not the portions)
         const bool wide = std::max(s.dim, s.vdim) > 32 * kAttnMaxPerLane;
         const size_t smem = ((size_t)kAttnWarps * s.vdim + 2 * kAttnWarps) * sizeof(float);
         const bool v_in_k = kp == vp && s.kv_heads == 1 && s.v_ld == s.dim && s.vdim <= s.dim;
         const size_t tsmem = attn_tiled_smem_bytes(s.dim, s.vdim, v_in_k);
         const bool tiled_ok = g_use_tiled_attn && n_tiles > 0 && s.dim % 4 == 0 && s.vdim % 4 == 0 && s.vdim <= 512 && tsmem <= g_smem_optin && (s.v_ld % 4 == 0);
         // bf16 mode, head sizes up to 128 in fours: the split-half tensor-core kernel (fp32-accurate); fp32 mode keeps true fp32 arithmetic
-        const bool h3_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles128 > 0 && s.dim <= 128 && s.vdim <= 128 && s.dim % 4 == 0 && s.vdim % 4 == 0 && s.v_ld == 0;
+        const bool h3_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles128 > 0 && h3_size(s);
         // bf16 mode, a shared key/value head with the values inside the key rows (latent attention), instantiated sizes: tensor cores
         const bool lat_size = (s.dim == 320 && s.vdim == 256) || (s.dim == 192 && s.vdim == 128) || (s.dim == 160 && s.vdim == 128) || (s.dim == s.vdim && s.dim % 4 == 0 && s.dim <= 512);
         const bool lat_ok = g_use_tiled_attn && g_use_tc && bf && n_tiles > 0 && v_in_k && (!s.out_gate || s.gate) && !s.qk_norm && lat_size;
-        const int* rest = (tiled_ok || h3_ok || lat_ok) ? d_small : nullptr;
-        const int n_rest = (tiled_ok || h3_ok || lat_ok) ? n_small : T;
-        if (lat_ok) {
+        const bool split_rows = only_small || tiled_ok || h3_ok || lat_ok;
+        const int* rest = split_rows ? d_small : nullptr;
+        const int n_rest = split_rows ? n_small : T;
+        if (only_small) {
+        } else if (lat_ok) {
             const dim3 grid(n_tiles, s.heads);
 #define TI_LAT_CASE(K, V, KT, X) latent_attention_h3_kernel<K, V, KT, X><<<grid, 256, latent_h3_smem_bytes<K, KT>(), g_stream>>>(q, sm, s, d_tiles, kp, out)
             if (s.dim == s.vdim) {   // no rotated part: rows of up to 512 in fours, padded to 128 / 256 / 512
@@ -1194,16 +1253,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
 #undef TI_LAT_CASE
             LAUNCHED();
         } else if (h3_ok) {
-            const dim3 grid(n_tiles128, s.heads);
-            const int dk = s.dim <= 64 ? 64 : 128, dv = s.vdim <= 64 ? 64 : 128;
-            const bool sized = dk == s.dim && dv == s.vdim;
-#define TI_H3_CASE(K, V, X) window_attention_h3_kernel<K, V, X><<<grid, kTcThreads, window_h3_smem_bytes<K, V>(), g_stream>>>(q, sm, s, d_tiles128, kp, vp, out)
-            if (dk == 64 && dv == 64) { if (sized) TI_H3_CASE(64, 64, true); else TI_H3_CASE(64, 64, false); }
-            else if (dk == 128 && dv == 128) { if (sized) TI_H3_CASE(128, 128, true); else TI_H3_CASE(128, 128, false); }
-            else if (dk == 64) TI_H3_CASE(64, 128, false);
-            else TI_H3_CASE(128, 64, false);
-#undef TI_H3_CASE
-            LAUNCHED();
+            TRY(h3_attention(sm, s, q, kp, vp, out));
         } else if (tiled_ok) {
             const dim3 grid(n_tiles, s.heads);
             if (s.vdim <= 64) window_attention_tiled_kernel<1><<<grid, 256, tsmem, g_stream>>>(q, sm, s, d_tiles, kp, vp, out);
@@ -1366,17 +1416,43 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         ls.rot_half = d.rot_half;
         TRY(launch_dep(latent_prepare_kernel, dim3(T), dim3(128), 0, (const float*)m.proj.p, sm, ls, (const float*)L.inv_freq.p, L.cnorm, pool, m.aux.p));
         LAUNCHED();
-        // the key up-projection moves to the query: qabs[t][h][0 .. rank) = Uk_h^T q_h
-        TRY(gemm_heads(m, m.proj.p + L.off_q, nf, d.dim + dr, L.ukT.p, m.aux.p, H * kd, kd, H, T, rank, d.dim));
         AttnShape s{};
         s.heads = H; s.kv_heads = 1; s.dim = kd; s.vdim = rank; s.window = d.window; s.chunk = d.chunk; s.rot_dims = 0; s.qk_norm = 0;
         s.scale = d.scale; s.eps = eps; s.ld = H * kd; s.v_ld = kd; s.sink = L.sink;
         // (a gate of one number a head commutes with the value up-projection behind the weighted sum; a gate per coordinate rides in its epilogue)
         const float* g = d.out_gate ? m.proj.p + L.off_g : nullptr;
         s.out_gate = d.out_gate == TI_SEQ_GATE_HEAD ? 1 : 0; s.gate = s.out_gate ? g : nullptr; s.gate_ld = nf;
+        const float* eg = d.out_gate == TI_SEQ_GATE_ELEMENT ? g : nullptr;
+        // the key up-projection moves to the query, qabs[t][h][0 .. rank) = Uk_h^T q_h; the value up-projection goes behind the weighted sum,
+        // out[t][h] = Uv_h (sum_j p_j c_j); rows r0 .. r0 + n - 1
+        auto to_latent = [&](int r0, int n) { return gemm_heads(m, m.proj.p + (size_t)r0 * nf + L.off_q, nf, d.dim + dr, L.ukT.p, m.aux.p + (size_t)r0 * H * kd, H * kd, kd, H, n, rank, d.dim); };
+        auto from_latent = [&](int r0, int n) {
+            return gemm_heads(m, m.aux2.p + (size_t)r0 * H * rank, H * rank, rank, L.uv, out + (size_t)r0 * ldo, ldo, d.vdim, H, n, d.vdim, rank, eg ? eg + (size_t)r0 * nf : nullptr, nf);
+        };
+        AttnShape x = s;   // the portions' form on expanded keys and values
+        x.kv_heads = H; x.dim = d.dim; x.vdim = d.vdim; x.v_ld = 0; x.ld = nf; x.out_ld = ldo; x.egate = eg; x.egate_ld = nf;
+        const size_t xrows = xpages.size() * kPageTokens;
+        const double direct = xpairs * 6.0 * (d.dim + d.vdim) + 0.4 * (double)xrows * rank * (d.dim + d.vdim);   // (0.4: two operations on tcgen05, a fifth of the time)
+        if (L.uk && xrows > 32 && g_use_tiled_attn && h3_size(x) && direct < xpairs * 12.0 * rank && (double)xrows * H * (d.dim + d.vdim) * 4 < 4e9) {
+            TRY(m.cx.ensure(xrows * rank));
+            TRY(m.kx.ensure(xrows * H * d.dim));
+            TRY(m.vx.ensure(xrows * H * d.vdim));
+            TRY(launch_dep(latent_gather_kernel, dim3(grid_for(xrows * rank / 4)), dim3(256), 0, (const float*)pool, kd, rank, d_xpages, (int)xrows, m.cx.p));
+            LAUNCHED();
+            TRY(gemm_tc(m, m.cx.p, rank, L.uk, m.kx.p, H * d.dim, (int)xrows, H * d.dim, rank));
+            TRY(gemm_tc(m, m.cx.p, rank, L.uv, m.vx.p, H * d.vdim, (int)xrows, H * d.vdim, rank));
+            StepMeta sx = sm;
+            sx.page_table = d_xtable;
+            TRY(h3_attention(sx, x, m.proj.p + L.off_q, m.kx.p, m.vx.p, out));
+            if (n_small == 0) return 0;
+            for (size_t i = 0; i < small_runs.size(); i += 2) TRY(to_latent(small_runs[i], small_runs[i + 1]));
+            TRY(attention(s, m.aux.p, pool, pool, m.aux2.p, true));
+            for (size_t i = 0; i < small_runs.size(); i += 2) TRY(from_latent(small_runs[i], small_runs[i + 1]));
+            return 0;
+        }
+        TRY(to_latent(0, T));
         TRY(attention(s, m.aux.p, pool, pool, m.aux2.p));
-        // ... and the value up-projection behind the weighted sum: out[t][h] = Uv_h (sum_j p_j c_j)
-        return gemm_heads(m, m.aux2.p, H * rank, rank, L.uv, out, ldo, d.vdim, H, T, d.vdim, rank, d.out_gate == TI_SEQ_GATE_ELEMENT ? g : nullptr, nf);
+        return from_latent(0, T);
     };
     auto route_shape = [&](const ti_seq_layer_desc& d) {
         RouteShape r{};
@@ -1418,9 +1494,13 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         const bool few = few_rows(T, D);
         Fuse fn;
         const float* in = m.x.p;
+        // many rows in bf16 mode: the norm leaves the front product's input as bf16, and so does a dense feed-forward's activation the back product's
+        const bool in16 = !few && tc_ok(m, L.front, T, L.n_front, D);
+        const bool out16 = in16 && F > 0 && d.ff_kind == TI_SEQ_FF_DENSE && L.back_ff % 8 == 0 && tc_ok(m, L.back, T, D, KB) && m.act16.p;
         if (few) { fn.norm_gain = L.norm1; fn.eps = eps; fn.gvec = gv; }
         else {
-            TRY(launch_dep(rmsnorm_kernel, dim3(T), dim3(nt), 0, (const float*)m.x.p, D, (const int*)nullptr, D, L.norm1, gv, eps, m.h.p));
+            if (in16) TRY(launch_dep(rmsnorm_bf16_kernel, dim3(T), dim3(256), 0, (const float*)m.x.p, D, D, L.norm1, gv, eps, m.abf.p));
+            else TRY(launch_dep(rmsnorm_kernel, dim3(T), dim3(nt), 0, (const float*)m.x.p, D, (const int*)nullptr, D, L.norm1, gv, eps, m.h.p));
             LAUNCHED();
             in = m.h.p;
         }
@@ -1431,11 +1511,15 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
         const bool sparse = routed && few && bf && d.experts > 0 && T * rper <= 40 * 1024;   // the router first, then only the chosen experts' rows
         if (dense) {   // the activation rides in the product's epilogue, its columns go straight to the back product's rows
             Fuse f = few ? fn : Fuse{};
-            f.glu = GluCols{F, d.ff_act, L.off_up, 0.f, ffo, KB, 1};
-            TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, L.n_front, D, EPI_NONE, 1.f, &f));
+            f.glu = GluCols{F, d.ff_act, L.off_up, 0.f, ffo, KB, 1, nullptr};
+            if (out16) f.glu.out16 = m.act16.p + L.back_ff;
+            if (in16) TRY(gemm_tc(m, m.abf.p, D, L.front, m.proj.p, nf, T, L.n_front, D, EPI_NONE, 1.f, 0.f, &f.glu));
+            else TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, L.n_front, D, EPI_NONE, 1.f, &f));
+        } else if (in16) {
+            TRY(gemm_tc(m, m.abf.p, D, L.front, m.proj.p, nf, T, L.n_front, D));
         } else if (few && gated) {
             Fuse f = fn;
-            f.glu = GluCols{F, d.ff_act, L.off_up, d.ff_limit, ffo, KB, 0};
+            f.glu = GluCols{F, d.ff_act, L.off_up, d.ff_limit, ffo, KB, 0, nullptr};
             TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, L.off_up + F, D, EPI_NONE, 1.f, &f));
         } else {
             TRY(gemm(m, in, D, L.front, m.proj.p, nf, T, sparse ? L.off_up : L.n_front, D, EPI_NONE, 1.f, few ? &fn : nullptr));
@@ -1520,6 +1604,11 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
                 fk.kskip = ExpertSkip{used, L.back_ff, F, Ex};
             }
             TRY(moe_act(L, nf, wdense, ffo, KB));
+        }
+        if (out16) {   // (the activation is there already: only the mixers' columns are left to round)
+            rows_to_bf16_kernel<<<grid_for((size_t)T * L.back_ff / 4), 256, 0, g_stream>>>(m.act.p, KB, T, L.back_ff, m.act16.p, KB);
+            LAUNCHED();
+            return gemm_tc(m, m.act16.p, KB, L.back, m.x.p, D, T, D, KB, EPI_ADD);
         }
         return gemm(m, m.act.p, KB, L.back, m.x.p, D, T, D, KB, EPI_ADD, 1.f, &fk);
     };
@@ -2325,7 +2414,12 @@ int ti_seq_model_finalize(ti_seq_model_t h) {
                 transpose_heads_kernel<float><<<grid_for(n), 256, 0, g_stream>>>((const float*)P(p + "mix.uk"), H, L.d.dim, L.d.kv_rank, (float*)L.ukT.p);
             LAUNCHED();
             CK(cudaStreamSynchronize(g_stream));
-            release(p + "mix.uk");
+            // prompt portions may expand keys and values (bf16 mode, no rotated part, sizes of the tensor-core attention)
+            if (m.d.mode == TI_SEQ_BF16 && g_use_tc && L.d.rot_dims == 0 && L.d.kv_rank >= 64 && L.d.kv_rank % 8 == 0 && L.d.dim <= 128 && L.d.vdim <= 128 && L.d.dim % 4 == 0 &&
+                L.d.vdim % 4 == 0 && H * L.d.dim >= 64 && H * L.d.vdim >= 64 && (reinterpret_cast<uintptr_t>(P(p + "mix.uk")) & 15) == 0 && (reinterpret_cast<uintptr_t>(P(p + "mix.uv")) & 15) == 0) {
+                L.uk = P(p + "mix.uk");
+                m.any_expand = true;
+            } else release(p + "mix.uk");
             L.uv = P(p + "mix.uv");
             ti_seq_layer_desc rd = L.d;   // frequencies of the rotated part: every pair of it turns
             rd.rot_scaled = 0;

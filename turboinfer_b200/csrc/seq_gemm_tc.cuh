@@ -135,7 +135,19 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                 const int nbase = nb * kSgBN + c0;
                 if (g.cols.ff > 0 && nbase + 16 > g.cols.first) {   // activated columns (and the last plain ones beside them)
                     float* orow = g.cols.out + (size_t)row * g.cols.ld - g.cols.first;
-                    if (nbase >= g.cols.first && nbase + 16 <= g.N && (reinterpret_cast<uintptr_t>(orow + nbase) & 15) == 0) {
+                    __nv_bfloat16* hrow = g.cols.out16 + (size_t)row * g.cols.ld - g.cols.first;
+                    if (g.cols.out16 && nbase >= g.cols.first && nbase + 16 <= g.N && (reinterpret_cast<uintptr_t>(hrow + nbase) & 15) == 0) {
+#pragma unroll
+                        for (int i = 0; i < 16; i += 8) {
+                            uint32_t pk[4];
+#pragma unroll
+                            for (int q = 0; q < 4; ++q) {
+                                const __nv_bfloat162 h2 = __floats2bfloat162_rn(ff_act(__uint_as_float(a[i + 2 * q]), g.cols.act), ff_act(__uint_as_float(a[i + 2 * q + 1]), g.cols.act));
+                                pk[q] = *reinterpret_cast<const uint32_t*>(&h2);
+                            }
+                            *reinterpret_cast<uint4*>(hrow + nbase + i) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
+                        }
+                    } else if (!g.cols.out16 && nbase >= g.cols.first && nbase + 16 <= g.N && (reinterpret_cast<uintptr_t>(orow + nbase) & 15) == 0) {
 #pragma unroll
                         for (int i = 0; i < 16; i += 4)
                             *reinterpret_cast<float4*>(orow + nbase + i) = make_float4(ff_act(__uint_as_float(a[i]), g.cols.act), ff_act(__uint_as_float(a[i + 1]), g.cols.act),
@@ -145,7 +157,8 @@ gemm_bf16_tc_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
                         for (int i = 0; i < 16; ++i) {
                             const int n = nbase + i;
                             if (n >= g.N) break;
-                            if (n >= g.cols.first) orow[n] = ff_act(__uint_as_float(a[i]), g.cols.act);
+                            if (n >= g.cols.first && g.cols.out16) hrow[n] = __float2bfloat16_rn(ff_act(__uint_as_float(a[i]), g.cols.act));
+                            else if (n >= g.cols.first) orow[n] = ff_act(__uint_as_float(a[i]), g.cols.act);
                             else epi_put(g.C + (size_t)row * g.ldc + n, __uint_as_float(a[i]), g.epi, g.alpha, g.beta);
                         }
                     }

@@ -100,6 +100,30 @@ __global__ void rmsnorm_kernel(const float* x, int ldx, const int* rows, int D, 
     const float sc = 1.f / sqrtf(ss / (float)D + eps);
     for (int d = threadIdx.x; d < D; d += blockDim.x) y[(size_t)t * D + d] = xr[d] * sc * gain[gvec ? d : 0];
 }
+// The same norm of whole rows with the result rounded to bf16 (the input of a tensor-core product); D a multiple of 4
+__global__ void __launch_bounds__(256) rmsnorm_bf16_kernel(const float* x, int ldx, int D, const float* gain, int gvec, float eps, __nv_bfloat16* y) {
+    pdl_launch_dependents();
+    pdl_wait_prior_grid();
+    __shared__ float red[32];
+    const int t = blockIdx.x;
+    const float* xr = x + (size_t)t * ldx;
+    float ss = 0.f;
+    for (int d = threadIdx.x * 4; d < D; d += blockDim.x * 4) {
+        const float4 v = *reinterpret_cast<const float4*>(xr + d);
+        ss += (v.x * v.x + v.y * v.y) + (v.z * v.z + v.w * v.w);
+    }
+    ss = block_sum(ss, red);
+    const float sc = 1.f / sqrtf(ss / (float)D + eps);
+    for (int d = threadIdx.x * 4; d < D; d += blockDim.x * 4) {
+        const float4 v = *reinterpret_cast<const float4*>(xr + d);
+        const float4 g = gvec ? *reinterpret_cast<const float4*>(gain + d) : make_float4(gain[0], gain[0], gain[0], gain[0]);
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x * sc * g.x, v.y * sc * g.y), hi = __floats2bfloat162_rn(v.z * sc * g.z, v.w * sc * g.w);
+        uint2 pk;
+        pk.x = *reinterpret_cast<const uint32_t*>(&lo);
+        pk.y = *reinterpret_cast<const uint32_t*>(&hi);
+        *reinterpret_cast<uint2*>(y + (size_t)t * D + d) = pk;
+    }
+}
 // The end of a sublayer: x[t] += norm(m[t]) with m = the sublayer's result, optionally
 //   * multiplied first by sigmoid(gate[t][d] + gate_bias[d]) (a gated residual: `gate` is a slice of the sublayer's fused input
 //     projection, row stride gate_ld), and
@@ -328,6 +352,7 @@ struct GluCols {
     float* out;
     int ld;
     int single;
+    __nv_bfloat16* out16;   // single, tcgen05 product only: the activated columns go here as bf16 instead of to out
 };
 // eight consecutive weights as they lie in memory (kept packed while the loads are in flight) and as fp32
 template <typename WT> struct Raw8;
@@ -826,6 +851,8 @@ struct AttnShape {
     const float* pb;                  // [heads] or null: no softmax, a visible key's weight is sigmoid(score + pb[h])
     int out_ld = 0;                   // row stride of the output; 0: heads * vdim
     float out_scale = 1.f;            // factor on the output
+    const float* egate = nullptr;     // window_attention_h3_kernel: the output coordinate is multiplied by sigmoid(egate[t * egate_ld + h * vdim + c])
+    int egate_ld = 0;
     int chunk = 0;                    // > 0: a row sees no key in front of its own chunk of positions (pos / chunk * chunk)
 };
 // the first key position a row at `pos` sees (never later for an earlier row)
@@ -1456,8 +1483,8 @@ __global__ void gather_rows_kernel(const float* x, const int* rows, int D, float
     const int t = blockIdx.x;
     for (int d = threadIdx.x; d < D; d += blockDim.x) y[(size_t)t * D + d] = x[(size_t)rows[t] * D + d];
 }
-// A[M][lda] (fp32) -> Y[M][K] (bf16, dense rows), four elements a thread; K a multiple of 4
-__global__ void rows_to_bf16_kernel(const float* A, int lda, int M, int K, __nv_bfloat16* y) {
+// A[M][lda] (fp32) -> Y[M][ldy] (bf16), K columns, four elements a thread; K and ldy multiples of 4
+__global__ void rows_to_bf16_kernel(const float* A, int lda, int M, int K, __nv_bfloat16* y, int ldy) {
     const size_t n4 = (size_t)M * (K / 4);
     const bool vec = (lda % 4 == 0) && ((reinterpret_cast<uintptr_t>(A) & 15) == 0);
     for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n4; i += (size_t)gridDim.x * blockDim.x) {
@@ -1466,7 +1493,7 @@ __global__ void rows_to_bf16_kernel(const float* A, int lda, int M, int K, __nv_
         float4 v;
         if (vec) v = *reinterpret_cast<const float4*>(src);
         else v = make_float4(src[0], src[1], src[2], src[3]);
-        __nv_bfloat162* d = reinterpret_cast<__nv_bfloat162*>(y + r * K + c);
+        __nv_bfloat162* d = reinterpret_cast<__nv_bfloat162*>(y + r * ldy + c);
         d[0] = __floats2bfloat162_rn(v.x, v.y);
         d[1] = __floats2bfloat162_rn(v.z, v.w);
     }

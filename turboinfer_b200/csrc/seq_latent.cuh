@@ -10,6 +10,10 @@
 // sliding window, chunks, a sink term and an output gate are the layer's choice: a gate of one number a head commutes with Uv and is
 // applied to the weighted sum, a gate per coordinate in the epilogue of the product with Uv).  rot may be 0: no rotated part.  This file
 // holds what is special: the cache append and the query's rotated part.
+//
+// A prompt portion may also go the direct way: keys Uk_h c_j and values Uv_h c_j of its sequence's cached rows are expanded once per step
+// (latent_gather_kernel and two products), and the portion attends with heads of its own size -- (dim + vdim) instead of 2 rank
+// multiply-adds a pair and head, which pays as soon as the portion has more than a few rows.
 #pragma once
 #include "seq_attn_tc.cuh"
 #include "seq_kernels.cuh"
@@ -73,6 +77,21 @@ __global__ void transpose_heads_kernel(const WT* uk, int heads, int dim, int ran
     for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
         const size_t h = i / ((size_t)dim * rank), r = (i / dim) % rank, d = i % dim;
         out[i] = uk[(h * dim + d) * rank + r];
+    }
+}
+
+// Cached rows of whole pages as bf16, page after page: row r = rows[pages[r / 64] * 64 + r % 64] of the pool (row stride ld, `rank`
+// leading coordinates, in fours) -- the input of the products that expand a sequence's keys and values for a prompt portion
+__global__ void latent_gather_kernel(const float* pool, int ld, int rank, const int* pages, int n_rows, __nv_bfloat16* y) {
+    pdl_launch_dependents();
+    pdl_wait_prior_grid();
+    const size_t n = (size_t)n_rows * (rank / 4);
+    for (size_t i = blockIdx.x * (size_t)blockDim.x + threadIdx.x; i < n; i += (size_t)gridDim.x * blockDim.x) {
+        const size_t r = i / (rank / 4), c = (i % (rank / 4)) * 4;
+        const float4 v = *reinterpret_cast<const float4*>(pool + ((size_t)pages[r / kPageTokens] * kPageTokens + r % kPageTokens) * ld + c);
+        __nv_bfloat162* d = reinterpret_cast<__nv_bfloat162*>(y + r * rank + c);
+        d[0] = __floats2bfloat162_rn(v.x, v.y);
+        d[1] = __floats2bfloat162_rn(v.z, v.w);
     }
 }
 
