@@ -66,6 +66,10 @@ MECHANISMS = {
     "latent_rank_512": make_config([latent(heads=2, dim=16, vdim=32, kv_rank=512, q_rank=24)], width=64),
     "latent_rank_300": make_config([latent(heads=3, dim=20, vdim=12, kv_rank=300, q_rank=24)], width=64),
     "latent_rank_600": make_config([latent(heads=2, dim=8, vdim=8, kv_rank=600, q_rank=24)], width=64),
+    "latent_rank_128_large_heads": make_config([latent(heads=2, dim=120, vdim=140, kv_rank=128, q_rank=32)], width=64),   # (not worth expanding: on the cached rows themselves)
+    "latent_rank_256_large_heads": make_config([latent(heads=2, dim=136, vdim=24, kv_rank=256, q_rank=32)], width=64),
+    "latent_rank_512_large_heads": make_config([latent(heads=2, dim=16, vdim=132, kv_rank=512, q_rank=32)], width=64),
+    "latent_heads_wider_than_the_rank": make_config([latent(heads=2, dim=128, vdim=128, kv_rank=96, q_rank=32)], width=64),
     "latent_rank_one": make_config([latent(heads=2, dim=3, vdim=2, kv_rank=1, q_rank=1)]),
     "delta_one_tap": make_config([delta(conv=1)]),
     "delta_nine_taps": make_config([delta(conv=9)]),
@@ -416,6 +420,27 @@ def test_keys_that_repeat_and_keys_that_barely_exist():
             check_logits(whole(m, toks), ref, dtype)
             check_logits(run_schedule(m, {"a": toks}, [[("a", 100)]] + [[("a", 1)]] * 70)["a"], ref, dtype)
             m.free()
+
+
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_decays_from_none_to_everything(dtype):
+    """Logarithms of the decay between -0.001 and -1000 a token in the same head: sums over a portion are large, differences between
+    neighbouring tokens small, and a state survives the one and not the other."""
+    cfg = make_config([delta(heads=4, kv_heads=2, dim=32, vdim=24, conv=2), delta(heads=2, kv_heads=1, dim=128, vdim=16, conv=4)], width=64)
+    W = random_weights(cfg, seed=30)
+    W["l0.mix.A_log"] = to_bf16_values(np.array([-8.0, 0.0, 3.0, 5.0], np.float32))
+    W["l1.mix.A_log"] = to_bf16_values(np.array([4.0, -3.0], np.float32))
+    for i in range(2):
+        W["l%d.mix.a" % i] = to_bf16_values(W["l%d.mix.a" % i] * 6.0)
+        W["l%d.mix.dt_bias" % i] = to_bf16_values(np.full_like(W["l%d.mix.dt_bias" % i], -6.0))
+    lg = np.log(np.maximum(plain.delta_decay({k: np.asarray(v, np.float64) for k, v in W.items()}, "l0.mix.", plain.norm(W["embed"].astype(np.float64), W["l0.norm1"], 1e-5)), 1e-300))
+    assert lg[:, 3].min() < -300 and lg[:, 3].max() > -0.5
+    toks = tokens(300, cfg["vocab"], 5)
+    want, _ = plain.run(cfg, W, toks)
+    m = build_engine(cfg, W, dtype)
+    for sizes in ([300], [100, 7, 193], [250] + [1] * 50):
+        check_logits(run_schedule(m, {"a": toks}, [[("a", n)] for n in sizes])["a"], want, dtype)
+    m.free()
 
 
 def test_states_cross_every_cut():

@@ -15,7 +15,7 @@ namespace tib {
 namespace seq {
 
 constexpr int kAttnTcTile = kTcQ;   // 128 rows a block
-template <int DK, int DV> constexpr size_t window_h3_smem_bytes() { return 2 * sizeof(__half) * ((size_t)(kTcQ + kTcKT) * (DK + 8) + (size_t)kTcKT * (DV + 8)); }
+template <int DK, int DV> constexpr size_t window_h3_smem_bytes() { return 2 * sizeof(__half) * ((size_t)(kTcQ + kTcKT) * (DK + 8) + (size_t)kTcKT * (DV + 8)) + sizeof(float) * (size_t)kTcKT * (DK + DV); }
 
 template <int DK, int DV, bool SIZED>
 __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(const float* qkvg, StepMeta m, AttnShape s, const int* tiles,
@@ -29,7 +29,9 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
     __half* Kl = Kh + kTcKT * LD;
     __half* Vh = Kl + kTcKT * LD;
     __half* Vl = Vh + kTcKT * LDV;
-    const int row0 = tiles[2 * blockIdx.x], M = tiles[2 * blockIdx.x + 1], h = blockIdx.y;
+    float* Kr = reinterpret_cast<float*>(Vl + kTcKT * LDV);   // [64][DK], [64][DV]: the next tile's rows as they are cached
+    float* Vr = Kr + kTcKT * DK;
+    const int row0 = tiles[2 * blockIdx.y], M = tiles[2 * blockIdx.y + 1], h = blockIdx.x;   // (heads run fastest: the tiles come longest first)
     const int pos0 = m.row_pos[row0];
     const int* table = m.page_table + (size_t)m.ent_slot[m.row_ent[row0]] * m.table_stride;
     const int gkv = h / (s.heads / s.kv_heads);
@@ -66,35 +68,37 @@ __global__ void __launch_bounds__(kTcThreads, 1) window_attention_h3_kernel(cons
     const uint32_t v_ld = (uint32_t)(((lr + 8 * (lm & 1)) * LDV + 8 * (lm >> 1)) * 2);
     const uint32_t kh_s = smem_u32(Kh), kl_s = smem_u32(Kl), vh_s = smem_u32(Vh), vl_s = smem_u32(Vl);
     const size_t kpitch = (size_t)s.kv_heads * d, vpitch = (size_t)s.kv_heads * dv;
-    for (int t0 = lo / kPageTokens * kPageTokens; t0 <= last_pos; t0 += kTcKT) {   // a key tile = a page
-        __syncthreads();
+    // the raw rows of the next key tile are on their way (cp.async) while the warps work on this one's halves
+    auto fetch = [&](int t0) {
         const size_t tok0 = (size_t)table[t0 / kPageTokens] * kPageTokens;
-        if constexpr (DK == DV) {
-            for (int i = tid; i < kTcKT * (DK / 4); i += kTcThreads) {
-                const int kk = i / (DK / 4), d4 = (i % (DK / 4)) * 4, tk = t0 + kk;
-                float4 kv = make_float4(0.f, 0.f, 0.f, 0.f), vv = kv;
-                if (tk >= lo && tk <= last_pos) {
-                    if (d4 < d) kv = *reinterpret_cast<const float4*>(k_pool + (tok0 + kk) * kpitch + (size_t)gkv * d + d4);
-                    if (d4 < dv) vv = *reinterpret_cast<const float4*>(v_pool + (tok0 + kk) * vpitch + (size_t)gkv * dv + d4);
-                }
-                store_split4(kv, Kh + kk * LD + d4, Kl + kk * LD + d4);
-                store_split4(vv, Vh + kk * LDV + d4, Vl + kk * LDV + d4);
-            }
-        } else {
-            for (int i = tid; i < kTcKT * (DK / 4); i += kTcThreads) {
-                const int kk = i / (DK / 4), d4 = (i % (DK / 4)) * 4, tk = t0 + kk;
-                float4 kv = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (tk >= lo && tk <= last_pos && d4 < d) kv = *reinterpret_cast<const float4*>(k_pool + (tok0 + kk) * kpitch + (size_t)gkv * d + d4);
-                store_split4(kv, Kh + kk * LD + d4, Kl + kk * LD + d4);
-            }
-            for (int i = tid; i < kTcKT * (DV / 4); i += kTcThreads) {
-                const int kk = i / (DV / 4), d4 = (i % (DV / 4)) * 4, tk = t0 + kk;
-                float4 vv = make_float4(0.f, 0.f, 0.f, 0.f);
-                if (tk >= lo && tk <= last_pos && d4 < dv) vv = *reinterpret_cast<const float4*>(v_pool + (tok0 + kk) * vpitch + (size_t)gkv * dv + d4);
-                store_split4(vv, Vh + kk * LDV + d4, Vl + kk * LDV + d4);
-            }
+        for (int i = tid; i < kTcKT * (DK / 4); i += kTcThreads) {
+            const int kk = i / (DK / 4), d4 = (i % (DK / 4)) * 4, tk = t0 + kk;
+            const bool ok = tk >= lo && tk <= last_pos && d4 < d;
+            cp_async16(Kr + kk * DK + d4, k_pool + (ok ? (tok0 + kk) * kpitch + (size_t)gkv * d + d4 : 0), ok);
+        }
+        for (int i = tid; i < kTcKT * (DV / 4); i += kTcThreads) {
+            const int kk = i / (DV / 4), d4 = (i % (DV / 4)) * 4, tk = t0 + kk;
+            const bool ok = tk >= lo && tk <= last_pos && d4 < dv;
+            cp_async16(Vr + kk * DV + d4, v_pool + (ok ? (tok0 + kk) * vpitch + (size_t)gkv * dv + d4 : 0), ok);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    fetch(lo / kPageTokens * kPageTokens);
+    for (int t0 = lo / kPageTokens * kPageTokens; t0 <= last_pos; t0 += kTcKT) {   // a key tile = a page
+        asm volatile("cp.async.wait_group 0;" ::: "memory");
+        __syncthreads();
+#pragma unroll 4
+        for (int i = tid; i < kTcKT * (DK / 4); i += kTcThreads) {
+            const int kk = i / (DK / 4), d4 = (i % (DK / 4)) * 4;
+            store_split4(*reinterpret_cast<const float4*>(Kr + kk * DK + d4), Kh + kk * LD + d4, Kl + kk * LD + d4);
+        }
+#pragma unroll 4
+        for (int i = tid; i < kTcKT * (DV / 4); i += kTcThreads) {
+            const int kk = i / (DV / 4), d4 = (i % (DV / 4)) * 4;
+            store_split4(*reinterpret_cast<const float4*>(Vr + kk * DV + d4), Vh + kk * LDV + d4, Vl + kk * LDV + d4);
         }
         __syncthreads();
+        if (t0 + kTcKT <= last_pos) fetch(t0 + kTcKT);
         if (t0 > warp_last || t0 + kTcKT - 1 < warp_lo || 16 * warp >= M) continue;   // nothing of this page is visible to the warp's rows
         float sc[kTcKT / 8][4];
 #pragma unroll

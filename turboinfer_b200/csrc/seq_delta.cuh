@@ -407,9 +407,6 @@ __global__ void __launch_bounds__(256) delta_chunk_prepare_kernel(DeltaChunkArgs
     }
 }
 
-__device__ __forceinline__ void cp_async16(float* dst, const float* src, bool valid) {   // (16 bytes of zeros when not valid)
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
-}
 template <int DKP> constexpr size_t delta_chunk_smem_bytes() {
     return sizeof(float) * (2 * (size_t)kDeltaChunk * (DKP + 8) + (size_t)kDeltaChunk * (DKP + 16) + (size_t)kDeltaChunk * 72 + (size_t)kDeltaChunk * 36 + (size_t)DKP * 20);
 }

@@ -994,6 +994,18 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
             r0 += counts[e];
         }
     }
+    // longest first: a tile's work grows with its last position (the blocks of the last ones fill the gaps at the end of a launch)
+    const auto longest_first = [&](std::vector<int>& v) {
+        std::vector<std::pair<int, int>> p(v.size() / 2);
+        for (size_t i = 0; i < p.size(); ++i) p[i] = {v[2 * i], v[2 * i + 1]};
+        std::vector<int> last(T);
+        for (int e = 0, r = 0; e < E; ++e)
+            for (int i = 0; i < counts[e]; ++i, ++r) last[r] = m.seqs[seqs[e]].len + i;
+        std::stable_sort(p.begin(), p.end(), [&](const auto& a, const auto& b) { return last[a.first] + a.second > last[b.first] + b.second; });
+        for (size_t i = 0; i < p.size(); ++i) { v[2 * i] = p[i].first; v[2 * i + 1] = p[i].second; }
+    };
+    longest_first(tiles);
+    longest_first(tiles128);
     const int n_tiles = (int)tiles.size() / 2, n_tiles128 = (int)tiles128.size() / 2, n_small = (int)small_rows.size();
     // the head-mixing attention cuts EVERY entry into tiles of up to 64 rows and wants the tile of every row
     std::vector<int> mtiles, row_tile;
@@ -1210,7 +1222,7 @@ int run_step(Model& m, int E, const int32_t* seqs, const int32_t* counts, const 
     // paged softmax attention of all rows of the step (prompt portions in tiles, the other rows one by one or split over their keys)
     auto h3_size = [](const AttnShape& s) { return s.dim <= 128 && s.vdim <= 128 && s.dim % 4 == 0 && s.vdim % 4 == 0 && s.v_ld == 0; };
     auto h3_attention = [&](const StepMeta& sm, const AttnShape& s, const float* q, const float* kp, const float* vp, float* out) -> int {   // the portions' tiles
-        const dim3 grid(n_tiles128, s.heads);
+        const dim3 grid(s.heads, n_tiles128);
         const int dk = s.dim <= 64 ? 64 : 128, dv = s.vdim <= 64 ? 64 : 128;
         const bool sized = dk == s.dim && dv == s.vdim;
 #define TI_H3_CASE(K, V, X) window_attention_h3_kernel<K, V, X><<<grid, kTcThreads, window_h3_smem_bytes<K, V>(), g_stream>>>(q, sm, s, d_tiles128, kp, vp, out)

@@ -50,6 +50,10 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
     return s;
 }
 
+__device__ __forceinline__ void cp_async16(float* dst, const float* src, bool valid) {   // (16 bytes of zeros when not valid; both 16-byte aligned)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_u32(dst)), "l"(src), "r"(valid ? 16 : 0) : "memory");
+}
+
 // ---- embedding -----------------------------------------------------------------------------------------------------
 // x[t] = embed[tok[t]] (+ the sinusoidal position vector: entry 2i = sin(pos * pos_freq[i]), entry 2i + 1 = cos of the same angle,
 // angle and functions in fp32); x0 (optional) keeps the embedding output for the looped block's input projection; copies > 1: the row

@@ -447,7 +447,7 @@ def nubipel_descs(cfg: dict, mode: int, max_tokens: int, max_seqs: int):
     m.norm_eps = float(_req(_req(cfg, "norm", "the model"), "eps", "norm"))
     m.norm_kind, m.norm_place = _seq.NORM_VECTOR, _seq.NORMS_SHARED
     m.embed_scale = float(_req(_req(cfg, "embedding", "the model"), "scale", "embedding"))
-    m.logit_scale, m.logit_softcap = float(_req(cfg, "logit_scale", "the model")), float(_req(cfg, "logit_softcap", "the model"))
+    m.logit_scale, m.logit_softcap = float(_req(cfg, "logit_scale", "the model")), float(_req(cfg, "logit_softcap", "the model") or 0.0)
     m.tied_head = 1
     m.mode, m.max_tokens, m.max_seqs = mode, int(max_tokens), int(max_seqs)
     return m, layers
