@@ -194,9 +194,9 @@ __device__ __forceinline__ unsigned long long argmax_pack(float v, int idx) {
 
 // ---- shared-memory carve-up ------------------------------------------------------------------------
 // The block starts at the kernel's dynamic shared memory (declared 128-byte aligned) and is carved with plain pointer
-// arithmetic on that array: the compiler then knows every pointer is a shared-memory one and emits LDS / STS / ATOMS and
-// constant shared-window addresses.  (Carving through uintptr_t, as the first version did, loses the address space: every
-// access became a generic LD / ST / ATOM, several times slower, and every barrier address a ~10-instruction conversion.)
+// arithmetic on that array: the compiler then knows that every pointer is a shared-memory one.  (Carving through uintptr_t, as
+// the first version did, loses the address space: accesses become generic ones and barrier addresses need a conversion; the
+// kernel was several times slower.)
 // The mbarriers and the ring come first so that their addresses are compile-time offsets from the base.
 constexpr int kBarBlockBytes = 128;   // full[kMaxStages], empty[kMaxStages], padding
 struct GemvSmem {

@@ -672,7 +672,7 @@ __global__ void __maxnreg__(96) mega_decode_kernel(const __grid_constant__ MegaA
     extern __shared__ __align__(128) uint8_t smem_raw[];
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
     // carve: mbarriers | ring | x digits | column sums | reduction scratch | attention scratch | phase descriptors -- plain
-    // pointer arithmetic on the shared array (every block is a multiple of 16 bytes), so that the accesses stay LDS / STS
+    // pointer arithmetic on the shared array (every block is a multiple of 16 bytes), so that the address space is known
     uint8_t* tail = nullptr;
     const GemvSmem sm = gemv_carve_for(smem_raw, m.stages, m.max_kpad, m.max_units, &tail);
     float* attn_sm = reinterpret_cast<float*>(tail);
